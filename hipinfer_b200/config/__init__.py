@@ -7,6 +7,8 @@ from .vegodra import (ChunkedAttentionConfig, GlaConfig, LatentAttentionConfig, 
 from .runopel import DenseFFConfig, Mamba2Config, RoutedFFConfig, RunopelConfig, RunopelLayerConfig, WindowLatentConfig
 from .mavinex import (MavinexConfig, MavinexLayerConfig, ScaledRotaryConfig, SelectiveScanConfig, SideBySideConfig,
                       SinkLatentConfig, WindowAttentionConfig)
+from .gakupel import (DistanceAttentionConfig, GakupelConfig, GakupelLayerConfig, GatedDeltaConfig, GeluFFConfig, GroupedExpertsConfig,
+                      MatrixMemoryConfig, ParallelMixerConfig, QueryTemperatureConfig, SharedKeyAttentionConfig)
 
 __all__ = ["Architecture", "ConfigError", "ModelConfig", "config_from_dict", "get_architecture", "load_config",
            "register_architecture", "registered_architectures", "save_config", "take", "Llama3RopeScaling",
@@ -14,4 +16,5 @@ __all__ = ["Architecture", "ConfigError", "ModelConfig", "config_from_dict", "ge
            "ChunkedAttentionConfig", "GlaConfig", "LatentAttentionConfig", "RotaryConfig", "VegodraConfig", "VegodraLayerConfig",
            "DenseFFConfig", "Mamba2Config", "RoutedFFConfig", "RunopelConfig", "RunopelLayerConfig", "WindowLatentConfig",
            "MavinexConfig", "MavinexLayerConfig", "ScaledRotaryConfig", "SelectiveScanConfig", "SideBySideConfig", "SinkLatentConfig",
-           "WindowAttentionConfig"]
+           "WindowAttentionConfig", "DistanceAttentionConfig", "GakupelConfig", "GakupelLayerConfig", "GatedDeltaConfig", "GeluFFConfig",
+           "GroupedExpertsConfig", "MatrixMemoryConfig", "ParallelMixerConfig", "QueryTemperatureConfig", "SharedKeyAttentionConfig"]

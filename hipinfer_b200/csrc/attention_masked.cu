@@ -6,6 +6,7 @@
 //     mask 2 (chunk):   floor(j / chunk) == floor(p / chunk), chunks counted from position 0 of the sequence
 // The softmax may have a sink: a number per head that joins the denominator as exp(sink), with no key and no value,
 // unscaled, once. The head's result may be multiplied by sigmoid of a gate, one number per element or one per head.
+// A distance bias (r1, r2: a number per head) is taken off the score: r1 ln(1 + r2 (p - j)).
 // Keys are D wide and values E wide; each plane is addressed by a row stride of its own, so that the values may be
 // the first E columns of the key rows (a latent that serves as both). Query head h reads kv head h / (H / G).
 // Scores, the running maximum and sums, exp and the sums over values are 32-bit; the result is rounded once, into an
@@ -40,6 +41,7 @@ struct MaskedArgs {
   float* part;                      // [T][G][ZT][splits][RT][E + 2]
   int* arrived;                     // [T][G][ZT] zeroed counters; the last block leaves 0
   int splits;
+  const float* r1; const float* r2; // [H] or null: the distance bias
 };
 
 __device__ __forceinline__ void ma_range(const MaskedArgs& A, int p, int& lo, int& keep) {
@@ -116,6 +118,7 @@ __global__ void __launch_bounds__(MA_THREADS) attn_masked_rows_kernel(MaskedArgs
           const float* qr = qs + r * D;
           a = 0.f;
           for (int d = 0; d < D; d++) a = fmaf(qr[d], hb_to_float(kr[d]), a);
+          if (A.r1) a -= A.r1[head0 + r] * logf(fmaf(A.r2[head0 + r], (float)(p - (k0 + j)), 1.f));
         }
         sc[r * MK + j] = a;
       }
@@ -252,7 +255,7 @@ HB_EXPORT int hb_attn_masked(const void* q, int q_dt, long ldq, const void* kc, 
                              const float* gate, long ld_gate, int gate_off, int gate_mode, void* out, int o_dt, long ldo,
                              int T, int H, int G, int D, int E, int page_size, int mask, int window, int keep_first,
                              int chunk, float scale, const int* q_len, int row_limit, float* part, long n_part,
-                             int* arrived, int max_pos, cudaStream_t s) {
+                             int* arrived, int max_pos, const float* r1, const float* r2, cudaStream_t s) {
   if (T <= 0) return 0;
   if (G <= 0 || H % G) HB_FAIL("hb_attn_masked: %d heads are not a multiple of %d kv heads", H, G);
   if (T > 65535) HB_FAIL("hb_attn_masked: %d rows are beyond the grid limit", T);
@@ -261,7 +264,8 @@ HB_EXPORT int hb_attn_masked(const void* q, int q_dt, long ldq, const void* kc, 
   A.row_req = row_req; A.pos = pos; A.sink = sink; A.gate = gate; A.ld_gate = ld_gate; A.gate_off = gate_off;
   A.gate_mode = gate ? gate_mode : 0; A.out = out; A.ldo = ldo; A.H = H; A.G = G; A.D = D; A.E = E; A.page_size = page_size;
   A.mask = mask; A.window = window; A.keep_first = keep_first; A.chunk = chunk; A.scale = scale; A.q_len = q_len;
-  A.row_limit = row_limit; A.part = part; A.arrived = arrived;
+  A.row_limit = row_limit; A.part = part; A.arrived = arrived; A.r1 = r1; A.r2 = r2;
+  if ((r1 != nullptr) != (r2 != nullptr)) HB_FAIL("hb_attn_masked: a distance bias needs both of its vectors");
   const int HG = H / G;
   A.RT = ma_head_tile(HG, D, E, 96 * 1024);
   const int ZT = (HG + A.RT - 1) / A.RT;

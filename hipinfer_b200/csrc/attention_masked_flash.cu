@@ -27,6 +27,7 @@ struct FlashMaskedArgs {
   void* out; long ldo;
   int H, G, page_size, mask, window, keep_first, chunk;
   float scale;
+  const float* r1; const float* r2;     // [H] or null: r1 ln(1 + r2 (i - j)) is taken off the score
 };
 
 __device__ __forceinline__ void fm_cp16(uint32_t dst, const void* src) {
@@ -107,8 +108,20 @@ __global__ void __launch_bounds__(FM_THREADS) attn_masked_flash_kernel(FlashMask
     }
   };
 
+  // The distance bias of a tile: row minus key takes 127 values in it, so a thread makes one of them, a tile or two ahead
+  // (three slots: the one being read, the next, and the one being made); in units of log 2 as the scores are.
+  __shared__ float dist[3][FM_ROWS + FM_KEYS];
+  const float r1 = A.r1 ? A.r1[h] : 0.f, r2 = A.r1 ? A.r2[h] : 0.f;
+  auto distances = [&](int slot, int tile) {
+    dist[slot][tid] = r1 * log2f(fmaf(r2, (float)max(p0 - tile * FM_KEYS + tid - (FM_KEYS - 1), 0), 1.f));
+  };
+
   locate(0, tile_at(0));
   if (n_tiles > 1) locate(1, tile_at(1));
+  if (A.r1) {
+    distances(0, tile_at(0));
+    if (n_tiles > 1) distances(1, tile_at(1));
+  }
   __syncthreads();
   load_tile(0, 0);
   fm_commit();
@@ -150,7 +163,10 @@ __global__ void __launch_bounds__(FM_THREADS) attn_masked_flash_kernel(FlashMask
       fm_wait<0>();
     }
     __syncthreads();
-    if (it + 2 < n_tiles) locate(buf, tile_at(it + 2));     // this slot's copies are issued; visible after the next barrier
+    if (it + 2 < n_tiles) {
+      locate(buf, tile_at(it + 2));                         // this slot's copies are issued; visible after the next barrier
+      if (A.r1) distances((it + 2) % 3, tile_at(it + 2));
+    }
     const __nv_bfloat16* kt = Ks + buf * FM_KEYS * KP;
     const __nv_bfloat16* vt = Vs + buf * FM_KEYS * VP;
     float s[8][4];
@@ -173,7 +189,22 @@ __global__ void __launch_bounds__(FM_THREADS) attn_masked_flash_kernel(FlashMask
     float mx_a = -INFINITY, mx_b = -INFINITY;
     // a tile every key of which both rows see (the common case away from the diagonal and the mask's edge) needs no test
     const bool whole = va && vb && k0 + FM_KEYS - 1 <= pa && k0 >= lo_b;
-    if (whole) {
+    if (A.r1) {
+      const float* da = dist[it % 3] + ra - qi * 2 + (FM_KEYS - 1);        // da[-key]: the bias of row ra against the tile's key
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+#pragma unroll
+        for (int c = 0; c < 4; c++) {
+          const int kk = j * 8 + (c & 1), key = k0 + kk + qi * 2;
+          const bool top = c < 2;
+          const int p = top ? pa : pb, lo = top ? lo_a : lo_b, keep = top ? keep_a : keep_b;
+          const bool vis = whole || ((top ? va : vb) && key <= p && (key >= lo || key < keep));
+          const float v = vis ? fmaf(s[j][c], sl2, -da[(top ? 0 : 8) - kk]) : -INFINITY;
+          s[j][c] = v;
+          if (top) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
+        }
+      }
+    } else if (whole) {
 #pragma unroll
       for (int j = 0; j < 8; j++) {
         s[j][0] *= sl2; s[j][1] *= sl2; s[j][2] *= sl2; s[j][3] *= sl2;
@@ -276,7 +307,7 @@ __global__ void __launch_bounds__(FM_THREADS) attn_masked_flash_kernel(FlashMask
 }
 
 // the (D, E) pairs that are instantiated
-#define FM_SIZES(X) X(4, 8) X(4, 6) X(8, 16) X(6, 8) X(12, 16) X(2, 4) X(4, 4) X(8, 8) X(3, 4)
+#define FM_SIZES(X) X(6, 12) X(6, 6) X(3, 6) X(4, 8) X(4, 6) X(8, 16) X(6, 8) X(12, 16) X(2, 4) X(4, 4) X(8, 8) X(3, 4)
 
 HB_EXPORT int hb_attn_masked_flash_supported(int D, int E) {
 #define FM_CHECK(DK, EN) if (D == 16 * DK && E == 8 * EN) return 1;
@@ -290,15 +321,16 @@ HB_EXPORT int hb_attn_masked_flash(const void* q, long ldq, const void* kc, long
                                    const int* q_len, const int* ctx_len, int req0, int n_requests, int max_q_len, int row_limit,
                                    const float* sink, const float* gate, long ld_gate, int gate_off, int gate_mode, void* out,
                                    int o_dt, long ldo, int H, int G, int D, int E, int page_size, int mask, int window,
-                                   int keep_first, int chunk, float scale, cudaStream_t s) {
+                                   int keep_first, int chunk, float scale, const float* r1, const float* r2, cudaStream_t s) {
   if (n_requests <= 0 || max_q_len <= 0) return 0;
   if (G <= 0 || H % G) HB_FAIL("hb_attn_masked_flash: %d heads are not a multiple of %d kv heads", H, G);
   if (!hb_attn_masked_flash_supported(D, E)) HB_FAIL("hb_attn_masked_flash: keys of %d with values of %d are not a size it takes", D, E);
   if ((ldq | k_page | k_head | k_row | v_page | v_head | v_row) & 7 || (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15))
     HB_FAIL("hb_attn_masked_flash: rows of q, keys and values must start on 16-byte boundaries");
   if (H > 65535 || n_requests > 65535) HB_FAIL("hb_attn_masked_flash: the grid is too large");
+  if ((r1 != nullptr) != (r2 != nullptr)) HB_FAIL("hb_attn_masked_flash: a distance bias needs both of its vectors");
   FlashMaskedArgs A;
-  A.q = (const __nv_bfloat16*)q; A.ldq = ldq; A.kc = (const __nv_bfloat16*)kc; A.k_page = k_page; A.k_head = k_head; A.k_row = k_row;
+  A.r1 = r1; A.r2 = r2; A.q = (const __nv_bfloat16*)q; A.ldq = ldq; A.kc = (const __nv_bfloat16*)kc; A.k_page = k_page; A.k_head = k_head; A.k_row = k_row;
   A.vc = (const __nv_bfloat16*)vc; A.v_page = v_page; A.v_head = v_head; A.v_row = v_row; A.bt = bt; A.bt_stride = bt_stride;
   A.q_start = q_start; A.q_len = q_len; A.ctx_len = ctx_len; A.req0 = req0; A.row_limit = row_limit; A.sink = sink; A.gate = gate;
   A.ld_gate = ld_gate; A.gate_off = gate_off; A.gate_mode = gate ? gate_mode : 0; A.out = out; A.ldo = ldo; A.H = H; A.G = G;

@@ -31,6 +31,7 @@ struct HeadsArgs {
   const int* q_len; int row_limit;
   float* part;                          // [T][G][ZT][splits][16 MT][E + 4]
   int splits;
+  const float* r1; const float* r2;     // [H] or null: r1 ln(1 + r2 (p - j)) is taken off the score
 };
 
 __device__ __forceinline__ void hs_cp16(uint32_t dst, const void* src) {
@@ -125,6 +126,14 @@ __global__ void __launch_bounds__(HS_THREADS) attn_masked_heads_kernel(HeadsArgs
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
   const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(Qs + (mt * 16 + (lane & 15)) * KP + (lane >> 4) * 8);
 
+  // the distance bias of this thread's two heads
+  float r1a = 0.f, r2a = 0.f, r1b = 0.f, r2b = 0.f;
+  if (A.r1) {
+    const int ha = mt * 16 + quad, hb = ha + 8;
+    const size_t head = (size_t)g * HG + h0;
+    if (ha < nh) { r1a = A.r1[head + ha]; r2a = A.r2[head + ha]; }
+    if (hb < nh) { r1b = A.r1[head + hb]; r2b = A.r2[head + hb]; }
+  }
   // scores are kept in units of log 2 (scale * log2(e) folded into one factor): exp is then one exp2 an element
   const float sl2 = A.scale * 1.4426950408889634f;
   for (int it = i0; it < i1; it++) {
@@ -165,7 +174,8 @@ __global__ void __launch_bounds__(HS_THREADS) attn_masked_heads_kernel(HeadsArgs
       for (int c = 0; c < 4; c++) {
         const int key = k0 + j * 8 + qi * 2 + (c & 1);
         const bool vis = key <= p && (key >= lo || key < keep);
-        const float v = vis ? s[j][c] * sl2 : -INFINITY;
+        float v = vis ? s[j][c] * sl2 : -INFINITY;
+        if (A.r1 && vis) v -= (c < 2 ? r1a : r1b) * __log2f(fmaf(c < 2 ? r2a : r2b, (float)(p - key), 1.f));
         s[j][c] = v;
         if (c < 2) mx = fmaxf(mx, v); else mx_b = fmaxf(mx_b, v);
       }
@@ -203,6 +213,7 @@ __global__ void __launch_bounds__(HS_THREADS) attn_masked_heads_kernel(HeadsArgs
       pf[3] = hs_pack(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
       for (int n = 0; n < ENW; n += 2) {
+        if (e_base + n * 8 >= E) break;
         uint32_t b[4];
         asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                      : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(v_addr + (uint32_t)((kk * 16 * VP + n * 8) * 2)));
@@ -227,6 +238,7 @@ __global__ void __launch_bounds__(HS_THREADS) attn_masked_heads_kernel(HeadsArgs
 #pragma unroll
   for (int n = 0; n < ENW; n++) {
     const int e = e_base + n * 8 + qi * 2;
+    if (e >= E) break;
     stage[ra * RS + e] = o[n][0]; stage[ra * RS + e + 1] = o[n][1];
     stage[rb * RS + e] = o[n][2]; stage[rb * RS + e + 1] = o[n][3];
   }
@@ -385,9 +397,11 @@ static int hs_splits(int mask, int window, int keep_first, int chunk, int max_po
 static int hs_enw(int H, int G, int D, int E, int alias) {
   if (G <= 0 || H % G || D % 16 || E % 8 || D > 1024) return 0;
   const int MT = hs_mt(H / G), ES = 4 / MT;
-  if (E % (8 * ES)) return 0;
-  const int enw = E / 8 / ES;
-  if (enw != 2 && enw != 4 && enw != 8 && enw != 16 && enw != 32) return 0;
+  if (E % 16) return 0;
+  // the smallest built width that covers E in ES slices; a slice (or a part of one) beyond E does nothing
+  int enw = 2;
+  while (enw <= 32 && enw * 8 * ES < E) enw *= 2;
+  if (enw > 32) return 0;
   if (alias && E > D) return 0;
   if (hs_smem_bytes(MT, D, E, alias) > 200 * 1024) return 0;
   return enw;
@@ -406,15 +420,17 @@ HB_EXPORT int hb_attn_masked_heads(const void* q, long ldq, const void* kc, long
                                    const int* row_req, const int* pos, const float* sink, const float* gate, long ld_gate,
                                    int gate_off, int gate_mode, void* out, int o_dt, long ldo, int T, int H, int G, int D, int E,
                                    int page_size, int mask, int window, int keep_first, int chunk, float scale, const int* q_len,
-                                   int row_limit, float* part, long n_part, int max_pos, cudaStream_t s) {
+                                   int row_limit, float* part, long n_part, int max_pos, const float* r1, const float* r2,
+                                   cudaStream_t s) {
   if (T <= 0) return 0;
   const int enw = hs_enw(H, G, D, E, alias);
   if (!enw) HB_FAIL("hb_attn_masked_heads: %d heads over %d kv heads with keys of %d and values of %d are not sizes it takes", H, G, D, E);
   if (T > 65535) HB_FAIL("hb_attn_masked_heads: %d rows are beyond the grid limit", T);
   if ((ldq | k_page | k_head | k_row | v_page | v_head | v_row) & 7 || (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15))
     HB_FAIL("hb_attn_masked_heads: rows of q, keys and values must start on 16-byte boundaries");
+  if ((r1 != nullptr) != (r2 != nullptr)) HB_FAIL("hb_attn_masked_heads: a distance bias needs both of its vectors");
   HeadsArgs A;
-  A.q = (const __nv_bfloat16*)q; A.ldq = ldq; A.kc = (const __nv_bfloat16*)kc; A.k_page = k_page; A.k_head = k_head; A.k_row = k_row;
+  A.r1 = r1; A.r2 = r2; A.q = (const __nv_bfloat16*)q; A.ldq = ldq; A.kc = (const __nv_bfloat16*)kc; A.k_page = k_page; A.k_head = k_head; A.k_row = k_row;
   A.vc = (const __nv_bfloat16*)vc; A.v_page = v_page; A.v_head = v_head; A.v_row = v_row; A.alias = alias; A.bt = bt;
   A.bt_stride = bt_stride; A.row_req = row_req; A.pos = pos; A.sink = sink; A.gate = gate; A.ld_gate = ld_gate; A.gate_off = gate_off;
   A.gate_mode = gate ? gate_mode : 0; A.out = out; A.ldo = ldo; A.H = H; A.G = G; A.D = D; A.E = E; A.page_size = page_size;

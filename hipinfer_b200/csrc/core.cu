@@ -315,13 +315,14 @@ __global__ void bias_act_kernel(const float* __restrict__ x, long ldx, const TB_
   const size_t m = i / n, c = i - m * n;
   float v = x[m * ldx + c] + (bias ? hb_to_float(bias[c]) : 0.f);
   if (act == 1) v = tanhf(v);
+  else if (act == 2) v = 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
   y[m * ldy + c] = hb_from_float<TO>(v);
 }
 
 HB_EXPORT int hb_bias_act(const float* x, long ldx, const void* bias, int bias_dt, void* y, int y_dt, long ldy, int M,
                           int n, int act, cudaStream_t s) {
   if (M <= 0 || n <= 0) return 0;
-  if (act < 0 || act > 1) HB_FAIL("hb_bias_act: unknown activation %d", act);
+  if (act < 0 || act > 2) HB_FAIL("hb_bias_act: unknown activation %d", act);
   const size_t tot = (size_t)M * n;
   HB_DISPATCH_2(bias_dt, y_dt, "hb_bias_act",
                 (hb_launch(bias_act_kernel<TA, TB>, (unsigned)((tot + 255) / 256), 256, 0, s, x, ldx, (const TA*)bias,
@@ -613,7 +614,8 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
                                                               int pairing, int unit_norm, float eps, TQ* __restrict__ q_out,
                                                               TQ* __restrict__ kc, TQ* __restrict__ vc, int H, int G, int D,
                                                               int E, int page_size, const TW* __restrict__ pre_wq,
-                                                              const TW* __restrict__ pre_wk, float pre_eps) {
+                                                              const TW* __restrict__ pre_wk, float pre_eps, int pre_head,
+                                                              float temp_coef, double temp_every) {
   extern __shared__ float rn_sh[];      // [8 warps][D], then 32 floats for the sums of a row norm
   hb_pdl_launch();
   hb_pdl_wait();
@@ -624,9 +626,12 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
   const size_t page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
   float* buf = rn_sh + warp * D;
   const int n_heads = H + (slot >= 0 ? G : 0);
+  // the query's temperature: a factor that grows with the position, 1 + coef ln(floor((p + 1) / every) + 1)
+  const float tq = temp_every > 0.0 ? fmaf(temp_coef, logf((float)floor((double)(pos[t] + 1) / temp_every) + 1.f), 1.f) : 1.f;
   // a norm over the WHOLE q row and the whole k row (all heads at once), with a weight per column, before the rotation
+  // (pre_head: over each head by itself, with one weight per dimension that the heads share)
   float fq = 1.f, fk = 1.f;
-  if (pre_wq) {
+  if (pre_wq && !pre_head) {
     float* red = rn_sh + 8 * D;
     float sq = 0.f, sk = 0.f;
     for (int i = threadIdx.x; i < H * D; i += 256) sq = fmaf(row[q_off + i], row[q_off + i], sq);
@@ -640,8 +645,13 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
   for (int hh = blockIdx.y * 8 + warp; hh < n_heads; hh += 8 * gridDim.y) {
     const float* src = hh < H ? row + q_off + (size_t)hh * D : row + k_off + (size_t)(hh - H) * D;
     if (pre_wq) {
-      const TW* pw = hh < H ? pre_wq + (size_t)hh * D : pre_wk + (size_t)(hh - H) * D;
-      const float pf = hh < H ? fq : fk;
+      const TW* pw = hh < H ? pre_wq + (pre_head ? 0 : (size_t)hh * D) : pre_wk + (pre_head ? 0 : (size_t)(hh - H) * D);
+      float pf = hh < H ? fq : fk;
+      if (pre_head) {
+        float sh = 0.f;
+        for (int d = lane; d < D; d += 32) sh = fmaf(src[d], src[d], sh);
+        pf = rsqrtf(hb_warp_sum(sh) / (float)D + pre_eps);
+      }
       for (int d = lane; d < D; d += 32) buf[d] = src[d] * pf * hb_to_float(pw[d]);
     } else {
       for (int d = lane; d < D; d += 32) buf[d] = src[d];
@@ -662,6 +672,7 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
       for (int d = lane; d < D; d += 32) ss = fmaf(buf[d], buf[d], ss);
       f = rsqrtf(hb_warp_sum(ss) / (float)D + eps);
     }
+    if (hh < H) f *= tq;
     TQ* dst = hh < H ? q_out + ((size_t)t * H + hh) * D : kc + ((page * G + (hh - H)) * page_size + off) * D;
     for (int d = lane; d < D; d += 32) dst[d] = hb_from_float<TQ>(buf[d] * f);
     __syncwarp();
@@ -676,7 +687,8 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
 HB_EXPORT int hb_rope_norm_store(const float* proj, long ld, int q_off, int k_off, int v_off, const int* pos,
                                  const int* slot_map, const void* table, int rot, int rot_off, int pairing, int unit_norm,
                                  float eps, void* q_out, void* kc, void* vc, int q_dt, int T, int H, int G, int D, int E, int page_size,
-                                 const void* pre_wq, const void* pre_wk, int pre_dt, float pre_eps, cudaStream_t s) {
+                                 const void* pre_wq, const void* pre_wk, int pre_dt, float pre_eps, int pre_head, float temp_coef,
+                                 double temp_every, cudaStream_t s) {
   if (T <= 0) return 0;
   if (rot < 0 || rot_off < 0 || rot_off + rot > D || (rot & 1)) HB_FAIL("hb_rope_norm_store: %d rotated dimensions from %d on of a head of %d", rot, rot_off, D);
   if (slot_map && (!kc || !vc || G <= 0 || E <= 0 || page_size <= 0)) HB_FAIL("hb_rope_norm_store: a slot map without caches or sizes");
@@ -695,7 +707,7 @@ HB_EXPORT int hb_rope_norm_store(const float* proj, long ld, int q_off, int k_of
   HB_DISPATCH_2(q_dt, pre_dt, "hb_rope_norm_store",
                 (hb_launch(rope_norm_store_kernel<TA, TB>, dim3(T, split), 256, smem, s, proj, ld, q_off, k_off, v_off, pos, slot_map,
                            (const float2*)table, rot, rot_off, pairing, unit_norm, eps, (TA*)q_out, (TA*)kc, (TA*)vc, H, G, D, E,
-                           page_size, (const TB*)pre_wq, (const TB*)pre_wk, pre_eps)));
+                           page_size, (const TB*)pre_wq, (const TB*)pre_wk, pre_eps, pre_head, temp_coef, temp_every)));
   HB_CHECK_LAUNCH("hb_rope_norm_store");
   return 0;
 }

@@ -16,7 +16,7 @@
 // drains and returns.
 #include "tc_common.cuh"
 
-enum { EPI_F32 = 0, EPI_BF16 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_ROPE_KV = 4, EPI_GEGLU_BF16 = 5 };
+enum { EPI_F32 = 0, EPI_BF16 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_ROPE_KV = 4, EPI_GEGLU_BF16 = 5, EPI_GELU_BF16 = 6 };   // 6: bf16 after the exact (erf) GELU, no gate
 
 // The gated epilogues: act(gate) * up over 16-interleaved columns, act = silu (3) or the tanh form of GELU (5), which is
 // g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)).
@@ -56,6 +56,12 @@ struct GemmSmem {
   static constexpr int TOTAL_TS = STAGING_OFFSET + 4 * 2 * 4096 + 1024;
 };
 
+#define EPI_IS_BF16(E) ((E) == EPI_BF16 || (E) == EPI_GELU_BF16)
+template <int EPI> __device__ __forceinline__ float hb_bf16_act(float v) {
+  if (EPI == EPI_GELU_BF16) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  return v;
+}
+
 template <int EPI>
 __device__ __forceinline__ void epilogue_store(const float* v, void* C, long ldc, int row, int col0, int M, int N) {
   // v: 32 consecutive columns col0.. of `row`
@@ -76,16 +82,16 @@ __device__ __forceinline__ void epilogue_store(const float* v, void* C, long ldc
     } else {
       for (int j = 0; j < 16 && o0 + j < n_out; j++) out[j] = r[j];
     }
-  } else if (EPI == EPI_BF16) {
+  } else if (EPI_IS_BF16(EPI)) {
     __nv_bfloat16* out = (__nv_bfloat16*)C + (size_t)row * ldc + col0;
     if (col0 + 32 <= N && ((ldc & 7) == 0)) {
       __align__(16) __nv_bfloat16 r[32];
 #pragma unroll
-      for (int j = 0; j < 32; j++) r[j] = __float2bfloat16_rn(v[j]);
+      for (int j = 0; j < 32; j++) r[j] = __float2bfloat16_rn(hb_bf16_act<EPI>(v[j]));
 #pragma unroll
       for (int j = 0; j < 4; j++) *(uint4*)(out + 8 * j) = *(const uint4*)(r + 8 * j);
     } else {
-      for (int j = 0; j < 32 && col0 + j < N; j++) out[j] = __float2bfloat16_rn(v[j]);
+      for (int j = 0; j < 32 && col0 + j < N; j++) out[j] = __float2bfloat16_rn(hb_bf16_act<EPI>(v[j]));
     }
   } else {
     float* out = (float*)C + (size_t)row * ldc + col0;
@@ -145,7 +151,7 @@ __device__ __forceinline__ void rope_head_store(float* x1, float* x2, int head, 
 template <int EPI>
 __device__ __forceinline__ void ts_chunk(const float* v, int c, int n0, int N, int row0, uint8_t* boxes, int lane,
                                          const CUtensorMap* map_c) {
-  constexpr int PER = EPI_IS_GLU(EPI) ? 4 : EPI == EPI_BF16 ? 2 : 1;
+  constexpr int PER = EPI_IS_GLU(EPI) ? 4 : EPI_IS_BF16(EPI) ? 2 : 1;
   uint8_t* box = boxes + ((c / PER) & 1) * 4096;
   if (c % PER == 0) {
     if (lane == 0) hb_tma_store_wait_read<1>();   // the store that last read this box is done with it
@@ -163,12 +169,15 @@ __device__ __forceinline__ void ts_chunk(const float* v, int c, int n0, int N, i
     for (int j = 0; j < 2; j++)
       asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(b + ((((c % PER) * 2 + j) ^ (lane & 7)) << 4)),
                    "r"(r[4 * j]), "r"(r[4 * j + 1]), "r"(r[4 * j + 2]), "r"(r[4 * j + 3]) : "memory");
-  } else if constexpr (EPI == EPI_BF16) {
+  } else if constexpr (EPI_IS_BF16(EPI)) {
 #pragma unroll
-    for (int j = 0; j < 4; j++)
-      asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(b + ((((c % PER) * 4 + j) ^ (lane & 7)) << 4)),
-                   "r"(hb_pack_bf16(v[8 * j], v[8 * j + 1])), "r"(hb_pack_bf16(v[8 * j + 2], v[8 * j + 3])),
-                   "r"(hb_pack_bf16(v[8 * j + 4], v[8 * j + 5])), "r"(hb_pack_bf16(v[8 * j + 6], v[8 * j + 7])) : "memory");
+    for (int j = 0; j < 4; j++) {
+      uint32_t r[4];
+#pragma unroll
+      for (int i = 0; i < 4; i++) r[i] = hb_pack_bf16(hb_bf16_act<EPI>(v[8 * j + 2 * i]), hb_bf16_act<EPI>(v[8 * j + 2 * i + 1]));
+      asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(b + ((((c % PER) * 4 + j) ^ (lane & 7)) << 4)), "r"(r[0]),
+                   "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < 8; j++)
@@ -601,6 +610,7 @@ static int dispatch_epi(int epi, const CUtensorMap& ma, const CUtensorMap& mw, v
     case EPI_ADD_F32: return launch_gemm_tc<BN, STAGES, EPI_ADD_F32>(ma, mw, C, ldc, M, N, K, status, s);
     case EPI_SWIGLU_BF16: return launch_gemm_tc<BN, STAGES, EPI_SWIGLU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
     case EPI_GEGLU_BF16: return launch_gemm_tc<BN, STAGES, EPI_GEGLU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
+    case EPI_GELU_BF16: return launch_gemm_tc<BN, STAGES, EPI_GELU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
   }
   HB_FAIL("hb_gemm_tc: unknown epilogue %d", epi);
 }
@@ -641,6 +651,7 @@ HB_EXPORT int hb_gemm_tc(const void* A, long lda, const void* W, long ldw, void*
       case EPI_ADD_F32: r = launch_gemm_pair<EPI_ADD_F32>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       case EPI_SWIGLU_BF16: r = launch_gemm_pair<EPI_SWIGLU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       case EPI_GEGLU_BF16: r = launch_gemm_pair<EPI_GEGLU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
+      case EPI_GELU_BF16: r = launch_gemm_pair<EPI_GELU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       default: HB_FAIL("hb_gemm_tc: unknown epilogue %d", epi);
     }
     if (r) return r;

@@ -6,6 +6,10 @@
 // A second form (route mode 1, `at_output`): z = Wr h + b; the `top` largest LOGITS choose; the weights are the softmax over
 // the chosen logits alone and multiply the expert's RESULT, which, the down product being linear, is the activation times
 // the weight, silu(g) * u * s, again in 32-bit.
+// A third form (route mode 2): s = sigmoid(z); c = s + correction chooses, where the experts form equal groups of neighbours
+// only among the groups that rank best by the sum of their two largest c; the weights are the chosen s (without the
+// correction) divided by their sum, times a constant. Beside the router's rows one more row may give a number per token,
+// sigmoid(w . h), that a shared expert's result is multiplied by.
 //
 // moe_route_kernel          scores and the chosen experts of every row: expert [T][top], weight [T][top]
 // Few rows (decoding): no sorting, nothing on the host
@@ -29,24 +33,55 @@ constexpr int MR_THREADS = 128;
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restrict__ xn, long ldx, const TW* __restrict__ router,
                                                                const TW* __restrict__ bias, int* __restrict__ expert,
-                                                               float* __restrict__ weight, int W, int E, int top, int mode) {
-  extern __shared__ float mr_sm[];     // [W] the row, [E] the scores
+                                                               float* __restrict__ weight, int W, int E, int top, int mode,
+                                                               const TW* __restrict__ correction, int groups, int keep, float scale,
+                                                               const TW* __restrict__ shared_gate, float* __restrict__ shared_weight) {
+  extern __shared__ float mr_sm[];     // [W] the row, [E] the scores, (mode 2) [E] the scores without the correction
   float* row = mr_sm;
   float* sc = mr_sm + W;
+  float* plain = sc + E;
   hb_pdl_launch();
   hb_pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   for (int i = threadIdx.x; i < W; i += MR_THREADS) row[i] = hb_to_float(xn[(size_t)t * ldx + i]);
   __syncthreads();
-  for (int e = warp; e < E; e += MR_THREADS / 32) {
-    const TW* wr = router + (size_t)e * W;
+  for (int e = warp; e < E + (shared_gate ? 1 : 0); e += MR_THREADS / 32) {
+    const TW* wr = e < E ? router + (size_t)e * W : shared_gate;
     float acc = 0.f;
     for (int i = lane; i < W; i += 32) acc = fmaf(row[i], hb_to_float(wr[i]), acc);
     acc = hb_warp_sum(acc);
+    if (e == E) {
+      if (lane == 0) shared_weight[t] = 1.f / (1.f + expf(-acc));
+      continue;
+    }
     if (bias) acc += hb_to_float(bias[e]);
-    if (lane == 0) sc[e] = mode == 0 ? 1.f / (1.f + expf(-acc)) : acc;
+    if (lane == 0) {
+      const float v = mode == 1 ? acc : 1.f / (1.f + expf(-acc));
+      sc[e] = mode == 2 ? v + hb_to_float(correction[e]) : v;
+      if (mode == 2) plain[e] = v;
+    }
   }
   __syncthreads();
+  if (mode == 2 && groups > 1 && threadIdx.x == 0) {
+    // the groups that do not stay are marked as taken, the worst group first (ties: the higher index goes first)
+    const int span = E / groups;
+    for (int gone = 0; gone < groups - keep; gone++) {
+      int worst = -1;
+      float ws = 0.f;
+      for (int q = 0; q < groups; q++) {
+        if (sc[q * span] != sc[q * span]) continue;
+        float a = -INFINITY, b = -INFINITY;            // the two largest
+        for (int e = q * span; e < (q + 1) * span; e++) {
+          const float v = sc[e];
+          if (v > a) { b = a; a = v; } else if (v > b) b = v;
+        }
+        const float v = span > 1 ? a + b : a;
+        if (worst < 0 || v <= ws) { worst = q; ws = v; }
+      }
+      if (worst < 0) break;
+      for (int e = worst * span; e < (worst + 1) * span; e++) sc[e] = __int_as_float(0x7fc00000);
+    }
+  }
   if (threadIdx.x == 0) {
     float first = 0.f, den = 0.f;
     for (int k = 0; k < top; k++) {
@@ -63,7 +98,10 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
       if (best < 0) best = 0;          // every score NaN (bad weights or input): stay inside the tables
       expert[(size_t)t * top + k] = best;
       if (mode == 0) weight[(size_t)t * top + k] = bs;
-      else {
+      else if (mode == 2) {
+        weight[(size_t)t * top + k] = plain[best];
+        den += plain[best];
+      } else {
         // softmax over the chosen logits alone: the first chosen one is the largest
         if (k == 0) first = bs;
         const float ex = expf(bs - first);
@@ -72,24 +110,33 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
       }
       sc[best] = __int_as_float(0x7fc00000);
     }
-    if (mode != 0)
+    if (mode == 1)
       for (int k = 0; k < top; k++) weight[(size_t)t * top + k] /= den;
+    if (mode == 2)
+      for (int k = 0; k < top; k++) weight[(size_t)t * top + k] = weight[(size_t)t * top + k] / (den + 1e-20f) * scale;
   }
 }
 
 // mode 0: the scores are sigmoid(z) and the chosen scores are the weights; mode 1: the largest logits z choose and the
-// weights are the softmax over the chosen logits alone. bias (the router's element type, or null) is added to z.
+// weights are the softmax over the chosen logits alone; mode 2: sigmoid(z) + correction [E] chooses, within the `keep` best of
+// `groups` groups, and the weights are the chosen sigmoid(z) over their sum, times scale. bias (the router's element type, or
+// null) is added to z. shared_gate [W] (or null): shared_weight[t] = sigmoid(shared_gate . row).
 HB_EXPORT int hb_moe_route(const void* xn, int x_dt, long ldx, const void* router, const void* bias, int w_dt, int* expert,
-                           float* weight, int T, int W, int E, int top, int mode, cudaStream_t s) {
+                           float* weight, int T, int W, int E, int top, int mode, const void* correction, int groups, int keep,
+                           float scale, const void* shared_gate, float* shared_weight, cudaStream_t s) {
   if (T <= 0) return 0;
+  if (mode == 2 && !correction) HB_FAIL("hb_moe_route: the third form needs its corrections");
+  if (groups > 1 && (E % groups || keep < 1 || keep > groups || (long)keep * (E / groups) < top))
+    HB_FAIL("hb_moe_route: %d experts in %d groups of which %d stay, %d chosen", E, groups, keep, top);
+  if (shared_gate && !shared_weight) HB_FAIL("hb_moe_route: a shared expert's gate needs a place for its result");
   if (top < 1 || top > E) HB_FAIL("hb_moe_route: top %d of %d experts", top, E);
-  const size_t smem = (size_t)(W + E) * sizeof(float);
+  const size_t smem = (size_t)(W + 2 * E) * sizeof(float);
   if (smem > 200 * 1024) HB_FAIL("hb_moe_route: a row of %d with %d experts does not fit shared memory", W, E);
   HB_DISPATCH_2(x_dt, w_dt, "hb_moe_route", do {
     auto kern = moe_route_kernel<TA, TB>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     hb_launch(kern, dim3(T), dim3(MR_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert, weight,
-              W, E, top, mode);
+              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_route");
   return 0;

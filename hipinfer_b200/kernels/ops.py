@@ -36,7 +36,7 @@ _SIGS = {
         "hb_layernorm": [_p, _p, _p, _i, _p, _i, _p, _i, _i, _f, _p],
         "hb_gated_act": [_p, _i, _l, _p, _i, _l, _i, _i, _i, _i, _p],
         "hb_rope_norm_store": [_p, _l, _i, _i, _i, _p, _p, _p, _i, _i, _i, _i, _f, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _p, _i,
-                               _f, _p],
+                               _f, _i, _f, C.c_double, _p],
         "hb_polynorm": [_p, _l, _p, _i, _l, _i, _i, _f, _f, _f, _f, _f, _p],
         "hb_scale_add": [_p, _p, _l, _p, _i, _i, _i, _p],
         "hb_bias_act": [_p, _l, _p, _i, _p, _i, _l, _i, _i, _i, _p],
@@ -45,16 +45,16 @@ _SIGS = {
     },
     "seqmix": {
         "hb_attn_masked": [_p, _i, _l, _p, _l, _p, _l, _i, _p, _i, _p, _p, _p, _p, _l, _i, _i, _p, _i, _l, _i, _i, _i, _i, _i,
-                           _i, _i, _i, _i, _i, _f, _p, _i, _p, _l, _p, _i, _p],
+                           _i, _i, _i, _i, _i, _f, _p, _i, _p, _l, _p, _i, _p, _p, _p],
         "hb_latent_prepare": [_p, _l, _i, _i, _i, _p, _p, _i, _p, _p, _p, _i, _f, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p],
         "hb_heads_linear": [_p, _l, _l, _p, _i, _p, _i, _l, _l, _i, _i, _i, _i, _p, _l, _i, _i, _i, _p, _p, _p, _p, _i, _i, _i, _p],
         "hb_gather_rows": [_p, _i, _p, _p, _i, _i, _i, _p],
         "hb_attn_masked_flash_supported": [_i, _i],
         "hb_attn_masked_heads_supported": [_i, _i, _i, _i, _i],
         "hb_attn_masked_heads": [_p, _l, _p, _l, _l, _l, _p, _l, _l, _l, _i, _p, _i, _p, _p, _p, _p, _l, _i, _i, _p, _i, _l, _i, _i,
-                                 _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _i, _p, _l, _i, _p],
+                                 _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _i, _p, _l, _i, _p, _p, _p],
         "hb_attn_masked_flash": [_p, _l, _p, _l, _l, _l, _p, _l, _l, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _p, _p, _l, _i, _i, _p,
-                                 _i, _l, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p],
+                                 _i, _l, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _p],
         "hb_gla": [_p, _l, _i, _i, _i, _i, _p, _l, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _f, _p],
     },
     "hybrid": {
@@ -71,7 +71,7 @@ _SIGS = {
                               _p],
         "hb_split_rounded": [_p, _l, _p, _p, _i, _i, _p],
         "hb_residual_norm": [_p, _p, _p, _p, _p, _p, _i, _f, _f, _f, _p, _f, _p, _i, _i, _i, _p],
-        "hb_moe_route": [_p, _i, _l, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _p],
+        "hb_moe_route": [_p, _i, _l, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _f, _p, _p, _p],
         "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p],
         "hb_moe_down_rows": [_p, _i, _p, _i, _p, _p, _l, _i, _i, _i, _i, _p],
         "hb_moe_sort": [_p, _p, _p, _p, _i, _i, _p],
@@ -79,6 +79,13 @@ _SIGS = {
         "hb_moe_gather": [_p, _i, _l, _p, _p, _i, _i, _i, _p],
         "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p],
         "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p],
+    },
+    "memory": {
+        "hb_ms_walk": [_p, _l, _p, _l, _p, _l, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _i, _p, _p, _p, _p],
+        "hb_ms_exp_gates": [_p, _p, _l, _p, _p, _i, _f, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _p],
+        "hb_ms_delta_prepare": [_p, _l, _i, _i, _p, _p, _l, _p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _p],
+        "hb_ms_finish": [_p, _p, _p, _f, _p, _i, _i, _p, _l, _i, _p, _i, _l, _i, _i, _i, _f, _p],
+        "hb_output_norm": [_p, _p, _p, _f, _f, _p, _p, _i, _f, _i, _p, _p, _i, _p, _p, _p, _l, _p, _i, _i, _i, _p],
     },
     "mixers": {
         "hb_delta_rule": [_p, _l, _i, _i, _i, _i, _i, _p, _l, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _f, _f, _f,
@@ -227,14 +234,14 @@ def scale_add(x: torch.Tensor, y: torch.Tensor, scale: torch.Tensor) -> torch.Te
 
 
 def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, act: str = "none") -> torch.Tensor:
-    """out = act(x + bias) for float32 rows x (a view of some columns is fine); act "none" or "tanh"."""
+    """out = act(x + bias) for float32 rows x (a view of some columns is fine); act "none", "tanh" or "gelu" (the exact form, z Phi(z))."""
     _need_cuda(x, bias, out)
     _rows_contiguous(x, "bias_act in")
     _rows_contiguous(out, "bias_act out")
     assert x.dtype == torch.float32 and x.shape == out.shape
     M, n = x.shape
     _call("core", "hb_bias_act", x.data_ptr(), x.stride(0), _ptr(bias), _dt(bias) if bias is not None else 0,
-          out.data_ptr(), _dt(out), out.stride(0), M, n, {"none": 0, "tanh": 1}[act], _stream())
+          out.data_ptr(), _dt(out), out.stride(0), M, n, {"none": 0, "tanh": 1, "gelu": 2}[act], _stream())
     return out
 
 
@@ -770,6 +777,18 @@ def linear_gated(a: torch.Tensor, w_gate_up: "Weight", act_out: torch.Tensor, gr
     return a.is_cuda and fast.linear_gated(a, w_gate_up, act_out, group, act)
 
 
+def linear_act(a: torch.Tensor, w: "Weight", out: torch.Tensor, act: str) -> torch.Tensor:
+    """out = act(a @ w.T), act "gelu" (the exact form): the activation in the product's epilogue where one takes these
+    sizes, else the product's 32-bit rows through `bias_act`."""
+    from . import fast
+
+    if a.is_cuda and fast.linear_act(a, w, out, act):
+        return out
+    z = torch.empty(a.shape[0], w.shape[0], dtype=torch.float32, device=a.device)
+    linear(a, w, z)
+    return bias_act(z, None, out, act)
+
+
 _rope_tables = {}
 
 
@@ -823,13 +842,15 @@ PAIRINGS = {"half": 0, "interleaved": 1}
 def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_map: Optional[torch.Tensor],
                     table: torch.Tensor, rot: int, pairing: str, unit_norm: bool, eps: float, q_out: torch.Tensor,
                     k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], n_heads: int, n_kv_heads: int,
-                    dim: int, vdim: int, page_size: int, rot_off: int = 0, row_norm=None, row_norm_eps: float = 0.0) -> torch.Tensor:
+                    dim: int, vdim: int, page_size: int, rot_off: int = 0, row_norm=None, row_norm_eps: float = 0.0,
+                    head_norm=None, q_temp=None) -> torch.Tensor:
     """From a float32 projection result whose rows hold q, k, v at the column `offsets` (q, k, v): q and k rotated on
     the `rot` dimensions from `rot_off` on (pairing "half": (i, i + rot/2); "interleaved": (2i, 2i + 1)) and, with unit_norm,
     divided by their root mean square over `dim`; q to q_out [T, n_heads * dim], k and v (vdim wide, raw) to their page
     slots. slot_map None: q alone. row_norm (wq [n_heads * dim], wk [n_kv_heads * dim]): before the rotation the whole
     q row and the whole k row are divided by their root mean square (row_norm_eps inside the root) and multiplied by the
-    weights, column by column."""
+    weights, column by column. head_norm (wq [dim], wk [dim]) instead: each head by itself, with weights the heads share.
+    q_temp (coef, every): q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     _need_cuda(proj, positions, slot_map, table, q_out, k_cache, v_cache)
     _rows_contiguous(proj, "rope_norm_store in")
     T = proj.shape[0]
@@ -839,15 +860,19 @@ def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_m
         assert k_cache.dtype == v_cache.dtype == q_out.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
         assert k_cache.shape[-1] == dim and v_cache.shape[-1] == vdim
     q_off, k_off, v_off = (int(o) for o in offsets)
-    wq_pre, wk_pre = row_norm if row_norm is not None else (None, None)
+    assert row_norm is None or head_norm is None
+    per_head = head_norm is not None
+    wq_pre, wk_pre = row_norm if row_norm is not None else head_norm if per_head else (None, None)
     if wq_pre is not None:
         _need_cuda(wq_pre, wk_pre)
-        assert wq_pre.dtype == wk_pre.dtype and wq_pre.numel() == n_heads * dim and wk_pre.numel() == n_kv_heads * dim
+        assert wq_pre.dtype == wk_pre.dtype and wq_pre.numel() == (1 if per_head else n_heads) * dim
+        assert wk_pre.numel() == (1 if per_head else n_kv_heads) * dim
+    coef, every = q_temp if q_temp is not None else (0.0, 0.0)
     _call("core", "hb_rope_norm_store", proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, positions.data_ptr(),
           _ptr(slot_map), table.data_ptr(), int(rot), int(rot_off), PAIRINGS[pairing], 1 if unit_norm else 0, float(eps), q_out.data_ptr(),
           _ptr(k_cache) if slot_map is not None else None, _ptr(v_cache) if slot_map is not None else None, _dt(q_out), T,
           n_heads, n_kv_heads, dim, vdim, page_size, _ptr(wq_pre), _ptr(wk_pre), _dt(wq_pre) if wq_pre is not None else 0,
-          float(row_norm_eps), _stream())
+          float(row_norm_eps), 1 if per_head else 0, float(coef), float(every), _stream())
     return q_out
 
 
@@ -859,7 +884,7 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
                      page_size: int, scale: float, mask: str = "causal", window: int = 0, keep_first: int = 0, chunk: int = 0,
                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
                      gate_per_head: bool = False, force_rows: bool = False, row_limit: int = 0,
-                     force_plain: bool = False) -> torch.Tensor:
+                     force_plain: bool = False, distance=None) -> torch.Tensor:
     """Attention of the step's rows over their requests' pages (csrc/attention_masked.cu; requests that bring many rows:
     csrc/attention_masked_flash.cu). With row_limit, rows of requests that bring that many rows or more are left alone (the
     caller has another path for them). Keys `dim` and values `vdim`
@@ -867,7 +892,12 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
     the values are then its first `vdim` columns). mask "causal", "window" (the last `window` keys and the first
     `keep_first`) or "chunk" (the keys of the row's own chunk of `chunk` positions). sink: float32 [n_heads], joins the
     softmax's denominator as exp(sink). gate: float32 [T, *], sigmoid(gate[:, gate_offset + ...]) multiplies the result,
-    one number per element or, with gate_per_head, one per head. out may be float32 beside bfloat16 q."""
+    one number per element or, with gate_per_head, one per head. out may be float32 beside bfloat16 q. distance (r1, r2),
+    float32 [n_heads] each: r1 ln(1 + r2 (i - j)) is taken off the score of query i and key j."""
+    r1, r2 = distance if distance is not None else (None, None)
+    _need_cuda(r1, r2)
+    for r in (r1, r2):
+        assert r is None or (r.dtype == torch.float32 and r.numel() == n_heads and r.is_contiguous())
     _need_cuda(q, k_cache, v_cache, out, gate, sink)
     T = q.shape[0]
     bt = batch.block_tables[group]
@@ -899,7 +929,8 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
               batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_ctx_len.data_ptr(), 0, batch.n_requests,
               batch.max_q_len, MASKED_FLASH_MIN_ROWS, _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
               int(gate_offset), (2 if gate_per_head else 1) if gate is not None else 0, out.data_ptr(), _dt(out), out.stride(0),
-              n_heads, n_kv_heads, dim, vdim, page_size, m, int(window), int(keep_first), int(chunk), float(scale), _stream())
+              n_heads, n_kv_heads, dim, vdim, page_size, m, int(window), int(keep_first), int(chunk), float(scale), _ptr(r1), _ptr(r2),
+              _stream())
         if min(batch.h_q_len) >= MASKED_FLASH_MIN_ROWS:
             return out
     limit = int(row_limit) or (MASKED_FLASH_MIN_ROWS if flash else 0)
@@ -918,7 +949,7 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
               gate.stride(0) if gate is not None else 0, int(gate_offset), (2 if gate_per_head else 1) if gate is not None else 0,
               out.data_ptr(), _dt(out), out.stride(0), T, n_heads, n_kv_heads, dim, vdim, page_size, m, int(window),
               int(keep_first), int(chunk), float(scale), batch.req_q_len.data_ptr() if limit else None, limit, _ptr(ws), n_ws,
-              max_pos, _stream())
+              max_pos, _ptr(r1), _ptr(r2), _stream())
         return out
     n_ws = lib.hb_attn_masked_workspace(T, n_heads, n_kv_heads, dim, vdim, m, int(window), int(keep_first), int(chunk), max_pos)
     ws = arrived = None
@@ -932,7 +963,8 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
           batch.positions.data_ptr(), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate_offset),
           (2 if gate_per_head else 1) if gate is not None else 0, out.data_ptr(), _dt(out), out.stride(0), T, n_heads,
           n_kv_heads, dim, vdim, page_size, m, int(window), int(keep_first), int(chunk), float(scale),
-          batch.req_q_len.data_ptr() if limit else None, limit, _ptr(ws), n_ws, _ptr(arrived), max_pos, _stream())
+          batch.req_q_len.data_ptr() if limit else None, limit, _ptr(ws), n_ws, _ptr(arrived), max_pos, _ptr(r1),
+          _ptr(r2), _stream())
     return out
 
 
@@ -1032,7 +1064,7 @@ def attention_flash_tokens(q, keys, values, batch, request: int, out, n_heads: i
           batch.req_q_len.data_ptr(), batch.req_ctx_len.data_ptr(), int(request), 1, int(batch.h_q_len[request]), 1, _ptr(sink),
           _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate_offset), (2 if gate_per_head else 1) if gate is not None else 0,
           out.data_ptr(), _dt(out), out.stride(0), n_heads, n_kv_heads, dim, vdim, 1, 1 if window else 0, int(window), 0, 0,
-          float(scale), _stream())
+          float(scale), None, None, _stream())
     return out
 
 
@@ -1283,14 +1315,22 @@ def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, pair: Optio
     return x
 
 
-MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1}
+MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "sigmoid_normed": 2}
 
 
-def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[torch.Tensor] = None, score: str = "sigmoid"):
+def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[torch.Tensor] = None, score: str = "sigmoid",
+              correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
+              shared_gate: Optional[torch.Tensor] = None, shared_weight: Optional[torch.Tensor] = None):
     """(expert int32 [T, top], weight float32 [T, top]): the `top` experts with the largest z = router @ row (+ bias), 32-bit
     sums; the largest first, ties to the lower index. score "sigmoid": the weights are sigmoid(z) of the chosen ones;
-    "softmax_chosen": the softmax over the chosen logits alone."""
-    _need_cuda(xn, router, bias)
+    "softmax_chosen": the softmax over the chosen logits alone. "sigmoid_normed": sigmoid(z) + correction chooses, with
+    groups > 1 only among the experts of the `keep` groups (of neighbours) whose two largest sums are largest; the weights are
+    the chosen sigmoid(z), without the correction, over their sum (+ 1e-20), times scale. shared_gate [1, W] or [W]: also
+    shared_weight[t] (float32 [T]) = sigmoid(shared_gate . row)."""
+    _need_cuda(xn, router, bias, correction, shared_gate, shared_weight)
+    assert correction is None or (correction.dtype == router.dtype and correction.numel() == router.shape[0] and correction.is_contiguous())
+    assert shared_gate is None or (shared_gate.dtype == router.dtype and shared_gate.numel() == router.shape[1]
+                                   and shared_weight.dtype == torch.float32 and shared_weight.numel() == xn.shape[0])
     assert bias is None or (bias.dtype == router.dtype and bias.numel() == router.shape[0] and bias.is_contiguous())
     _rows_contiguous(xn, "moe_route in")
     T, (E, W) = xn.shape[0], router.shape
@@ -1298,7 +1338,8 @@ def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[t
     expert = torch.empty(T, top, dtype=torch.int32, device=xn.device)
     weight = torch.empty(T, top, dtype=torch.float32, device=xn.device)
     _call("hybrid", "hb_moe_route", xn.data_ptr(), _dt(xn), xn.stride(0), router.data_ptr(), _ptr(bias), _dt(router),
-          expert.data_ptr(), weight.data_ptr(), T, W, E, int(top), MOE_SCORES[score], _stream())
+          expert.data_ptr(), weight.data_ptr(), T, W, E, int(top), MOE_SCORES[score], _ptr(correction), int(groups), int(keep), float(scale),
+          _ptr(shared_gate), _ptr(shared_weight), _stream())
     return expert, weight
 
 
@@ -1376,3 +1417,138 @@ def moe_combine(ys: torch.Tensor, pos: torch.Tensor, y: torch.Tensor, top: int) 
     assert ys.dtype == y.dtype == torch.float32 and ys.is_contiguous() and ys.shape == (T * top, W)
     _call("hybrid", "hb_moe_combine", ys.data_ptr(), pos.data_ptr(), y.data_ptr(), y.stride(0), T, W, int(top), _stream())
     return y
+
+
+# ------------------------------------------------------------------------------------------
+# The `memory` library: recurrences with one state matrix per head, and the residual row after a sublayer whose result is
+# normed (csrc/matrix_state.cu, depth_average.cu)
+# ------------------------------------------------------------------------------------------
+MS_PIECE_TOKENS = 64    # tokens a piece of the linear recurrence (ms_walk); 0: always one walk a request
+
+
+def ms_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, state: torch.Tensor, batch,
+            y: torch.Tensor, q_scale: float = 1.0, kq: Optional[torch.Tensor] = None, nstate: Optional[torch.Tensor] = None,
+            nq: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The walk of a recurrence with one state matrix per head over the step's rows, request by request, from and into each
+    request's state slot. q, k float32 [T, groups * N], v float32 [T, heads * P] (views of wider rows are fine); a, b float32
+    [T, heads]; state float32 [slots, heads, N, P]; y float32 [T, heads * P].
+
+    Without kq: S <- a S + b k v^T, y = S^T q * q_scale and, with nstate [slots, heads, N], n <- a n + b k,
+    nq [T, heads] = n . q * q_scale. With kq float32 [T, groups] (k . q of the rows): the delta rule,
+    S <- a S; u = b (v - S^T k); S <- S + k u^T; y = S^T q * q_scale.
+
+    A step of the first form whose longest portion has at least three times MS_PIECE_TOKENS rows runs in pieces of that
+    many tokens; the results differ from the walk in one go by rounding only."""
+    _need_cuda(q, k, v, a, b, state, y, kq, nstate, nq)
+    for t, what in ((q, "q"), (k, "k"), (v, "v")):
+        _rows_contiguous(t, "ms_walk " + what)
+    T, H = a.shape
+    slots, Hs, N, P = state.shape
+    G = q.shape[1] // N
+    assert Hs == H and q.shape == k.shape == (T, G * N) and v.shape == (T, H * P) and y.shape == (T, H * P)
+    assert all(t.dtype == torch.float32 for t in (q, k, v, a, b, state, y)) and all(t.is_contiguous() for t in (a, b, state, y))
+    assert b.shape == (T, H) and (kq is None or (kq.shape == (T, G) and kq.is_contiguous() and kq.dtype == torch.float32))
+    if nstate is not None:
+        assert nstate.shape == (slots, H, N) and nstate.is_contiguous() and nq.shape == (T, H) and nq.is_contiguous()
+    L, pieces, ps, pn, pd = int(MS_PIECE_TOKENS), 0, None, None, None
+    if kq is None and L > 0 and batch.max_q_len >= 3 * L:
+        pieces = -(-batch.max_q_len // L)
+        room = T // L + batch.n_requests               # every request ends with at most one short piece
+        ps = torch.empty(room, H, N, P, dtype=torch.float32, device=q.device)
+        pn = torch.empty(room, H, N, dtype=torch.float32, device=q.device) if nstate is not None else None
+        pd = torch.empty(room, H, dtype=torch.float32, device=q.device)
+    _call("memory", "hb_ms_walk", q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), a.data_ptr(),
+          b.data_ptr(), _ptr(kq), state.data_ptr(), _ptr(nstate), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(),
+          batch.req_state_slot.data_ptr(), y.data_ptr(), _ptr(nq), batch.n_requests, H, G, N, P, float(q_scale),
+          0 if kq is None else 1, L, pieces, _ptr(ps), _ptr(pn), _ptr(pd), _stream())
+    return y
+
+
+def ms_exp_gates(zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float, m_state: torch.Tensor, batch):
+    """Exponential gates with a running maximum: from zi, zf float32 [T, heads] (views of the same wider rows) and biases
+    [heads], li = cap tanh((zi + bi) / cap) and lf = -softplus(-cap tanh((zf + bf) / cap)), m_t = max(lf + m_(t-1), li) along
+    each request from and into m_state float32 [slots, heads]. Returns float32 [T, heads] each:
+    a = exp(lf + m_(t-1) - m_t), b = exp(li - m_t), e = exp(-m_t)."""
+    _need_cuda(zi, zf, bi, bf, m_state)
+    T, H = zi.shape
+    assert zi.dtype == zf.dtype == m_state.dtype == torch.float32 and zi.stride() == zf.stride() and zi.stride(1) == 1
+    assert bi.dtype == bf.dtype and bi.numel() == bf.numel() == H and m_state.is_contiguous() and m_state.shape[1:] == (H,)
+    a, b, e = (torch.empty(T, H, dtype=torch.float32, device=zi.device) for _ in range(3))
+    _call("memory", "hb_ms_exp_gates", zi.data_ptr(), zf.data_ptr(), zi.stride(0), bi.data_ptr(), bf.data_ptr(), _dt(bi), float(cap),
+          m_state.data_ptr(), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_state_slot.data_ptr(), a.data_ptr(),
+          b.data_ptr(), e.data_ptr(), batch.n_requests, batch.max_q_len, H, _stream())
+    return a, b, e
+
+
+def ms_delta_prepare(qkv: torch.Tensor, offsets, za: torch.Tensor, zb: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                     groups: int, dim: int, q_scale: float, unit_eps: float):
+    """Rows qkv float32 [T, *] with q and k [groups * dim] at the column `offsets` (q, k): every head's q and k become
+    x / sqrt(sum x^2 + unit_eps), q also times q_scale, in place. Returns (a, b, kq): a = exp(-exp(a_log) softplus(za +
+    dt_bias)) and b = sigmoid(zb), float32 [T, heads], and kq = k . q, float32 [T, groups]. za, zb: views of the same rows."""
+    _need_cuda(qkv, za, zb, a_log, dt_bias)
+    _rows_contiguous(qkv, "ms_delta_prepare qkv")
+    T, H = za.shape
+    assert qkv.dtype == za.dtype == zb.dtype == torch.float32 and za.stride() == zb.stride() and za.stride(1) == 1
+    assert a_log.dtype == dt_bias.dtype and a_log.numel() == dt_bias.numel() == H
+    a, b = (torch.empty(T, H, dtype=torch.float32, device=za.device) for _ in range(2))
+    kq = torch.empty(T, groups, dtype=torch.float32, device=za.device)
+    _call("memory", "hb_ms_delta_prepare", qkv.data_ptr(), qkv.stride(0), int(offsets[0]), int(offsets[1]), za.data_ptr(), zb.data_ptr(),
+          za.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), _dt(a_log), kq.data_ptr(), a.data_ptr(), b.data_ptr(), T, H, int(groups),
+          int(dim), float(q_scale), float(unit_eps), _stream())
+    return a, b, kq
+
+
+GATE_KINDS = {"sigmoid": 0, "silu": 1}
+
+
+def ms_finish(y: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, gate_kind: str, out: torch.Tensor, heads: int, eps: float,
+              nq: Optional[torch.Tensor] = None, floor: Optional[torch.Tensor] = None, den_eps: float = 0.0) -> torch.Tensor:
+    """out = y (/ (max(|nq|, floor) + den_eps) per token and head) with each head divided by its root mean square, times
+    weight ([P]: shared by the heads; [heads * P]: per channel), times act(gate) ("sigmoid" or "silu"); y float32
+    [T, heads * P], gate float32 [T, heads * P] (a view of wider rows is fine), out rounded once."""
+    _need_cuda(y, weight, gate, out, nq, floor)
+    _rows_contiguous(gate, "ms_finish gate")
+    _rows_contiguous(out, "ms_finish out")
+    T, HP = y.shape
+    P = HP // heads
+    assert y.dtype == gate.dtype == torch.float32 and y.is_contiguous() and gate.shape == out.shape == (T, HP)
+    assert weight.numel() in (P, HP) and weight.is_contiguous()
+    assert nq is None or (nq.shape == floor.shape == (T, heads) and nq.is_contiguous() and floor.is_contiguous())
+    _call("memory", "hb_ms_finish", y.data_ptr(), _ptr(nq), _ptr(floor), float(den_eps), weight.data_ptr(), _dt(weight),
+          1 if weight.numel() == P else 0, gate.data_ptr(), gate.stride(0), GATE_KINDS[gate_kind], out.data_ptr(), _dt(out), out.stride(0),
+          T, heads, P, float(eps), _stream())
+    return out
+
+
+class ScaledPair:
+    """Two side-by-side results that have yet to be joined: ca a + cb b, a and b float32 [T, W]."""
+    __slots__ = ("a", "b", "ca", "cb")
+
+    def __init__(self, a, b, ca, cb):
+        self.a, self.b, self.ca, self.cb = a, b, float(ca), float(cb)
+
+
+def output_norm(x: torch.Tensor, y, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                rounded: Optional[torch.Tensor] = None, keep_in: Optional[torch.Tensor] = None, keep: Optional[torch.Tensor] = None,
+                states: Optional[torch.Tensor] = None, coef: Optional[torch.Tensor] = None, center: bool = True) -> torch.Tensor:
+    """The residual rows x float32 [T, W] after a sublayer with result y (float32 [T, W], or a ScaledPair), in place and in
+    one pass: x' = x + layer norm of y (weight, bias or None; center False: the RMS norm). keep_in / keep (float32 [T, W]): copies of x as it came and of
+    x'. states float32 [n, T, W] with coef float32 [n + 1]: x <- sum_j coef[j] states[j] + coef[n] x' instead of x' (where
+    keep_in is given states[0] is x as it came). rounded: receives a copy of the new x in its element type."""
+    a, b, ca, cb = (y.a, y.b, y.ca, y.cb) if isinstance(y, ScaledPair) else (y, None, 1.0, 0.0)
+    _need_cuda(x, a, b, weight, bias, rounded, keep_in, keep, states, coef)
+    T, W = x.shape
+    for t in (x, a, b, keep_in, keep):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, W))
+    assert weight.numel() == W and weight.is_contiguous()
+    assert bias is None or (bias.dtype == weight.dtype and bias.numel() == W and bias.is_contiguous())
+    assert rounded is None or (rounded.is_contiguous() and rounded.shape == (T, W))
+    n = 0
+    if states is not None:
+        n = states.shape[0]
+        assert states.dtype == coef.dtype == torch.float32 and states.shape[1:] == (T, W) and states[0].is_contiguous()
+        assert coef.is_contiguous() and coef.numel() == n + 1
+    _call("memory", "hb_output_norm", x.data_ptr(), a.data_ptr(), _ptr(b), ca, cb, weight.data_ptr(), _ptr(bias), _dt(weight), float(eps),
+          1 if center else 0, x.data_ptr(), _ptr(rounded), _dt(rounded) if rounded is not None else 0, _ptr(keep_in), _ptr(keep), _ptr(states),
+          states.stride(0) if states is not None else 0, _ptr(coef), n, T, W, _stream())
+    return x

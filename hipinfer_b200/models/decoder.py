@@ -26,6 +26,19 @@ class StepCachePlan:
     write: bool  # False: the step reads the cache another step writes
 
 
+class DepthHistory:
+    """The states a step keeps along its depth for blocks that average over them: the embedding rows and every layer's
+    result, float32 [states, rows, width]. A block takes the next plane and fills it on its way over the row."""
+
+    def __init__(self, n_states, x):
+        self.states = torch.empty((n_states,) + tuple(x.shape), dtype=torch.float32, device=x.device)
+        self.count = 0
+
+    def next(self) -> torch.Tensor:
+        self.count += 1
+        return self.states[self.count - 1]
+
+
 class DecoderModel:
     def __init__(self, spec: ModelSpec, ctx: BuildContext):
         spec.validate()
@@ -103,6 +116,8 @@ class DecoderModel:
         # it), or that next norm already prepared by the layer's last product (kernels.fast.NormFeed); else None
         carry = None
         order = self.spec.order
+        keeps = any(getattr(layer, "takes_history", False) for layer in self.layers)
+        history = DepthHistory(len(order) + 1, x) if keeps else None
         for i, st in enumerate(order):
             layer = self.layers[st.layer]
             cache, state = storage.layer_cache(self.cache_plan[i]), storage.layer_state(i)
@@ -115,9 +130,19 @@ class DecoderModel:
                 kw["pending"] = carry
             if getattr(layer, "takes_next_norm", False) and i + 1 < len(order):
                 kw["next_norm"] = getattr(self.layers[order[i + 1].layer], "mixer_norm", None)
+            if history is not None:
+                if getattr(layer, "takes_history", False):
+                    kw["history"] = history
+                elif history.count == 0:
+                    history.next().copy_(x)
             batch.dump_step = i
             left = layer.forward(x, batch, cache, state, **kw)
             carry = left if left is not None and not isinstance(left, torch.Tensor) else None
+            if history is not None and "history" not in kw:       # a block without an average: its result is a state all the same
+                if isinstance(carry, ops.Pending):
+                    carry.finish()
+                    carry = None
+                history.next().copy_(x)
             if planes.dumping(batch):          # a dumped step leaves nothing pending: x is whole where a plane is taken
                 if isinstance(carry, ops.Pending):
                     carry.finish()

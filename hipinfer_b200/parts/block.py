@@ -12,7 +12,7 @@ import torch
 from ..kernels import ops
 from ..weights import ParamSpec
 from . import planes
-from .norm import RMSNorm
+from .norm import LayerNorm, RMSNorm
 from .registry import Part, build_part, register_part, to_compute
 
 
@@ -390,7 +390,7 @@ class PostNormBlock(Part):
         if isinstance(pending, ops.Pending):
             pending.finish()
         h = self._rows(x, pending)
-        if hasattr(self.mixer, "forward_pair"):
+        if getattr(self.mixer, "join", None) == "normed":
             h = self._close(x, self.mixer_norm, pair=self.mixer.forward_pair(h, batch, cache, state))
         else:
             y = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
@@ -409,7 +409,107 @@ class PostNormBlock(Part):
         return None if h is None or planes.dumping(batch) else RoundedRows(x, h)
 
 
+class OutputNormBlock(Part):
+    """The norm on the sublayer's RESULT only: x <- x + norm1(mixer(x)), then x <- x + norm2(feed_forward(x)). The sublayers read
+    the residual rows themselves (rounded to the compute element type for their products; the 32-bit engine reads x as it
+    is). The feed-forward with its norm is optional (a layer that gives no `feed_forward` part has the first half only).
+
+    With `average` (the number of states the layer averages over: itself and every layer before it, and the embedding rows)
+    the layer's result is kept as a state of the step's depth history and what goes on is sum_j weight[j] X_j
+    (models/decoder.py hands the history to blocks that set `takes_history`).
+
+    The norm, the residual sum, the average and the rounded copy for the next reader are one pass over the row
+    (ops.output_norm); a mixer that offers `forward_pair` with a scaled join has it in the same pass. The norms are layer norms
+    or RMS norms.
+
+    params: layer (the LayerSpec), hidden_size, average (default 0: none), average_name (default "dwa")."""
+
+    SLOTS = {"mixer": "mixer", "mixer_norm": "norm", "feed_forward": "feed_forward", "feed_forward_norm": "norm"}
+    OPTIONAL = ("feed_forward", "feed_forward_norm")
+    takes_pending = True
+
+    def __init__(self, params, ctx, prefix=""):
+        super().__init__(params, ctx, prefix)
+        layer = params["layer"]
+        self.has_ff = "feed_forward" in layer.parts
+        slots = {n: r for n, r in self.SLOTS.items() if self.has_ff or n not in self.OPTIONAL}
+        self.parts = build_slots(self, layer, slots, ctx, prefix)
+        if not self.has_ff:
+            self.feed_forward = self.feed_forward_norm = None
+        for norm in (self.mixer_norm, self.feed_forward_norm):
+            if norm is not None and not isinstance(norm, (LayerNorm, RMSNorm)):
+                raise ValueError(f"layer {layer.prefix!r}: block 'output_norm' takes layer norms and RMS norms")
+        self.hidden, self.average = int(params["hidden_size"]), int(params.get("average", 0))
+        self.average_name, self.coef = prefix + params.get("average_name", "dwa"), None
+
+    @property
+    def takes_history(self):
+        return self.average > 0
+
+    def param_specs(self):
+        specs = [s for p in self.parts for s in p.param_specs()]
+        if self.average:
+            specs.append(ParamSpec(self.average_name, (self.average,), init="ones"))
+        return specs
+
+    def load(self, tensors):
+        for p in self.parts:
+            p.load(tensors)
+        if self.average:
+            self.coef = tensors[self.average_name].to(torch.float32).contiguous()
+
+    def weight_bytes(self):
+        return sum(p.weight_bytes() for p in self.parts)
+
+    def _close(self, x, norm, y, history=None, last=True):
+        """x <- x + norm(y), at the layer's end (`last`) averaged over the depth; returns the rounded copy of the new x (None
+        in the 32-bit engine)."""
+        rounded = None if self.ctx.dtype == torch.float32 else torch.empty(x.shape, dtype=self.ctx.dtype, device=x.device)
+        keep_in = keep = states = None
+        if history is not None:
+            if history.count == 0:
+                keep_in = history.next()
+            if last:
+                keep = history.next()
+                states = history.states[:history.count - 1]
+                if states.shape[0] + 1 != self.average:
+                    raise ValueError(f"{self.average_name}: an average over {self.average} states after {states.shape[0]} layers")
+        ops.output_norm(x, y, norm.weight, getattr(norm, "bias", None), norm.eps, rounded, keep_in, keep, states,
+                        self.coef if states is not None else None, center=isinstance(norm, LayerNorm))
+        return rounded
+
+    def _rows(self, x, carry):
+        if self.ctx.dtype == torch.float32:
+            return x
+        if isinstance(carry, RoundedRows) and carry.x is x:
+            return carry.rows
+        return ops.convert(x, self.ctx.dtype)
+
+    def forward(self, x, batch, cache, state, pending=None, history=None):
+        if isinstance(pending, ops.Pending):
+            pending.finish()
+        h = self._rows(x, pending)
+        if getattr(self.mixer, "join", None) == "scaled":
+            y = self.mixer.forward_pair(h, batch, cache, state)
+        else:
+            y = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
+            left = self.mixer.forward(h, y, batch, cache, state)
+            if isinstance(left, ops.Pending):
+                left.finish()
+        h = self._close(x, self.mixer_norm, y, history, last=not self.has_ff)
+        planes.record(batch, "after_mixer", x)
+        if self.has_ff:
+            y = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
+            left = self.feed_forward.forward(x if h is None else h, y, batch)
+            if isinstance(left, ops.Pending):
+                left.finish()
+            h = self._close(x, self.feed_forward_norm, y, history)
+        planes.record(batch, "after_feed_forward", x)
+        return None if h is None or planes.dumping(batch) else RoundedRows(x, h)
+
+
 register_part("block", "pre_norm", PreNormBlock)
+register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "post_norm", PostNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "pre_norm_scaled", ScaledPreNormBlock)

@@ -107,6 +107,39 @@ class GatedFF(Part):
         return None
 
 
+class ActivatedFF(Part):
+    """A dense feed-forward without a gate and without biases: out = Wdown act(Wup h), act "gelu" (the exact form, z Phi(z)),
+    computed on the product's 32-bit result and rounded once.
+
+    params: hidden_size, intermediate_size, activation (default "gelu"), up_name, down_name."""
+
+    def __init__(self, params, ctx, prefix=""):
+        super().__init__(params, ctx, prefix)
+        self.hidden, self.inter = int(params["hidden_size"]), int(params["intermediate_size"])
+        self.act = params.get("activation", "gelu")
+        if self.act != "gelu":
+            raise ValueError(f"feed-forward: activation {self.act!r} is not known (known: 'gelu')")
+        self.names = {k: prefix + params.get(k + "_name", f"mlp.{k}") for k in ("up", "down")}
+        self.wup = self.wdown = None
+
+    def param_specs(self):
+        return [ParamSpec(self.names["up"], (self.inter, self.hidden)), ParamSpec(self.names["down"], (self.hidden, self.inter))]
+
+    def load(self, tensors):
+        self.wup = ops.Weight(to_compute(tensors[self.names["up"]], self.ctx))
+        self.wdown = ops.Weight(to_compute(tensors[self.names["down"]], self.ctx))
+
+    def weight_bytes(self):
+        return self.wup.nbytes + self.wdown.nbytes
+
+    def forward(self, xn, x, batch):
+        act = torch.empty(xn.shape[0], self.inter, dtype=self.ctx.dtype, device=xn.device)
+        ops.linear_act(xn, self.wup, act, self.act)
+        planes.record(batch, "activation", act)
+        ops.linear_into_stream(act, self.wdown, x)
+        return None
+
+
 class PolyNormFF(Part):
     """A dense feed-forward without a gate: out = act(xn Wup^T) Wdown^T with the PolyNorm activation
     act(z) = c1 N(z) + c2 N(z^2) + c3 N(z^3) + c0, powers element by element, N(t) = t / sqrt(mean(t^2) + eps) over
@@ -205,4 +238,5 @@ class ClampedGLU(Part):
 register_part("feed_forward", "swiglu", SwiGLU)
 register_part("feed_forward", "polynorm", PolyNormFF)
 register_part("feed_forward", "gated", GatedFF)
+register_part("feed_forward", "activated", ActivatedFF)
 register_part("feed_forward", "clamped_glu", ClampedGLU)

@@ -3,13 +3,17 @@
     q, k, v = Wq h, Wk h, Wv h                         (heads x dim, kv_heads x dim, kv_heads x vdim; no biases)
     with row_norm: q <- q / rms(q) * wq, k <- k / rms(k) * wk, each over its WHOLE row (all heads at once, before they are
                    split into heads and before the rotation; eps inside the root; a weight per column)
+    with head_norm: the same per head, over its dim values, with a weight per dimension that the heads share
     q, k rotated on their first `rot_dims` dimensions   (pairing "half": (i, i + rot_dims / 2); "interleaved": (2i, 2i + 1))
     q, k divided by their root mean square over dim     (with unit_norm; eps inside the root, no weight)
-    score = q . k * scale over the keys the mask shows:
+    with q_temp: q at position p times 1 + coef ln(floor((p + 1) / every) + 1)
+    with values "keys": there is no Wv; the values are Wk h as projected, before norm and rotation (vdim = dim)
+    score = q . k * scale, with distance_bias minus r1_h ln(1 + r2_h (i - j)), over the keys the mask shows:
         "causal"   every j <= i
         "window"   j <= i and (i - j < window or j < keep_first)
         "chunk"    j <= i and floor(i / chunk) == floor(j / chunk), chunks counted from position 0 of the sequence
-    softmax; with `sink` a learned number per head joins the denominator as exp(sink) (no key, no value, not scaled)
+    softmax; with `sink` a learned number per head joins the denominator as exp(sink) (no key, no value, not scaled); sink
+    "one": the constant 1 does (a sink of 0)
     head h's result times sigmoid(Wg h): one number per head (gate "head") or per element (gate "element")
     out = Wo concat(heads)
 
@@ -20,9 +24,9 @@ sizes of every layer that reads it; empty: everything), because the layers that 
 far. Rotation angles, the unit norm, scores, softmax and the gate are 32-bit; q, k, v are rounded once.
 
 params: hidden_size, heads, kv_heads, dim, vdim, scale, eps, rot_dims, rot_base, rot_scaling (ops.rope_frequencies),
-pairing, unit_norm, row_norm, mask, window, keep_first, chunk, sink, gate, reads_cache, cache_chunks, cache_keep_all (a
-window's cache keeps everything: a reader looks back further), and the tensor names q, k, v, g, o, sink, q_norm, k_norm
-(`<key>_name`).
+pairing, unit_norm, row_norm, head_norm, q_temp (coef, every), values ("own" or "keys"), distance_bias, mask, window,
+keep_first, chunk, sink, gate, reads_cache, cache_chunks, cache_keep_all (a window's cache keeps everything: a reader looks
+back further), and the tensor names q, k, v, g, o, sink, q_norm, k_norm, r1, r2 (`<key>_name`).
 """
 from __future__ import annotations
 
@@ -35,7 +39,7 @@ from . import planes
 from .registry import CacheNeed, Mixer, register_part, to_compute
 
 _DEFAULT_NAMES = dict(q="mix.q", k="mix.k", v="mix.v", g="mix.g", o="mix.o", sink="mix.sink", q_norm="mix.q.norm",
-                      k_norm="mix.k.norm")
+                      k_norm="mix.k.norm", r1="mix.r1", r2="mix.r2")
 
 
 def _chunks_dead(spec, q):
@@ -70,7 +74,18 @@ class MaskedAttentionMixer(Mixer):
         self.window, self.keep_first, self.chunk = int(p.get("window") or 0), int(p.get("keep_first") or 0), int(p.get("chunk") or 0)
         if (self.mask == "window" and self.window <= 0) or (self.mask == "chunk" and self.chunk <= 0):
             raise ValueError(f"attention: mask {self.mask!r} needs its size")
-        self.has_sink = bool(p.get("sink", False))
+        self.head_norm = bool(p.get("head_norm", False))
+        if self.head_norm and self.row_norm:
+            raise ValueError("attention: a norm over whole rows and one per head exclude each other")
+        self.q_temp = (float(p["q_temp"][0]), float(p["q_temp"][1])) if p.get("q_temp") else None
+        if self.q_temp and self.q_temp[1] <= 0:
+            raise ValueError(f"attention: a query temperature every {self.q_temp[1]} positions")
+        self.shared_values = p.get("values", "own") == "keys"
+        if self.shared_values and (self.vdim != self.dim or self.reads_cache_param(p)):
+            raise ValueError(f"attention: values that are the keys need vdim = dim and a cache of their own ({self.vdim}, {self.dim})")
+        self.distance_bias = bool(p.get("distance_bias", False))
+        self.sink_one = p.get("sink") == "one"
+        self.has_sink = bool(p.get("sink", False)) and not self.sink_one
         self.gate = p.get("gate") or "none"
         if self.gate not in ("none", "head", "element"):
             raise ValueError(f"attention: gate {self.gate!r} is not known (known: 'none', 'head', 'element')")
@@ -80,9 +95,13 @@ class MaskedAttentionMixer(Mixer):
         if self.mask != "chunk" and self.cache_chunks:
             raise ValueError("attention: the cache retains less than the mask sees")
         self.names = {k: prefix + p.get(k + "_name", d) for k, d in _DEFAULT_NAMES.items()}
-        self.w_in = self.wo = self.sink = self.table = self.row_norm_w = None
+        self.w_in = self.wo = self.sink = self.table = self.norm_w = self.distance = None
         if not ctx.is_meta:
             self.table = ops.shared_rope_table(self.rot_dims, self.rot_base, ctx.max_model_len, ctx.device, p.get("rot_scaling"))
+
+    @staticmethod
+    def reads_cache_param(p):
+        return bool(p.get("reads_cache", False))
 
     @property
     def n_q(self):
@@ -90,7 +109,7 @@ class MaskedAttentionMixer(Mixer):
 
     @property
     def n_kv(self):
-        return 0 if self.reads_cache else self.kv_heads * (self.dim + self.vdim)
+        return 0 if self.reads_cache else self.kv_heads * (self.dim + (0 if self.shared_values else self.vdim))
 
     @property
     def n_gate(self):
@@ -100,11 +119,15 @@ class MaskedAttentionMixer(Mixer):
         n, W = self.names, self.hidden
         specs = [ParamSpec(n["q"], (self.n_q, W))]
         if not self.reads_cache:
-            specs += [ParamSpec(n["k"], (self.kv_heads * self.dim, W)), ParamSpec(n["v"], (self.kv_heads * self.vdim, W))]
-        if self.row_norm:
-            specs.append(ParamSpec(n["q_norm"], (self.n_q,), init="ones"))
+            specs.append(ParamSpec(n["k"], (self.kv_heads * self.dim, W)))
+            if not self.shared_values:
+                specs.append(ParamSpec(n["v"], (self.kv_heads * self.vdim, W)))
+        if self.row_norm or self.head_norm:
+            specs.append(ParamSpec(n["q_norm"], (self.dim if self.head_norm else self.n_q,), init="ones"))
             if not self.reads_cache:
-                specs.append(ParamSpec(n["k_norm"], (self.kv_heads * self.dim,), init="ones"))
+                specs.append(ParamSpec(n["k_norm"], (self.dim if self.head_norm else self.kv_heads * self.dim,), init="ones"))
+        if self.distance_bias:
+            specs += [ParamSpec(n["r1"], (self.heads,), init="ones"), ParamSpec(n["r2"], (self.heads,), init="ones")]
         if self.has_sink:
             specs.append(ParamSpec(n["sink"], (self.heads,), init="zeros"))
         if self.n_gate:
@@ -114,14 +137,18 @@ class MaskedAttentionMixer(Mixer):
 
     def load(self, tensors):
         t = {k: to_compute(tensors[n], self.ctx) for k, n in self.names.items() if n in tensors}
-        mats = [t["q"]] + ([] if self.reads_cache else [t["k"], t["v"]]) + ([t["g"]] if self.n_gate else [])
+        mats = [t["q"]] + ([] if self.reads_cache else [t["k"]] if self.shared_values else [t["k"], t["v"]]) + ([t["g"]] if self.n_gate else [])
         dt = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
         self.w_in = ops.Weight(torch.cat([m.to(dt) for m in mats], 0).contiguous())     # rows [q | k | v | g] or [q | g]
         self.wo = ops.Weight(t["o"])
         self.sink = t["sink"].to(torch.float32).contiguous() if self.has_sink else None
-        if self.row_norm:
+        if self.sink_one:
+            self.sink = torch.zeros(self.heads, dtype=torch.float32, device=self.w_in.t.device)
+        if self.row_norm or self.head_norm:
             wq = t["q_norm"].to(torch.float32).contiguous()
-            self.row_norm_w = (wq, wq if self.reads_cache else t["k_norm"].to(torch.float32).contiguous())
+            self.norm_w = (wq, wq if self.reads_cache else t["k_norm"].to(torch.float32).contiguous())
+        if self.distance_bias:
+            self.distance = (t["r1"].to(torch.float32).contiguous(), t["r2"].to(torch.float32).contiguous())
 
     def weight_bytes(self):
         return self.w_in.nbytes + self.wo.nbytes
@@ -140,15 +167,17 @@ class MaskedAttentionMixer(Mixer):
         ops.linear_rows32(xn, self.w_in, proj)
         q = torch.empty(T, self.n_q, dtype=self.ctx.dtype, device=xn.device)
         write = cache.write and not self.reads_cache
-        ops.rope_norm_store(proj, (0, self.n_q, self.n_q + self.kv_heads * self.dim), batch.positions,
+        v_off = self.n_q if self.shared_values else self.n_q + self.kv_heads * self.dim
+        ops.rope_norm_store(proj, (0, self.n_q, v_off), batch.positions,
                             batch.slot_maps[cache.group] if write else None, self.table, self.rot_dims, self.pairing,
                             self.unit_norm, self.eps, q, cache.k, cache.v, self.heads, self.kv_heads, self.dim, self.vdim,
-                            self.ctx.page_size, row_norm=self.row_norm_w, row_norm_eps=self.eps)
+                            self.ctx.page_size, row_norm=self.norm_w if self.row_norm else None, row_norm_eps=self.eps,
+                            head_norm=self.norm_w if self.head_norm else None, q_temp=self.q_temp)
         att = torch.empty(T, self.heads * self.vdim, dtype=self.ctx.dtype, device=xn.device)
         ops.attention_masked(q, cache.k, cache.v, batch, cache.group, att, self.heads, self.kv_heads, self.dim, self.vdim,
                              self.ctx.page_size, self.scale, self.mask, self.window, self.keep_first, self.chunk, self.sink,
                              gate=proj if self.n_gate else None, gate_offset=self.n_q + self.n_kv,
-                             gate_per_head=self.gate == "head")
+                             gate_per_head=self.gate == "head", distance=self.distance)
         planes.record(batch, "q", q)
         planes.record(batch, "attention", att)
         ops.linear_into_stream(att, self.wo, x)

@@ -10,14 +10,22 @@ Without biases Wgate_e (s h) = s (Wgate_e h): the products run on h and the scor
 A second form is chosen by parameters: `router_bias` adds a bias to the router's logits; `score` "softmax_chosen" lets the
 `top` largest LOGITS choose and takes as weights the softmax over the chosen logits alone; `weight_at` "output" multiplies
 the expert's RESULT by the weight (brought in at the activation too: the down product is linear).
+A third: `score` "sigmoid_normed" chooses by sigmoid(z) + a correction per expert, where `groups` (count, keep) is given
+only within the `keep` groups of neighbouring experts that rank best by the sum of their two largest; the weights are the
+chosen sigmoid(z), without the correction, over their sum, times `weight_scale`.
+
+With `shared_size` a shared expert of the same form and that size runs for every token and is added; with `shared_gate` its
+result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits).
 Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: a few rows one
 by one, more of them sorted by expert so that an expert's weights are read once for all of its rows. A step with prompt
 portions sorts its (row, choice) pairs by expert and gives each expert's block of rows to the ordinary products (the
 tensor-core kernels in bfloat16), for which the host reads the experts' row counts once a layer.
 
 params: hidden_size, experts, top, expert_size, score (default "sigmoid"), weight_at (default "input"), router_bias
-(default False), router_name (default "mlp.router"), router_bias_name (default "mlp.router.b"), expert_prefix (default
-"mlp.e": expert i's tensors are <expert_prefix><i>.gate / .up / .down).
+(default False), groups (count, keep) (default none), weight_scale (default 1), shared_size (default none), shared_gate (default
+False), router_name (default "mlp.router"), router_bias_name (default "mlp.router.b"), correction_name (default
+"mlp.correction"), expert_prefix (default "mlp.e": expert i's tensors are <expert_prefix><i>.gate / .up / .down),
+shared_prefix (default "mlp.shared": .gate / .up / .down, and .sg for its gate).
 """
 from __future__ import annotations
 
@@ -29,6 +37,7 @@ from . import planes
 from .registry import Part, register_part, to_compute
 
 SORTED_MIN_PAIRS = 64     # fewer (row, choice) pairs than this never go to the ordinary products
+SHARED_MIN_ROWS = 9       # fewer rows run the shared expert row by row
 GROUPED_MIN_PAIRS = 20    # fewer than this run row by row; from here on an expert's rows share one pass over its weights
 
 
@@ -48,7 +57,19 @@ class RoutedFF(Part):
         self.router_bias_name = prefix + params.get("router_bias_name", "mlp.router.b") if params.get("router_bias") else None
         self.router_bias = None
         self.expert_prefix = prefix + params.get("expert_prefix", "mlp.e")
-        self.router = self.wgu = self.wdown = None
+        self.router = self.wgu = self.wdown = self.correction = None
+        self.correction_name = (prefix + params.get("correction_name", "mlp.correction")) if self.score == "sigmoid_normed" else None
+        self.groups, self.keep = (int(g) for g in (params.get("groups") or (1, 1)))
+        self.weight_scale = float(params.get("weight_scale", 1.0))
+        if self.experts % self.groups or not 1 <= self.keep <= self.groups or self.keep * (self.experts // self.groups) < self.top:
+            raise ValueError(f"routed feed-forward: {self.experts} experts in {self.groups} groups of which {self.keep} stay, "
+                             f"{self.top} chosen")
+        if self.groups > 1 and self.score != "sigmoid_normed":
+            raise ValueError(f"routed feed-forward: groups go with score 'sigmoid_normed', not {self.score!r}")
+        self.shared = int(params.get("shared_size") or 0)
+        self.shared_gated = bool(params.get("shared_gate", False)) and self.shared > 0
+        self.shared_prefix = prefix + params.get("shared_prefix", "mlp.shared")
+        self.shared_gate = self.s_gu = self.s_down = self.ones = self.index = None
 
     def _expert(self, i, key):
         return f"{self.expert_prefix}{i}.{key}"
@@ -57,6 +78,14 @@ class RoutedFF(Part):
         specs = [ParamSpec(self.router_name, (self.experts, self.hidden))]
         if self.router_bias_name:
             specs.append(ParamSpec(self.router_bias_name, (self.experts,), init="zeros"))
+        if self.correction_name:
+            specs.append(ParamSpec(self.correction_name, (self.experts,), init="zeros"))
+        if self.shared:
+            s = self.shared_prefix
+            specs += [ParamSpec(s + ".gate", (self.shared, self.hidden)), ParamSpec(s + ".up", (self.shared, self.hidden)),
+                      ParamSpec(s + ".down", (self.hidden, self.shared))]
+            if self.shared_gated:
+                specs.append(ParamSpec(s + ".sg", (1, self.hidden)))
         for i in range(self.experts):
             specs += [ParamSpec(self._expert(i, "gate"), (self.inter, self.hidden)),
                       ParamSpec(self._expert(i, "up"), (self.inter, self.hidden)),
@@ -68,6 +97,15 @@ class RoutedFF(Part):
         self.router = t(self.router_name)
         if self.router_bias_name:
             self.router_bias = t(self.router_bias_name).to(self.router.dtype).contiguous()
+        if self.correction_name:
+            self.correction = t(self.correction_name).to(self.router.dtype).contiguous()
+        if self.shared:
+            g, u, d = (t(f"{self.shared_prefix}.{k}") for k in ("gate", "up", "down"))
+            sdt = g.dtype if g.dtype == u.dtype == d.dtype else torch.float32
+            self.s_gu = ops.Weight(torch.cat([g.to(sdt), u.to(sdt)], 0).contiguous())        # gate rows, then up rows
+            self.s_down = ops.Weight(d.to(sdt).contiguous())
+            if self.shared_gated:
+                self.shared_gate = t(self.shared_prefix + ".sg").to(self.router.dtype).reshape(-1).contiguous()
         mats = [t(self._expert(i, k)) for i in range(self.experts) for k in ("gate", "up", "down")]
         dt = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
         E, F, W = self.experts, self.inter, self.hidden
@@ -80,11 +118,38 @@ class RoutedFF(Part):
     def weight_bytes(self):
         """What a single row reads: the router and `top` experts."""
         per = (self.wgu.numel() + self.wdown.numel()) * self.wgu.element_size() // self.experts
-        return self.router.numel() * self.router.element_size() + self.top * per
+        shared = self.s_gu.nbytes + self.s_down.nbytes if self.shared else 0
+        return self.router.numel() * self.router.element_size() + self.top * per + shared
+
+    def _row_index(self, T, dev):
+        """(0 .. T-1, zeros, ones): a shared expert as the one expert of every row."""
+        if self.index is None or self.index[0].numel() < T:
+            n = max(T, 2048)
+            self.index = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, 1, dtype=torch.int32, device=dev),
+                          torch.ones(n, dtype=torch.float32, device=dev))
+        return tuple(t[:T] for t in self.index)
+
+    def _add_shared(self, xn, x, weight):
+        """x += weight * shared expert: the weight enters at the activation in 32-bit (the down product is linear)."""
+        T, F = xn.shape[0], self.shared
+        rows, zeros, ones = self._row_index(T, xn.device)
+        weight = ones if weight is None else weight
+        if T < SHARED_MIN_ROWS:
+            ops.moe_rows(xn, self.s_gu.t.unsqueeze(0), self.s_down.t.unsqueeze(0), zeros, weight, x, True)
+            return
+        gu = torch.empty(T, 2 * F, dtype=torch.float32, device=xn.device)
+        ops.linear(xn, self.s_gu, gu)
+        act = torch.empty(T, F, dtype=self.ctx.dtype, device=xn.device)
+        ops.moe_act(gu, rows, weight, act, True)
+        ops.linear_into_stream(act, self.s_down, x)
 
     def forward(self, xn, x, batch):
         T, top, F = xn.shape[0], self.top, self.inter
-        expert, score = ops.moe_route(xn, self.router, top, self.router_bias, self.score)
+        shared_weight = torch.empty(T, dtype=torch.float32, device=xn.device) if self.shared_gated else None
+        expert, score = ops.moe_route(xn, self.router, top, self.router_bias, self.score, self.correction, self.groups, self.keep,
+                                      self.weight_scale, self.shared_gate, shared_weight)
+        if self.shared:
+            self._add_shared(xn, x, shared_weight)
         if T * top < GROUPED_MIN_PAIRS:
             ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output)
             return None
