@@ -544,8 +544,36 @@ def mavinex_configs(size: dict, window: int):
     return mavinex, runopel_configs(size, window)[0]
 
 
-DESIGNS = {"torirax": design_configs, "vegodra": vegodra_configs, "runopel": runopel_configs, "mavinex": mavinex_configs}
-BESIDE = {"torirax": "llama", "vegodra": "llama", "runopel": "vegodra", "mavinex": "runopel"}
+def gakupel_configs(size: dict, window: int):
+    """(Gakupel config, Mavinex config) of equal width, depth, head counts and feed-forward width; Mavinex is the closest of
+    the other designs (attention beside a recurrence, experts in grouped products). Gakupel's layers cycle attention with a
+    distance bias beside the matrix memory (heads of head_dim x head_dim), attention whose values are its keys, the first
+    again, the gated delta rule (heads of head_dim x head_dim, four taps). Feed-forwards alternate between the dense one
+    without a gate and eight experts of half its width in four groups, two per token, with a shared expert of a quarter.
+    There is no window in the design."""
+    W, L, H, G, D = size["width"], size["layers"], size["heads"], size["kv"], size["head_dim"]
+    layers = []
+    for i in range(L):
+        if i % 2 == 0:
+            mlp = dict(kind="dense", ff=size["ff"])
+        else:
+            mlp = dict(kind="moe", expert=dict(ff=size["ff"] // 2), router=dict(experts=8, top=2, groups=dict(count=4, keep=2), scale=1.5),
+                       shared=dict(ff=size["ff"] // 4))
+        if i % 2 == 0:
+            left = dict(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, q_temp=dict(coef=0.1, every=CONTEXT_LEN // 4))
+            right = dict(heads=H, dim=D, vdim=D, gate_cap=15.0)
+            layers.append(dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.5, right_scale=0.5), mlp=mlp))
+        elif i % 4 == 1:
+            m = dict(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, rot=dict(base=10000.0, dims=D // 2))
+            layers.append(dict(type="attention", mixer=m, mlp=mlp))
+        else:
+            layers.append(dict(type="delta", mixer=dict(heads=H, kv_heads=H, dim=D, vdim=D, conv=4), mlp=mlp))
+    gakupel = dict(architecture="Gakupel", vocab=size["vocab"], width=W, max_positions=CONTEXT_LEN, norm=dict(eps=1e-6), layers=layers)
+    return gakupel, mavinex_configs(size, window)[0]
+
+
+DESIGNS = {"gakupel": gakupel_configs, "torirax": design_configs, "vegodra": vegodra_configs, "runopel": runopel_configs, "mavinex": mavinex_configs}
+BESIDE = {"gakupel": "mavinex", "torirax": "llama", "vegodra": "llama", "runopel": "vegodra", "mavinex": "runopel"}
 
 
 def kernel_table(one, reps: int = 3):
@@ -590,7 +618,7 @@ def kernel_table(one, reps: int = 3):
 
 def design_bench(a) -> int:
     """Prefill and decode throughput of the chosen design and of the model beside it (the Llama decoder for Torirax and
-    Vegodra, Vegodra for Runopel, Runopel for Mavinex) at equal layer sizes, with each step's kernels by name; one JSON line. The default run
+    Vegodra, Vegodra for Runopel, Runopel for Mavinex, Mavinex for Gakupel) at equal layer sizes, with each step's kernels by name; one JSON line. The default run
     of this file is untouched by this option."""
     import torch
 

@@ -96,14 +96,17 @@ __device__ __forceinline__ void ad_load_rows(const __nv_bfloat16* __restrict__ k
 // row's first chunk adds the partials through distributed shared memory, in the same order and with the same
 // arithmetic as the merge through memory below: fence, counter and the partials' round trip through L2 (4 of a
 // layer's 11 us at 8 requests) become two cluster barriers. Blocks without keys only pass the barriers.
-template <int D, int G, bool TMA, int RW, int KW, int SR, bool CL>
+// EX: a distance bias, r1 ln(1 + r2 (p - j)) off the score of key j, and a sink, exp(sink) in the denominator (a number
+// per head each; the sink joins in the block of the row's first chunk).
+template <int D, int G, bool TMA, int RW, int KW, int SR, bool CL, bool EX>
 __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, int* __restrict__ status,
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
     const int* __restrict__ bt, int bt_stride, const int* __restrict__ row_req, const int* __restrict__ pos,
     __nv_bfloat16* __restrict__ out, float* __restrict__ part_acc, float* __restrict__ part_ml, int Hq, int Hkv,
     int page_size, int window, float scale_log2, int chunk, int S, const int* __restrict__ q_len, int row_limit,
-    const int* __restrict__ ctx_len, int* __restrict__ counters) {
+    const int* __restrict__ ctx_len, int* __restrict__ counters, const float* __restrict__ r1p,
+    const float* __restrict__ r2p, const float* __restrict__ sink) {
   constexpr int CH = D / 8, KS = D / 16, NT_O = D / 8, WK = 64;  // WK: keys per warp pass
   extern __shared__ __align__(128) uint8_t smem_dyn[];
   uint8_t* smem_raw = TMA ? (uint8_t*)(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023) : smem_dyn;   // the swizzle wants 1 KB
@@ -268,6 +271,16 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
       }
     }
     float mx = -INFINITY;
+    const float sl = EX ? 1.f : scale_log2;      // EX: the scores are scaled here, where their bias is taken off
+    if constexpr (EX) {
+      const float r1 = r1p && g < G ? r1p[h * G + g] : 0.f, r2 = r1p && g < G ? r2p[h * G + g] : 0.f;
+      const float d0 = (float)(p - k0 - kb - 2 * tq);
+#pragma unroll
+      for (int i = 0; i < RW / 8; i++)
+#pragma unroll
+        for (int e = 0; e < 2; e++)
+          sc[i][e] = fmaf(-r1, __log2f(fmaf(r2, d0 - (float)(i * 8 + e), 1.f)), sc[i][e] * scale_log2);
+    }
 #pragma unroll
     for (int i = 0; i < RW / 8; i++)
 #pragma unroll
@@ -277,14 +290,14 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
       }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-    const float mn = fmaxf(m_run, mx * scale_log2);   // mx is a real score here: a pass never runs without a visible key
+    const float mn = fmaxf(m_run, mx * sl);   // mx is a real score here: a pass never runs without a visible key
     const float corr = hb_exp2(m_run - mn);
     m_run = mn;
     float sum = 0.f;
     uint32_t pf[RW / 16][4];
 #pragma unroll
     for (int i = 0; i < RW / 8; i++) {
-      const float p0 = hb_exp2(sc[i][0] * scale_log2 - mn), p1 = hb_exp2(sc[i][1] * scale_log2 - mn);
+      const float p0 = hb_exp2(sc[i][0] * sl - mn), p1 = hb_exp2(sc[i][1] * sl - mn);
       sum += p0 + p1;
       pf[i >> 1][(i & 1) * 2] = hb_pack_bf16(p0, p1);
       pf[i >> 1][(i & 1) * 2 + 1] = 0u;  // rows 8..15 of the tile are padding
@@ -326,6 +339,11 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
 #pragma unroll
     for (int w = 0; w < AD_WARPS; w++) m = fmaxf(m, red_ml[(w * G + gg) * 2]);
     float a = 0.f, l = 0.f;
+    if (EX && sink && s == s_lo) {
+      const float sk = sink[h * G + gg] * 1.4426950408889634f;
+      m = fmaxf(m, sk);
+      l = hb_exp2(sk - m);
+    }
 #pragma unroll
     for (int w = 0; w < AD_WARPS; w++) {
       const float f = hb_exp2(red_ml[(w * G + gg) * 2] - m);  // 0 for a warp without keys
@@ -452,29 +470,30 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
   HB_TL_MARK(0, 3);
 }
 
-template <int D, bool TMA, int RW, int KW, int SR, bool CL = false>
+template <int D, bool TMA, int RW, int KW, int SR, bool CL, bool EX>
 static int launch_decode(int G, dim3 grid, size_t smem, cudaStream_t st, const CUtensorMap& mk, const CUtensorMap& mv,
                          int* status, const __nv_bfloat16* q, const __nv_bfloat16* kc, const __nv_bfloat16* vc,
                          const int* bt, int bt_stride, const int* row_req, const int* pos, __nv_bfloat16* out, float* pa,
                          float* pm, int Hq, int Hkv, int page_size, int window, float scale, int chunk, int S,
-                         const int* q_len, int row_limit, const int* ctx_len, int* counters) {
+                         const int* q_len, int row_limit, const int* ctx_len, int* counters, const float* r1, const float* r2,
+                         const float* sink) {
 #define HB_AD_CASE(GG)                                                                                              \
   case GG:                                                                                                          \
     {                                                                                                               \
       static bool configured = false;                                                                               \
       if (!configured) {                                                                                            \
-        cudaFuncSetAttribute(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+        cudaFuncSetAttribute(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
         configured = true;                                                                                          \
       }                                                                                                             \
     }                                                                                                               \
     if (CL)                                                                                                         \
-      hb_launch_cluster(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL>, grid, AD_THREADS, smem, st, dim3(grid.x, 1, 1), mk, mv, status, \
+      hb_launch_cluster(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, grid, AD_THREADS, smem, st, dim3(grid.x, 1, 1), mk, mv, status, \
                         q, kc, vc, bt, bt_stride, row_req, pos, out, pa, pm, Hq, Hkv, page_size, window, scale, chunk, S,    \
-                        q_len, row_limit, ctx_len, counters);                                                       \
+                        q_len, row_limit, ctx_len, counters, r1, r2, sink);                                         \
     else                                                                                                            \
-      hb_launch(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL>, grid, AD_THREADS, smem, st, mk, mv, status, q, kc, vc, bt, bt_stride, \
+      hb_launch(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, grid, AD_THREADS, smem, st, mk, mv, status, q, kc, vc, bt, bt_stride, \
                 row_req, pos, out, pa, pm, Hq, Hkv, page_size, window, scale, chunk, S, q_len, row_limit, ctx_len,  \
-                counters);                                                                                          \
+                counters, r1, r2, sink);                                                                            \
     return 0;
   switch (G) {
     HB_AD_CASE(1) HB_AD_CASE(2) HB_AD_CASE(3) HB_AD_CASE(4) HB_AD_CASE(5) HB_AD_CASE(6) HB_AD_CASE(7) HB_AD_CASE(8)
@@ -499,12 +518,14 @@ HB_EXPORT int hb_attn_decode_supported(int Hq, int Hkv, int D) {
 HB_EXPORT int hb_attn_decode(const void* q, const void* kc, const void* vc, long n_pages, const int* bt, int bt_stride,
                              const int* row_req, const int* pos, void* out, float* workspace, int* counters, int T,
                              int Hq, int Hkv, int D, int page_size, int window, float scale, int chunk, int max_pos,
-                             const int* q_len, int row_limit, const int* ctx_len, int* status, cudaStream_t st) {
+                             const int* q_len, int row_limit, const int* ctx_len, int* status, const float* r1, const float* r2,
+                             const float* sink, cudaStream_t st) {
   if (T <= 0) return 0;
   if (!hb_attn_decode_supported(Hq, Hkv, D)) HB_FAIL("hb_attn_decode: %d/%d heads of %d are not supported", Hq, Hkv, D);
   if (chunk <= 0 || chunk % 32) HB_FAIL("hb_attn_decode: chunk %d must be a positive multiple of 32", chunk);
   if (T > 65535 || Hkv > 65535 || max_pos / chunk + 1 > 65535) HB_FAIL("hb_attn_decode: %d rows / %d kv heads / %d chunks are beyond the grid limit", T, Hkv, max_pos / chunk + 1);
   const int G = Hq / Hkv, S = max_pos / chunk + 1;
+  if ((r1 != nullptr) != (r2 != nullptr)) HB_FAIL("hb_attn_decode: a distance bias needs both of its vectors");
   if (S > 1 && (!workspace || !counters)) HB_FAIL("hb_attn_decode: rows that span %d chunks need a workspace and counters", S);
   if (chunk % 64) HB_FAIL("hb_attn_decode: chunk %d must be a multiple of 64", chunk);
   const long cache_rows = n_pages * Hkv * page_size;
@@ -542,17 +563,26 @@ HB_EXPORT int hb_attn_decode(const void* q, const void* kc, const void* vc, long
   const float sl2 = scale * 1.4426950408889634f;
   int r = 1;
 #define HB_AD_ARGS G, grid, smem, st, mk, mv, status, qq, kk, vv, bt, bt_stride, row_req, pos, (__nv_bfloat16*)out, pa, pm, Hq, Hkv, \
-                   page_size, window, sl2, chunk, S, q_len, row_limit, ctx_len, counters
+                   page_size, window, sl2, chunk, S, q_len, row_limit, ctx_len, counters, r1, r2, sink
   // a step of few rows whose chunks fit one cluster: the chunks' partial results meet in distributed shared memory
   const bool cl = tma && S >= 2 && S <= 8 && T <= g_ad_cluster_rows;
-  if (D == 64 && resident && cl) r = launch_decode<64, true, 64, 128, 128, true>(HB_AD_ARGS);
-  else if (D == 64 && wide && cl) r = launch_decode<64, true, 64, 128, 64, true>(HB_AD_ARGS);
-  else if (halves && cl) r = launch_decode<128, true, 32, 64, 32, true>(HB_AD_ARGS);
-  else if (D == 64 && resident) r = launch_decode<64, true, 64, 128, 128>(HB_AD_ARGS);
-  else if (D == 64 && wide) r = launch_decode<64, true, 64, 128, 64>(HB_AD_ARGS);
-  else if (D == 64) r = tma ? launch_decode<64, true, 64, 64, 64>(HB_AD_ARGS) : launch_decode<64, false, 64, 64, 64>(HB_AD_ARGS);
-  else if (halves) r = launch_decode<128, true, 32, 64, 32>(HB_AD_ARGS);
-  else if (D == 128) r = tma ? launch_decode<128, true, 64, 64, 64>(HB_AD_ARGS) : launch_decode<128, false, 64, 64, 64>(HB_AD_ARGS);
+  if (r1 || sink) {
+    if (D == 64 && resident && cl) r = launch_decode<64, true, 64, 128, 128, true, true>(HB_AD_ARGS);
+    else if (D == 64 && wide && cl) r = launch_decode<64, true, 64, 128, 64, true, true>(HB_AD_ARGS);
+    else if (halves && cl) r = launch_decode<128, true, 32, 64, 32, true, true>(HB_AD_ARGS);
+    else if (D == 64 && resident) r = launch_decode<64, true, 64, 128, 128, false, true>(HB_AD_ARGS);
+    else if (D == 64 && wide) r = launch_decode<64, true, 64, 128, 64, false, true>(HB_AD_ARGS);
+    else if (halves) r = launch_decode<128, true, 32, 64, 32, false, true>(HB_AD_ARGS);
+    else HB_FAIL("hb_attn_decode: a distance bias or a sink wants whole pages of 8 to %d tokens and no window", D == 64 ? 64 : 32);
+  }
+  else if (D == 64 && resident && cl) r = launch_decode<64, true, 64, 128, 128, true, false>(HB_AD_ARGS);
+  else if (D == 64 && wide && cl) r = launch_decode<64, true, 64, 128, 64, true, false>(HB_AD_ARGS);
+  else if (halves && cl) r = launch_decode<128, true, 32, 64, 32, true, false>(HB_AD_ARGS);
+  else if (D == 64 && resident) r = launch_decode<64, true, 64, 128, 128, false, false>(HB_AD_ARGS);
+  else if (D == 64 && wide) r = launch_decode<64, true, 64, 128, 64, false, false>(HB_AD_ARGS);
+  else if (D == 64) r = tma ? launch_decode<64, true, 64, 64, 64, false, false>(HB_AD_ARGS) : launch_decode<64, false, 64, 64, 64, false, false>(HB_AD_ARGS);
+  else if (halves) r = launch_decode<128, true, 32, 64, 32, false, false>(HB_AD_ARGS);
+  else if (D == 128) r = tma ? launch_decode<128, true, 64, 64, 64, false, false>(HB_AD_ARGS) : launch_decode<128, false, 64, 64, 64, false, false>(HB_AD_ARGS);
 #undef HB_AD_ARGS
   if (r) HB_FAIL("hb_attn_decode: no kernel for group %d", G);
   HB_CHECK_LAUNCH("hb_attn_decode");

@@ -24,6 +24,12 @@
 // positions and a row's running max and sum are its own, a row's result does not depend on how
 // the prompt was cut or on what else is in the batch. Replaces flash_prefill_mma_kernel of the
 // reference (src/kernels.cuh:1335-1482). Every wait is bounded.
+//
+// EX: a distance bias, r1 ln(1 + r2 (i - j)) off the score of query i and key j (r1, r2 >= 0, a number per head), and a
+// sink, exp(sink) in the denominator (a number per head). The bias grows with the distance, so the unbiased maximum of a
+// tile less the bias of its nearest key bounds the tile's scores from above; that bound takes the maximum's place (any
+// reference value gives the same quotient; the caller keeps the bias's spread within a tile far from the exponent's range),
+// and a score meets its bias once, in the exponent.
 #include "tc_common.cuh"
 
 constexpr int FT_BM = 128, FT_BN = 128;
@@ -51,12 +57,13 @@ struct FtBars {
 
 // head_dim 128: operands of two 64-column tiles each, the output tile 128 columns wide (192 KB of
 // shared memory: one CTA per SM).
-template <int FT_D>
+template <int FT_D, bool EX>
 __global__ void __launch_bounds__(FT_D == 64 ? 256 : 192, FT_D == 64 ? 2 : 1) flash_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, const int* __restrict__ bt, int bt_stride, const int* __restrict__ q_start,
     const int* __restrict__ q_len, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, int Hq, int Hkv,
-    int page_size, int window, float scale_log2, int min_rows, int* status) {
+    int page_size, int window, float scale_log2, int min_rows, int* status, const float* __restrict__ r1p,
+    const float* __restrict__ r2p, const float* __restrict__ sink) {
   // the 128-byte swizzle wants the tiles on 1 KB boundaries; with no room for slack (two CTAs an SM) the
   // dynamic shared memory itself has to start on one, which is checked below
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -197,6 +204,7 @@ __global__ void __launch_bounds__(FT_D == 64 ? 256 : 192, FT_D == 64 ? 2 : 1) fl
     // l_run is in the same units, and O / l_run is exact whichever maxima were used.
     constexpr float FT_SLACK = 8.f;
     float m_run = -INFINITY, l_run = 0.f;
+    const float r1 = EX && r1p ? r1p[hq] : 0.f, r2 = EX && r1p ? r2p[hq] : 0.f;
     bool ok = true;   // every wait's outcome is made uniform over the warp: the tensor-memory accesses below are warp-wide
     for (int i = 0; i < n_tiles && ok; i++) {
       const int k_base = (kt_lo + i) * FT_BN;
@@ -227,7 +235,9 @@ __global__ void __launch_bounds__(FT_D == 64 ? 256 : 192, FT_D == 64 ? 2 : 1) fl
           for (int j = 0; j < 64; j++) mx4[j & 3] = fmaxf(mx4[j & 3], __uint_as_float(sr[j]));
         }
       }
-      const float m_tile = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+      float m_tile = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+      const float dist0 = (float)(qp - k_base);                     // of the tile's first key
+      if (EX) m_tile -= r1 * __log2f(fmaf(r2, fmaxf(dist0 - (FT_BN - 1), 0.f), 1.f));
       const bool grow = m_tile > m_run + FT_SLACK;   // also the first tile with a visible key: m_run is -inf
       float corr = 1.f;
       if (grow) {
@@ -253,8 +263,12 @@ __global__ void __launch_bounds__(FT_D == 64 ? 256 : 192, FT_D == 64 ? 2 : 1) fl
         }
 #pragma unroll
         for (int j = 0; j < 64; j += 2) {  // masked scores are -inf: 2^-inf = 0
-          const float p0 = hb_exp2(fmaf(__uint_as_float(sr[j]), scale_log2, -sub));
-          const float p1 = hb_exp2(fmaf(__uint_as_float(sr[j + 1]), scale_log2, -sub));
+          float e0 = fmaf(__uint_as_float(sr[j]), scale_log2, -sub), e1 = fmaf(__uint_as_float(sr[j + 1]), scale_log2, -sub);
+          if (EX) {   // (a key behind the row is masked: any finite bias will do)
+            e0 = fmaf(-r1, __log2f(fmaxf(fmaf(r2, dist0 - (float)(j + hh * 64), 1.f), 1.f)), e0);
+            e1 = fmaf(-r1, __log2f(fmaxf(fmaf(r2, dist0 - (float)(j + 1 + hh * 64), 1.f), 1.f)), e1);
+          }
+          const float p0 = hb_exp2(e0), p1 = hb_exp2(e1);
           sum4[(j >> 1) & 3] += p0 + p1;
           sr[j >> 1] = hb_pack_bf16(p0, p1);
         }
@@ -293,6 +307,7 @@ __global__ void __launch_bounds__(FT_D == 64 ? 256 : 192, FT_D == 64 ? 2 : 1) fl
     }
     if (ok && __all_sync(0xffffffffu, hb_mbar_wait(&bar->o_full, (n_tiles - 1) & 1, abort_flag))) {
       hb_tc_fence_after();
+      if (EX && sink) l_run += hb_exp2(fmaf(sink[hq], 1.4426950408889634f, -m_run));
       const float inv = 1.f / l_run;
       __nv_bfloat16* dst = out + ((size_t)(row0 + r) * Hq + hq) * FT_D;
 #pragma unroll
@@ -338,12 +353,15 @@ HB_EXPORT int hb_flash_prefill_tc_supported(int Hq, int Hkv, int D, int page_siz
 HB_EXPORT int hb_flash_prefill_tc(const void* q, const void* kc, const void* vc, long num_pages, const int* bt, int bt_stride,
                                   const int* q_start, const int* q_len, const int* ctx_len, void* out, int T, int R,
                                   int max_q_len, int Hq, int Hkv, int D, int page_size, int window, float scale,
-                                  int min_rows, int* status, cudaStream_t st) {
+                                  int min_rows, int* status, const float* r1, const float* r2, const float* sink,
+                                  cudaStream_t st) {
   if (R <= 0 || max_q_len <= 0 || T <= 0) return 0;
   if (!hb_flash_prefill_tc_supported(Hq, Hkv, D, page_size))
     HB_FAIL("hb_flash_prefill_tc: %d/%d heads of %d with pages of %d are not supported", Hq, Hkv, D, page_size);
   if (R > 65535 || max_q_len > 65535 * FT_BM) HB_FAIL("hb_flash_prefill_tc: %d requests / portions of %d rows are beyond the grid limit", R, max_q_len);
   if (!status) HB_FAIL("hb_flash_prefill_tc: no status word");
+  const bool ex = r1 || sink;
+  if ((r1 != nullptr) != (r2 != nullptr) || (ex && window > 0)) HB_FAIL("hb_flash_prefill_tc: a distance bias needs both of its vectors, and no window");
   CUtensorMap mq, mk, mv;
   if (hb_make_tensor_map_bf16(&mq, q, (uint64_t)T, (uint64_t)Hq * D, (uint64_t)Hq * D, FT_BM)) return -1;
   const uint64_t rows = (uint64_t)num_pages * Hkv * page_size;
@@ -352,27 +370,24 @@ HB_EXPORT int hb_flash_prefill_tc(const void* q, const void* kc, const void* vc,
   dim3 grid(Hq, (max_q_len + FT_BM - 1) / FT_BM, R);
   const float sl2 = scale * 1.4426950408889634f;
   cudaError_t e;
-  if (D == 64) {
-    const size_t smem = 7 * (size_t)FT_TILE + sizeof(FtBars);   // 113 KB: two CTAs an SM
-    static bool configured = false;
-    if (!configured) {
-      e = cudaFuncSetAttribute(flash_prefill_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) HB_FAIL("hb_flash_prefill_tc: %s", cudaGetErrorString(e));
-      configured = true;
-    }
-    e = hb_launch(flash_prefill_tc_kernel<64>, grid, 192, smem, st, mq, mk, mv, bt, bt_stride, q_start, q_len, ctx_len,
-                  (__nv_bfloat16*)out, Hq, Hkv, page_size, window, sl2, min_rows, status);
-  } else {
-    const size_t smem = 12 * (size_t)FT_TILE + sizeof(FtBars);  // Q, 2 K, 2 V of 32 KB each and P: 192 KB
-    static bool configured = false;
-    if (!configured) {
-      e = cudaFuncSetAttribute(flash_prefill_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) HB_FAIL("hb_flash_prefill_tc: %s", cudaGetErrorString(e));
-      configured = true;
-    }
-    e = hb_launch(flash_prefill_tc_kernel<128>, grid, 192, smem, st, mq, mk, mv, bt, bt_stride, q_start, q_len, ctx_len,
-                  (__nv_bfloat16*)out, Hq, Hkv, page_size, window, sl2, min_rows, status);
-  }
+  // head_dim 64: 113 KB, two CTAs an SM; head_dim 128: Q, 2 K, 2 V of 32 KB each and P: 192 KB
+  const size_t smem = (D == 64 ? 7 : 12) * (size_t)FT_TILE + sizeof(FtBars);
+#define FT_LAUNCH(DD, EX)                                                                                                       \
+  do {                                                                                                                          \
+    static bool configured = false;                                                                                             \
+    if (!configured) {                                                                                                          \
+      e = cudaFuncSetAttribute(flash_prefill_tc_kernel<DD, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
+      if (e != cudaSuccess) HB_FAIL("hb_flash_prefill_tc: %s", cudaGetErrorString(e));                                          \
+      configured = true;                                                                                                        \
+    }                                                                                                                           \
+    e = hb_launch(flash_prefill_tc_kernel<DD, EX>, grid, 192, smem, st, mq, mk, mv, bt, bt_stride, q_start, q_len, ctx_len,     \
+                  (__nv_bfloat16*)out, Hq, Hkv, page_size, window, sl2, min_rows, status, r1, r2, sink);                        \
+  } while (0)
+  if (D == 64 && !ex) FT_LAUNCH(64, false);
+  else if (D == 64) FT_LAUNCH(64, true);
+  else if (!ex) FT_LAUNCH(128, false);
+  else FT_LAUNCH(128, true);
+#undef FT_LAUNCH
   if (e != cudaSuccess) HB_FAIL("hb_flash_prefill_tc: %s", cudaGetErrorString(e));
   HB_CHECK_LAUNCH("hb_flash_prefill_tc");
   return 0;

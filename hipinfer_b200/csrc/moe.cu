@@ -28,93 +28,104 @@
 //   moe_combine_kernel      out[t] += sum over the choices, in their order, of the sorted results
 #include "common.cuh"
 
-constexpr int MR_THREADS = 128;
+constexpr int MR_THREADS = 512;
 
+// A warp a router row (and the shared expert's gate), the token's row read beside it; then warp 0 ranks the groups, marks the
+// experts of those that do not stay as taken (NaN), and picks the largest `top` times, ties to the lower index.
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restrict__ xn, long ldx, const TW* __restrict__ router,
                                                                const TW* __restrict__ bias, int* __restrict__ expert,
                                                                float* __restrict__ weight, int W, int E, int top, int mode,
                                                                const TW* __restrict__ correction, int groups, int keep, float scale,
-                                                               const TW* __restrict__ shared_gate, float* __restrict__ shared_weight) {
-  extern __shared__ float mr_sm[];     // [W] the row, [E] the scores, (mode 2) [E] the scores without the correction
-  float* row = mr_sm;
-  float* sc = mr_sm + W;
+                                                               const TW* __restrict__ shared_gate, float* __restrict__ shared_weight,
+                                                               int vec) {
+  extern __shared__ float mr_sm[];     // [E] the scores, [E] those without the correction, [groups] the groups' sums
+  float* sc = mr_sm;
   float* plain = sc + E;
+  float* gs = plain + E;
   hb_pdl_launch();
   hb_pdl_wait();
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int i = threadIdx.x; i < W; i += MR_THREADS) row[i] = hb_to_float(xn[(size_t)t * ldx + i]);
-  __syncthreads();
-  for (int e = warp; e < E + (shared_gate ? 1 : 0); e += MR_THREADS / 32) {
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const TA* row = xn + (size_t)t * ldx;
+  for (int e = warp; e < E + (shared_gate ? 1 : 0); e += nw) {
     const TW* wr = e < E ? router + (size_t)e * W : shared_gate;
     float acc = 0.f;
-    for (int i = lane; i < W; i += 32) acc = fmaf(row[i], hb_to_float(wr[i]), acc);
+    if (vec) {
+#pragma unroll 8
+      for (int i = lane * 4; i < W; i += 128) {
+        const float4 wv = hb_load4(wr + i), av = hb_load4(row + i);
+        acc = fmaf(wv.x, av.x, acc);
+        acc = fmaf(wv.y, av.y, acc);
+        acc = fmaf(wv.z, av.z, acc);
+        acc = fmaf(wv.w, av.w, acc);
+      }
+    } else {
+      for (int i = lane; i < W; i += 32) acc = fmaf(hb_to_float(row[i]), hb_to_float(wr[i]), acc);
+    }
     acc = hb_warp_sum(acc);
+    if (lane != 0) continue;
     if (e == E) {
-      if (lane == 0) shared_weight[t] = 1.f / (1.f + expf(-acc));
+      shared_weight[t] = 1.f / (1.f + expf(-acc));
       continue;
     }
     if (bias) acc += hb_to_float(bias[e]);
-    if (lane == 0) {
-      const float v = mode == 1 ? acc : 1.f / (1.f + expf(-acc));
-      sc[e] = mode == 2 ? v + hb_to_float(correction[e]) : v;
-      if (mode == 2) plain[e] = v;
-    }
+    const float v = mode == 1 ? acc : 1.f / (1.f + expf(-acc));
+    sc[e] = mode == 2 ? v + hb_to_float(correction[e]) : v;
+    plain[e] = v;
   }
   __syncthreads();
-  if (mode == 2 && groups > 1 && threadIdx.x == 0) {
-    // the groups that do not stay are marked as taken, the worst group first (ties: the higher index goes first)
+  if (warp != 0) return;
+  if (mode == 2 && groups > 1) {
     const int span = E / groups;
-    for (int gone = 0; gone < groups - keep; gone++) {
-      int worst = -1;
-      float ws = 0.f;
-      for (int q = 0; q < groups; q++) {
-        if (sc[q * span] != sc[q * span]) continue;
-        float a = -INFINITY, b = -INFINITY;            // the two largest
-        for (int e = q * span; e < (q + 1) * span; e++) {
-          const float v = sc[e];
-          if (v > a) { b = a; a = v; } else if (v > b) b = v;
-        }
-        const float v = span > 1 ? a + b : a;
-        if (worst < 0 || v <= ws) { worst = q; ws = v; }
-      }
-      if (worst < 0) break;
-      for (int e = worst * span; e < (worst + 1) * span; e++) sc[e] = __int_as_float(0x7fc00000);
-    }
-  }
-  if (threadIdx.x == 0) {
-    float first = 0.f, den = 0.f;
-    for (int k = 0; k < top; k++) {
-      int best = -1;
-      float bs = 0.f;
-      for (int e = 0; e < E; e++) {
+    for (int q = lane; q < groups; q += 32) {
+      float a = -INFINITY, b = -INFINITY;                  // the two largest
+      for (int e = q * span; e < (q + 1) * span; e++) {
         const float v = sc[e];
-        if (v != v) continue;          // NaN marks an expert that is taken
-        if (best < 0 || v > bs) {
-          bs = v;
-          best = e;
-        }
+        if (v > a) { b = a; a = v; } else if (v > b) b = v;
       }
-      if (best < 0) best = 0;          // every score NaN (bad weights or input): stay inside the tables
+      gs[q] = span > 1 ? a + b : a;
+    }
+    __syncwarp();
+    for (int q = lane; q < groups; q += 32) {
+      const float v = gs[q];
+      int ahead = 0;
+      for (int p = 0; p < groups; p++) ahead += gs[p] > v || (gs[p] == v && p < q);
+      if (ahead >= keep)
+        for (int e = q * span; e < (q + 1) * span; e++) sc[e] = __int_as_float(0x7fc00000);
+    }
+    __syncwarp();
+  }
+  float first = 0.f, den = 0.f;
+  for (int k = 0; k < top; k++) {
+    float bs = -INFINITY;
+    int best = E;
+    for (int e = lane; e < E; e += 32) {
+      const float v = sc[e];
+      if (v == v && (best == E || v > bs)) { bs = v; best = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bs, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best, o);
+      if (oe < E && (best == E || ov > bs || (ov == bs && oe < best))) { bs = ov; best = oe; }
+    }
+    if (best == E) best = 0;             // every score NaN (bad weights or input): stay inside the tables
+    // softmax over the chosen logits alone (mode 1): the first chosen one is the largest
+    if (k == 0) first = bs;
+    const float w = mode == 1 ? expf(bs - first) : plain[best];
+    den += w;
+    if (lane == 0) {
       expert[(size_t)t * top + k] = best;
-      if (mode == 0) weight[(size_t)t * top + k] = bs;
-      else if (mode == 2) {
-        weight[(size_t)t * top + k] = plain[best];
-        den += plain[best];
-      } else {
-        // softmax over the chosen logits alone: the first chosen one is the largest
-        if (k == 0) first = bs;
-        const float ex = expf(bs - first);
-        weight[(size_t)t * top + k] = ex;
-        den += ex;
-      }
+      weight[(size_t)t * top + k] = w;
       sc[best] = __int_as_float(0x7fc00000);
     }
-    if (mode == 1)
-      for (int k = 0; k < top; k++) weight[(size_t)t * top + k] /= den;
-    if (mode == 2)
-      for (int k = 0; k < top; k++) weight[(size_t)t * top + k] = weight[(size_t)t * top + k] / (den + 1e-20f) * scale;
+    __syncwarp();
   }
+  if (mode != 0 && lane == 0)
+    for (int k = 0; k < top; k++) {
+      const float w = weight[(size_t)t * top + k];
+      weight[(size_t)t * top + k] = mode == 1 ? w / den : w / (den + 1e-20f) * scale;
+    }
 }
 
 // mode 0: the scores are sigmoid(z) and the chosen scores are the weights; mode 1: the largest logits z choose and the
@@ -130,13 +141,15 @@ HB_EXPORT int hb_moe_route(const void* xn, int x_dt, long ldx, const void* route
     HB_FAIL("hb_moe_route: %d experts in %d groups of which %d stay, %d chosen", E, groups, keep, top);
   if (shared_gate && !shared_weight) HB_FAIL("hb_moe_route: a shared expert's gate needs a place for its result");
   if (top < 1 || top > E) HB_FAIL("hb_moe_route: top %d of %d experts", top, E);
-  const size_t smem = (size_t)(W + 2 * E) * sizeof(float);
-  if (smem > 200 * 1024) HB_FAIL("hb_moe_route: a row of %d with %d experts does not fit shared memory", W, E);
+  const size_t smem = (size_t)(2 * E + groups) * sizeof(float);
+  const int vec = W % 4 == 0 && ldx % 4 == 0 && !(((uintptr_t)router | (uintptr_t)shared_gate | (uintptr_t)xn) & 15);
+  const int rows = E + (shared_gate ? 1 : 0), threads = 32 * (rows < MR_THREADS / 32 ? rows : MR_THREADS / 32);
+  if (smem > 200 * 1024) HB_FAIL("hb_moe_route: %d experts in %d groups do not fit shared memory", E, groups);
   HB_DISPATCH_2(x_dt, w_dt, "hb_moe_route", do {
     auto kern = moe_route_kernel<TA, TB>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(kern, dim3(T), dim3(MR_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert, weight,
-              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight);
+    hb_launch(kern, dim3(T), dim3(threads), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert, weight,
+              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight, vec);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_route");
   return 0;

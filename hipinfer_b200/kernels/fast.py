@@ -24,10 +24,10 @@ _SIGS = {
     "hb_gemm_stream_finish": [_p, _p, _l, _i, _i, _i, _i, _p],
     "hb_add_rmsnorm_slices": [_p, _l, _p, _i, _l, _l, _p, _p, _p, _i, _i, _f, _p],
     "hb_rope_kv_slices": [_p, _i, _l, _l, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p],
-    "hb_attn_decode": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _i, _p, _p, _p],
+    "hb_attn_decode": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _i, _p, _p, _p, _p, _p, _p],
     "hb_flash_prefill": [_p, _p, _p, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p],
     "hb_flash_prefill_supported": [_i, _i, _i],
-    "hb_flash_prefill_tc": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p],
+    "hb_flash_prefill_tc": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p, _p, _p],
     "hb_flash_prefill_tc_supported": [_i, _i, _i, _i],
     "hb_gemm_tc_rope_kv": [_p, _l, _p, _l, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
     "hb_attn_decode_supported": [_i, _i, _i],
@@ -443,13 +443,15 @@ def _decode_counters(device, n):
 
 
 def attention_decode(q, k_cache, v_cache, block_table, row_request, positions, out, n_heads, n_kv_heads, head_dim,
-                     page_size, window, scale, max_pos, chunk=None, q_len=None, row_limit=0, ctx_len=None):
+                     page_size, window, scale, max_pos, chunk=None, q_len=None, row_limit=0, ctx_len=None, distance=None,
+                     sink=None):
     """The bf16 row-attention kernel itself (see csrc/attention_fast.cu); rows whose keys span several
     chunks are finished inside it. With q_len (int32 per request) rows of requests with row_limit
     rows or more are skipped. row_request None: row t is the only row of request t (a decode-only
     step). ctx_len (int32 per request): the tokens in the cache before this
     step; with it the kernel asks for their keys before the kernel ahead of it has ended, so
-    positions, tables and ctx_len must then be in place before that kernel starts."""
+    positions, tables and ctx_len must then be in place before that kernel starts. distance (an ops.DistanceBias) and sink
+    (float32 [n_heads]) as in ops.attention_masked."""
     from . import ops
 
     T = q.shape[0]
@@ -461,7 +463,7 @@ def attention_decode(q, k_cache, v_cache, block_table, row_request, positions, o
           None if ws is None else ws.data_ptr(), None if cnt is None else cnt.data_ptr(), T, n_heads, n_kv_heads,
           head_dim, page_size, int(window), float(scale), chunk, int(max_pos),
           None if q_len is None else q_len.data_ptr(), int(row_limit), None if ctx_len is None else ctx_len.data_ptr(),
-          status_word().data_ptr(), _stream())
+          status_word().data_ptr(), *_extras(distance, sink), _stream())
     return out
 
 
@@ -491,19 +493,35 @@ def flash_prefill_tc_supported(n_heads, n_kv_heads, head_dim, page_size) -> bool
 
 
 def flash_prefill_tc(q, k_cache, v_cache, block_table, q_start, q_len, ctx_len, out, max_q_len, n_heads, n_kv_heads,
-                     head_dim, page_size, window, scale, min_rows=1):
+                     head_dim, page_size, window, scale, min_rows=1, distance=None, sink=None):
     """The tcgen05 flash kernel for prompt portions (see csrc/attention_prefill_tc.cu); arguments as flash_prefill."""
     _call("hb_flash_prefill_tc", q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[0],
           block_table.data_ptr(), block_table.stride(0), q_start.data_ptr(), q_len.data_ptr(), ctx_len.data_ptr(),
           out.data_ptr(), q.shape[0], q_len.numel(), int(max_q_len), n_heads, n_kv_heads, head_dim, page_size, int(window),
-          float(scale), int(min_rows), status_word().data_ptr(), _stream())
+          float(scale), int(min_rows), status_word().data_ptr(), *_extras(distance, sink), _stream())
     return out
 
 
 FLASH_MIN_ROWS = 16     # portions of at least this many rows go to the flash kernel, shorter ones to the row kernel
 
 
-def attention(q, k_cache, v_cache, batch, group, out, n_heads, n_kv_heads, head_dim, page_size, window, scale) -> bool:
+def _extras(distance, sink):
+    return (None if distance is None else distance.r1.data_ptr(), None if distance is None else distance.r2.data_ptr(),
+            None if sink is None else sink.data_ptr())
+
+
+def attention_extras_ok(distance, sink, n_heads, n_kv_heads, head_dim, page_size) -> bool:
+    """Whether `attention` takes a distance bias and a sink at these sizes: pages the TMA kernels read whole, and a bias that
+    falls with the distance and spreads little enough within a key tile for its bound to stand in for the maximum."""
+    return ((distance is None or distance.spread <= 60.0) and page_size >= 8 and page_size <= (64 if head_dim == 64 else 32)
+            and flash_prefill_tc_supported(n_heads, n_kv_heads, head_dim, page_size))
+
+
+def attention(q, k_cache, v_cache, batch, group, out, n_heads, n_kv_heads, head_dim, page_size, window, scale, distance=None,
+              sink=None) -> bool:
+    if (distance is not None or sink is not None) and (window or not attention_extras_ok(distance, sink, n_heads, n_kv_heads, head_dim,
+                                                                                        page_size)):
+        return False
     if PLAIN_ONLY or q.dtype != torch.bfloat16 or not attention_decode_supported(n_heads, n_kv_heads, head_dim):
         return False
     use_flash = flash_prefill_supported(n_heads, n_kv_heads, head_dim) and batch.max_q_len >= FLASH_MIN_ROWS
@@ -511,14 +529,15 @@ def attention(q, k_cache, v_cache, batch, group, out, n_heads, n_kv_heads, head_
     bt = batch.block_tables[group]
     if use_flash:
         tc = flash_prefill_tc_supported(n_heads, n_kv_heads, head_dim, page_size)    # else: warp MMAs (other page sizes)
+        kw = dict(distance=distance, sink=sink) if tc else {}
         (flash_prefill_tc if tc else flash_prefill)(q, k_cache, v_cache, bt, batch.req_q_start, batch.req_q_len,
                                                     batch.req_ctx_len, out, batch.max_q_len, n_heads, n_kv_heads,
-                                                    head_dim, page_size, window, scale, FLASH_MIN_ROWS)
+                                                    head_dim, page_size, window, scale, FLASH_MIN_ROWS, **kw)
     if need_rows:
         # a step of single decode rows: row t is request t, which the kernel need not look up
         rows_are_requests = batch.max_q_len == 1 and batch.n_rows == batch.n_requests
         attention_decode(q, k_cache, v_cache, bt, None if rows_are_requests else batch.row_request, batch.positions, out, n_heads, n_kv_heads,
                          head_dim, page_size, window, scale, batch.max_pos,
                          q_len=batch.req_q_len if use_flash else None, row_limit=FLASH_MIN_ROWS,
-                         ctx_len=batch.req_ctx_len)
+                         ctx_len=batch.req_ctx_len, distance=distance, sink=sink)
     return True

@@ -14,6 +14,9 @@ scripts/bench.py:126-212, and reports GB/s or TFLOP/s from algorithmic bytes and
     python -m hipinfer_b200.kernels.microbench selective_scan --tokens 2048 --batch 1 --n 2048 --states 16   (a prompt portion)
     python -m hipinfer_b200.kernels.microbench selective_scan --tokens 1 --batch 64 --n 2048 --states 16     (single rows)
     python -m hipinfer_b200.kernels.microbench residual_norm --m 2048 --n 2048 [--pair]
+    python -m hipinfer_b200.kernels.microbench matrix_memory|gated_delta --tokens 2048 --batch 1 --heads 32 --head-dim 64  (the walk of a portion)
+    python -m hipinfer_b200.kernels.microbench matrix_memory|gated_delta --tokens 1 --batch 64   (single tokens: the whole mixer's kernel)
+    python -m hipinfer_b200.kernels.microbench output_norm --m 2048 --n 2048 --states 9          (states of the depth average)
 
 Between timed launches of kernels whose inputs fit in L2 a buffer larger than L2 is written
 (`--flush`, on by default) so that the figures are for operands coming from HBM.
@@ -64,7 +67,8 @@ def _prepared(fast, x, nw):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
     ap.add_argument("kernel", choices=["gemm_tc", "gemm_stream", "rows_add", "rows_swiglu", "rows_qkv", "attn_decode", "flash_prefill", "flash_prefill_tc", "rmsnorm",
-                                       "delta_rule", "attn_window", "layernorm", "polynorm", "scale_add", "selective_scan", "residual_norm"])
+                                       "delta_rule", "attn_window", "layernorm", "polynorm", "scale_add", "selective_scan", "residual_norm",
+                                       "matrix_memory", "gated_delta", "output_norm"])
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=16384)
     ap.add_argument("--k", type=int, default=2048)
@@ -114,6 +118,41 @@ def main(argv=None) -> int:
         nbytes = T * (I * 4 * (5 if pieces else 3) + 2 * N * 4 * (1.5 if pieces else 1) + I * 2) + 2 * R * I * N * 4
         out.update(requests=R, tokens=L, channels=I, states=N, pieces=bool(pieces), ms=ms, gbs=nbytes / ms / 1e6,
                    us_per_token=ms * 1e3 / L)
+    elif a.kernel in ("matrix_memory", "gated_delta"):
+        from types import SimpleNamespace
+
+        R, L, H, D, delta = a.batch, a.tokens, a.heads, a.head_dim, a.kernel == "gated_delta"
+        T = R * L
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        q, k, v, gate = (rnd(T, H * D) for _ in range(4))
+        dec, add = torch.rand(T, H, generator=g, device=dev) * 0.1 + 0.9, torch.rand(T, H, generator=g, device=dev)
+        state, y = torch.zeros(R, H, D, D, device=dev), torch.empty(T, H * D, device=dev)
+        ns, ms, nq = (torch.zeros(*s, device=dev) for s in ((R, H, D), (R, H), (T, H)))
+        batch = SimpleNamespace(n_requests=R, max_q_len=L, req_q_start=i32([r * L for r in range(R)]), req_q_len=i32([L] * R),
+                                req_state_slot=i32(list(range(R))), row_request=i32([r for r in range(R) for _ in range(L)]))
+        if L == 1:
+            vec, nw = rnd(H).bfloat16(), torch.ones(D if delta else H * D, device=dev).bfloat16()
+            out16 = torch.empty(T, H * D, dtype=torch.bfloat16, device=dev)
+            fn = lambda: ops.ms_single(q, k, v, dec, add, vec, vec, state, nw, gate, "silu" if delta else "sigmoid", out16, batch, D ** -0.5, 1e-5,
+                                       None if delta else ns, None if delta else ms, 15.0, 1e-6, 1e-6)
+            nbytes = R * H * (2 * D * D * 4 + 4 * D * 4 + 2 * D + (0 if delta else 8 * D))
+        else:
+            vec = torch.zeros(H, device=dev)
+            scal = ops.ms_delta_prepare(q, k, dec * -6.0, add, vec, vec, batch, D, D ** -0.5, 1e-6) if delta else None
+            fn = ((lambda: ops.ms_delta_walk(q, k, v, scal, state, batch, y)) if delta
+                  else lambda: ops.ms_walk(q, k, v, dec, add, state, batch, y, D ** -0.5, ns, nq))
+            pieces = not delta and L >= 3 * ops.MS_PIECE_TOKENS > 0
+            nbytes = T * H * D * 4 * (6 if pieces else 4) + 2 * R * H * D * D * 4
+        ms_ = timeit(fn, a.iters, a.flush)
+        out.update(requests=R, tokens=L, heads=H, head_dim=D, ms=ms_, gbs=nbytes / ms_ / 1e6, us_per_token=ms_ * 1e3 / L)
+    elif a.kernel == "output_norm":
+        M, W, n = a.m, a.n, a.states
+        x, y, states, coef = rnd(M, W), rnd(M, W), rnd(n + 1, M, W), rnd(n + 1)
+        w, b = torch.ones(W, device=dev).bfloat16(), torch.zeros(W, device=dev).bfloat16()
+        rounded = torch.empty(M, W, dtype=torch.bfloat16, device=dev)
+        fn = lambda: ops.output_norm(x, y, w, b, 1e-5, rounded, None, states[n], states[:n] if n else None, coef if n else None)
+        ms = timeit(fn, a.iters, a.flush)
+        out.update(m=M, n=W, states=n, ms=ms, gbs=M * W * (4 * (n + 4) + 2) / ms / 1e6)
     elif a.kernel == "residual_norm":
         M, W = a.m, a.n
         x, y, w = rnd(M, W), rnd(M, W), 1 + 0.1 * rnd(W)

@@ -81,10 +81,14 @@ _SIGS = {
         "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p],
     },
     "memory": {
-        "hb_ms_walk": [_p, _l, _p, _l, _p, _l, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _i, _p, _p, _p, _p],
+        "hb_ms_walk": [_p, _l, _p, _l, _p, _l, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p],
+        "hb_ms_delta_walk": [_p, _l, _p, _l, _p, _l, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p],
         "hb_ms_exp_gates": [_p, _p, _l, _p, _p, _i, _f, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _p],
-        "hb_ms_delta_prepare": [_p, _l, _i, _i, _p, _p, _l, _p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _p],
+        "hb_ms_delta_prepare": [_p, _p, _l, _p, _p, _l, _p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _p],
         "hb_ms_finish": [_p, _p, _p, _f, _p, _i, _i, _p, _l, _i, _p, _i, _l, _i, _i, _i, _f, _p],
+        "hb_ms_single_supported": [_i, _i, _i],
+        "hb_ms_single": [_p, _l, _p, _l, _p, _l, _p, _p, _l, _p, _p, _i, _f, _f, _f, _f, _f, _p, _p, _p, _p, _p, _p, _p, _i, _i, _p, _l, _i, _p,
+                         _i, _l, _i, _i, _i, _i, _i, _i, _p],
         "hb_output_norm": [_p, _p, _p, _f, _f, _p, _p, _i, _f, _i, _p, _p, _i, _p, _p, _p, _l, _p, _i, _i, _i, _p],
     },
     "mixers": {
@@ -876,6 +880,18 @@ def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_m
     return q_out
 
 
+class DistanceBias:
+    """A bias that falls with the distance, r1_h ln(1 + r2_h (i - j)) off the score of query i and key j: r1, r2 float32
+    [n_heads] on the device. `spread`: how far it falls within 128 positions, in units of log 2 (inf where a number is
+    negative)."""
+    __slots__ = ("r1", "r2", "spread")
+
+    def __init__(self, r1, r2):
+        self.r1, self.r2 = r1.to(torch.float32).contiguous(), r2.to(torch.float32).contiguous()
+        low = min(float(self.r1.min()), float(self.r2.min()))
+        self.spread = float((self.r1 * torch.log2(1.0 + 127.0 * self.r2.clamp(min=0.0))).max()) if low >= 0 else float("inf")
+
+
 MASKS = {"causal": 0, "window": 1, "chunk": 2}
 MASKED_FLASH_MIN_ROWS = 16
 
@@ -892,9 +908,11 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
     the values are then its first `vdim` columns). mask "causal", "window" (the last `window` keys and the first
     `keep_first`) or "chunk" (the keys of the row's own chunk of `chunk` positions). sink: float32 [n_heads], joins the
     softmax's denominator as exp(sink). gate: float32 [T, *], sigmoid(gate[:, gate_offset + ...]) multiplies the result,
-    one number per element or, with gate_per_head, one per head. out may be float32 beside bfloat16 q. distance (r1, r2),
-    float32 [n_heads] each: r1 ln(1 + r2 (i - j)) is taken off the score of query i and key j."""
-    r1, r2 = distance if distance is not None else (None, None)
+    one number per element or, with gate_per_head, one per head. out may be float32 beside bfloat16 q. distance (a
+    DistanceBias): r1 ln(1 + r2 (i - j)) is taken off the score of query i and key j.
+
+    Causal attention without a gate over keys and values of 64 or 128 goes to the TMA and tcgen05 kernels of `attention`."""
+    r1, r2 = (distance.r1, distance.r2) if distance is not None else (None, None)
     _need_cuda(r1, r2)
     for r in (r1, r2):
         assert r is None or (r.dtype == torch.float32 and r.numel() == n_heads and r.is_contiguous())
@@ -920,6 +938,11 @@ def attention_masked(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
     from . import fast
 
     kw, vw = k_cache.shape[-1], v_cache.shape[-1]
+    if (mask == "causal" and gate is None and v_cache is not k_cache and dim == vdim == kw == vw and not force_rows and not force_plain
+            and not row_limit and q.dtype == out.dtype == torch.bfloat16 and q.is_contiguous() and out.is_contiguous()
+            and hasattr(batch, "h_q_len")
+            and fast.attention(q, k_cache, v_cache, batch, group, out, n_heads, n_kv_heads, dim, page_size, 0, scale, distance, sink)):
+        return out
     flash = (q.dtype == torch.bfloat16 and not fast.PLAIN_ONLY and not force_rows and not force_plain and v_cache is not k_cache
              and getattr(batch, "max_q_len", 0) >= MASKED_FLASH_MIN_ROWS and masked_flash_supported(dim, vdim)
              and kw % 8 == 0 and vw % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0)
@@ -1426,41 +1449,76 @@ def moe_combine(ys: torch.Tensor, pos: torch.Tensor, y: torch.Tensor, top: int) 
 MS_PIECE_TOKENS = 64    # tokens a piece of the linear recurrence (ms_walk); 0: always one walk a request
 
 
-def ms_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, state: torch.Tensor, batch,
-            y: torch.Tensor, q_scale: float = 1.0, kq: Optional[torch.Tensor] = None, nstate: Optional[torch.Tensor] = None,
-            nq: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """The walk of a recurrence with one state matrix per head over the step's rows, request by request, from and into each
-    request's state slot. q, k float32 [T, groups * N], v float32 [T, heads * P] (views of wider rows are fine); a, b float32
-    [T, heads]; state float32 [slots, heads, N, P]; y float32 [T, heads * P].
-
-    Without kq: S <- a S + b k v^T, y = S^T q * q_scale and, with nstate [slots, heads, N], n <- a n + b k,
-    nq [T, heads] = n . q * q_scale. With kq float32 [T, groups] (k . q of the rows): the delta rule,
-    S <- a S; u = b (v - S^T k); S <- S + k u^T; y = S^T q * q_scale.
-
-    A step of the first form whose longest portion has at least three times MS_PIECE_TOKENS rows runs in pieces of that
-    many tokens; the results differ from the walk in one go by rounding only."""
-    _need_cuda(q, k, v, a, b, state, y, kq, nstate, nq)
+def _ms_rows(q, k, v, state, y):
     for t, what in ((q, "q"), (k, "k"), (v, "v")):
         _rows_contiguous(t, "ms_walk " + what)
-    T, H = a.shape
-    slots, Hs, N, P = state.shape
-    G = q.shape[1] // N
-    assert Hs == H and q.shape == k.shape == (T, G * N) and v.shape == (T, H * P) and y.shape == (T, H * P)
-    assert all(t.dtype == torch.float32 for t in (q, k, v, a, b, state, y)) and all(t.is_contiguous() for t in (a, b, state, y))
-    assert b.shape == (T, H) and (kq is None or (kq.shape == (T, G) and kq.is_contiguous() and kq.dtype == torch.float32))
+    slots, H, N, P = state.shape
+    T, G = q.shape[0], q.shape[1] // N
+    assert q.shape == k.shape == (T, G * N) and v.shape == y.shape == (T, H * P)
+    assert all(t.dtype == torch.float32 for t in (q, k, v, state, y)) and state.is_contiguous() and y.is_contiguous()
+    return T, H, G, N, P
+
+
+def ms_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, state: torch.Tensor, batch,
+            y: torch.Tensor, q_scale: float = 1.0, nstate: Optional[torch.Tensor] = None, nq: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The walk of a linear recurrence with one state matrix per head over the step's rows, request by request, from and into
+    each request's state slot: S <- a S + b k v^T, y = S^T q * q_scale and, with nstate [slots, heads, N], n <- a n + b k,
+    nq [T, heads] = n . q * q_scale. q, k float32 [T, groups * N], v float32 [T, heads * P] (views of wider rows are fine);
+    a, b float32 [T, heads]; state float32 [slots, heads, N, P]; y float32 [T, heads * P].
+
+    A step whose longest portion has at least three times MS_PIECE_TOKENS rows runs in pieces of that many tokens; the
+    results differ from the walk in one go by rounding only."""
+    _need_cuda(q, k, v, a, b, state, y, nstate, nq)
+    T, H, G, N, P = _ms_rows(q, k, v, state, y)
+    assert a.shape == b.shape == (T, H) and a.dtype == b.dtype == torch.float32 and a.is_contiguous() and b.is_contiguous()
     if nstate is not None:
-        assert nstate.shape == (slots, H, N) and nstate.is_contiguous() and nq.shape == (T, H) and nq.is_contiguous()
+        assert nstate.shape == (state.shape[0], H, N) and nstate.is_contiguous() and nq.shape == (T, H) and nq.is_contiguous()
     L, pieces, ps, pn, pd = int(MS_PIECE_TOKENS), 0, None, None, None
-    if kq is None and L > 0 and batch.max_q_len >= 3 * L:
+    if L > 0 and batch.max_q_len >= 3 * L:
         pieces = -(-batch.max_q_len // L)
         room = T // L + batch.n_requests               # every request ends with at most one short piece
         ps = torch.empty(room, H, N, P, dtype=torch.float32, device=q.device)
         pn = torch.empty(room, H, N, dtype=torch.float32, device=q.device) if nstate is not None else None
         pd = torch.empty(room, H, dtype=torch.float32, device=q.device)
     _call("memory", "hb_ms_walk", q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), a.data_ptr(),
-          b.data_ptr(), _ptr(kq), state.data_ptr(), _ptr(nstate), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(),
-          batch.req_state_slot.data_ptr(), y.data_ptr(), _ptr(nq), batch.n_requests, H, G, N, P, float(q_scale),
-          0 if kq is None else 1, L, pieces, _ptr(ps), _ptr(pn), _ptr(pd), _stream())
+          b.data_ptr(), state.data_ptr(), _ptr(nstate), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(),
+          batch.req_state_slot.data_ptr(), y.data_ptr(), _ptr(nq), batch.n_requests, H, G, N, P, float(q_scale), L, pieces, _ptr(ps),
+          _ptr(pn), _ptr(pd), _stream())
+    return y
+
+
+MS_SCAL = 12     # numbers per (token, head) that the delta rule's walk reads beside its rows (csrc/matrix_state.cu)
+
+
+def ms_delta_prepare(q: torch.Tensor, k: torch.Tensor, za: torch.Tensor, zb: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                     batch, dim: int, q_scale: float, unit_eps: float) -> torch.Tensor:
+    """float32 [T, heads, MS_SCAL]: what ms_delta_walk reads of a token beside its rows. q, k float32 [T, groups * dim] raw (views
+    of the same wider rows): the factors that make each head's q and k x / sqrt(sum x^2 + unit_eps) (q also times q_scale) and
+    products of neighbouring tokens' keys and queries; za, zb float32 [T, heads] (views of the same rows): the decay
+    exp(-exp(a_log) softplus(za + dt_bias)) and the write strength sigmoid(zb)."""
+    _need_cuda(q, k, za, zb, a_log, dt_bias)
+    T, H = za.shape
+    assert q.dtype == k.dtype == za.dtype == zb.dtype == torch.float32 and za.stride() == zb.stride() and za.stride(1) == 1
+    assert q.shape == k.shape and q.stride() == k.stride() and q.stride(1) == 1 and q.shape[1] % dim == 0
+    assert a_log.dtype == dt_bias.dtype and a_log.numel() == dt_bias.numel() == H
+    scal = torch.empty(T, H, MS_SCAL, dtype=torch.float32, device=q.device)
+    _call("memory", "hb_ms_delta_prepare", q.data_ptr(), k.data_ptr(), q.stride(0), za.data_ptr(), zb.data_ptr(), za.stride(0),
+          a_log.data_ptr(), dt_bias.data_ptr(), _dt(a_log), batch.row_request.data_ptr(), batch.req_q_start.data_ptr(), scal.data_ptr(), T, H,
+          q.shape[1] // dim, int(dim), float(q_scale), float(unit_eps), _stream())
+    return scal
+
+
+def ms_delta_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scal: torch.Tensor, state: torch.Tensor, batch,
+                  y: torch.Tensor) -> torch.Tensor:
+    """The gated delta rule over the step's rows, request by request, from and into each request's state slot, four tokens at a
+    time: S <- a S; u = b (v - S^T k^); S <- S + k^ u^T; y = S^T q^, with k^, q^ the unit rows (q^ scaled) and a, b in `scal` from
+    ms_delta_prepare over the same raw rows. Shapes as in ms_walk."""
+    _need_cuda(q, k, v, scal, state, y)
+    T, H, G, N, P = _ms_rows(q, k, v, state, y)
+    assert scal.shape == (T, H, MS_SCAL) and scal.is_contiguous() and scal.dtype == torch.float32
+    _call("memory", "hb_ms_delta_walk", q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), scal.data_ptr(),
+          state.data_ptr(), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_state_slot.data_ptr(), y.data_ptr(),
+          batch.n_requests, H, G, N, P, _stream())
     return y
 
 
@@ -1478,24 +1536,6 @@ def ms_exp_gates(zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch
           m_state.data_ptr(), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_state_slot.data_ptr(), a.data_ptr(),
           b.data_ptr(), e.data_ptr(), batch.n_requests, batch.max_q_len, H, _stream())
     return a, b, e
-
-
-def ms_delta_prepare(qkv: torch.Tensor, offsets, za: torch.Tensor, zb: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
-                     groups: int, dim: int, q_scale: float, unit_eps: float):
-    """Rows qkv float32 [T, *] with q and k [groups * dim] at the column `offsets` (q, k): every head's q and k become
-    x / sqrt(sum x^2 + unit_eps), q also times q_scale, in place. Returns (a, b, kq): a = exp(-exp(a_log) softplus(za +
-    dt_bias)) and b = sigmoid(zb), float32 [T, heads], and kq = k . q, float32 [T, groups]. za, zb: views of the same rows."""
-    _need_cuda(qkv, za, zb, a_log, dt_bias)
-    _rows_contiguous(qkv, "ms_delta_prepare qkv")
-    T, H = za.shape
-    assert qkv.dtype == za.dtype == zb.dtype == torch.float32 and za.stride() == zb.stride() and za.stride(1) == 1
-    assert a_log.dtype == dt_bias.dtype and a_log.numel() == dt_bias.numel() == H
-    a, b = (torch.empty(T, H, dtype=torch.float32, device=za.device) for _ in range(2))
-    kq = torch.empty(T, groups, dtype=torch.float32, device=za.device)
-    _call("memory", "hb_ms_delta_prepare", qkv.data_ptr(), qkv.stride(0), int(offsets[0]), int(offsets[1]), za.data_ptr(), zb.data_ptr(),
-          za.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), _dt(a_log), kq.data_ptr(), a.data_ptr(), b.data_ptr(), T, H, int(groups),
-          int(dim), float(q_scale), float(unit_eps), _stream())
-    return a, b, kq
 
 
 GATE_KINDS = {"sigmoid": 0, "silu": 1}
@@ -1518,6 +1558,33 @@ def ms_finish(y: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, gate_ki
           1 if weight.numel() == P else 0, gate.data_ptr(), gate.stride(0), GATE_KINDS[gate_kind], out.data_ptr(), _dt(out), out.stride(0),
           T, heads, P, float(eps), _stream())
     return out
+
+
+def ms_single(q, k, v, z1, z2, w1, w2, state, weight, gate, gate_kind: str, out, batch, q_scale: float, eps: float, nstate=None,
+              m_state=None, cap: float = 0.0, den_eps: float = 0.0, unit_eps: float = 0.0) -> bool:
+    """For a step of single tokens (every request brings one): the whole mixer between its projections and its output product
+    in one kernel. With nstate and m_state the matrix memory (z1, z2, w1, w2: input and forget gates and their biases; cap,
+    den_eps), else the gated delta rule (z1, z2: the decay's and the write strength's pre-activations, w1: dt_bias, w2: A_log;
+    q, k raw, unit_eps); the rest as in ms_exp_gates / ms_delta_prepare, ms_walk and ms_finish. False: nothing was done."""
+    slots, H, N, P = state.shape
+    delta = nstate is None
+    if (getattr(batch, "max_q_len", 0) != 1 or _fn("memory", "hb_ms_single_supported")(N, P, 1 if delta else 0) != 1
+            or w1.dtype != weight.dtype or v.stride(0) % 4 or v.data_ptr() % 16):
+        return False
+    _need_cuda(q, k, v, z1, z2, w1, w2, state, weight, gate, out, nstate, m_state)
+    T = q.shape[0]
+    G = q.shape[1] // N
+    assert q.shape == k.shape == (T, G * N) and v.shape == gate.shape == out.shape == (T, H * P) and z1.shape == z2.shape == (T, H)
+    assert all(t.dtype == torch.float32 for t in (q, k, v, z1, z2, state, gate)) and z1.stride() == z2.stride()
+    assert all(t.stride(1) == 1 for t in (q, k, v, z1, gate, out)) and state.is_contiguous() and w1.dtype == w2.dtype
+    assert w1.numel() == w2.numel() == H and weight.numel() in (P, H * P) and weight.is_contiguous()
+    assert delta or (nstate.shape == (slots, H, N) and m_state.shape == (slots, H) and nstate.is_contiguous() and m_state.is_contiguous())
+    _call("memory", "hb_ms_single", q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z1.data_ptr(),
+          z2.data_ptr(), z1.stride(0), w1.data_ptr(), w2.data_ptr(), _dt(w1), float(cap), float(unit_eps), float(q_scale), float(den_eps),
+          float(eps), state.data_ptr(), _ptr(nstate), _ptr(m_state), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(),
+          batch.req_state_slot.data_ptr(), weight.data_ptr(), _dt(weight), 1 if weight.numel() == P else 0, gate.data_ptr(), gate.stride(0),
+          GATE_KINDS[gate_kind], out.data_ptr(), _dt(out), out.stride(0), batch.n_requests, H, G, N, P, 1 if delta else 0, _stream())
+    return True
 
 
 class ScaledPair:

@@ -449,7 +449,7 @@ class OutputNormBlock(Part):
     def param_specs(self):
         specs = [s for p in self.parts for s in p.param_specs()]
         if self.average:
-            specs.append(ParamSpec(self.average_name, (self.average,), init="ones"))
+            specs.append(ParamSpec(self.average_name, (self.average,), init="average"))
         return specs
 
     def load(self, tensors):

@@ -77,13 +77,14 @@ class GatedDeltaMixer(Mixer):
         g, za, zb = torch.split(proj[:, C:], [self.n_v, H, H], 1)
         qkv = torch.empty(T, C, dtype=torch.float32, device=dev)
         ops.ssd_conv(proj, 0, self.conv_w, self.conv_b, state["conv"], batch, qkv)
-        a, b, kq = ops.ms_delta_prepare(qkv, (0, self.n_qk), za, zb, self.a_log, self.dt_bias, self.kv_heads, self.dim,
-                                        self.dim ** -0.5, self.unit_eps)
         q, k, v = torch.split(qkv, [self.n_qk, self.n_qk, self.n_v], 1)
-        y = torch.empty(T, self.n_v, dtype=torch.float32, device=dev)
-        ops.ms_walk(q, k, v, a, b, state["S"], batch, y, kq=kq)
         out = torch.empty(T, self.n_v, dtype=self.ctx.dtype, device=dev)
-        ops.ms_finish(y, self.norm_w, g, "silu", out, H, self.eps)
+        if not ops.ms_single(q, k, v, za, zb, self.dt_bias, self.a_log, state["S"], self.norm_w, g, "silu", out, batch, self.dim ** -0.5,
+                             self.eps, unit_eps=self.unit_eps):
+            scal = ops.ms_delta_prepare(q, k, za, zb, self.a_log, self.dt_bias, batch, self.dim, self.dim ** -0.5, self.unit_eps)
+            y = torch.empty(T, self.n_v, dtype=torch.float32, device=dev)
+            ops.ms_delta_walk(q, k, v, scal, state["S"], batch, y)
+            ops.ms_finish(y, self.norm_w, g, "silu", out, H, self.eps)
         planes.record(batch, "attention", out)
         ops.linear_into_stream(out, self.wo, x)
         return None

@@ -148,7 +148,7 @@ class MaskedAttentionMixer(Mixer):
             wq = t["q_norm"].to(torch.float32).contiguous()
             self.norm_w = (wq, wq if self.reads_cache else t["k_norm"].to(torch.float32).contiguous())
         if self.distance_bias:
-            self.distance = (t["r1"].to(torch.float32).contiguous(), t["r2"].to(torch.float32).contiguous())
+            self.distance = ops.DistanceBias(t["r1"], t["r2"])
 
     def weight_bytes(self):
         return self.w_in.nbytes + self.wo.nbytes

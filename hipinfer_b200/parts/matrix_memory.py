@@ -66,11 +66,13 @@ class MatrixMemoryMixer(Mixer):
         ops.linear_rows32(xn, self.w_in, proj)
         q, k, v, g, zi, zf = torch.split(proj, [HD, HD, HP, HP, H, H], 1)
         out = torch.empty(T, HP, dtype=self.ctx.dtype, device=dev)
-        a, b, e = ops.ms_exp_gates(zi, zf, self.b_i, self.b_f, self.cap, state["m"], batch)
-        y = torch.empty(T, HP, dtype=torch.float32, device=dev)
-        nq = torch.empty(T, H, dtype=torch.float32, device=dev)
-        ops.ms_walk(q, k, v, a, b, state["S"], batch, y, self.dim ** -0.5, nstate=state["n"], nq=nq)
-        ops.ms_finish(y, self.norm_w, g, "sigmoid", out, H, self.eps, nq, e, self.den_eps)
+        if not ops.ms_single(q, k, v, zi, zf, self.b_i, self.b_f, state["S"], self.norm_w, g, "sigmoid", out, batch, self.dim ** -0.5,
+                             self.eps, state["n"], state["m"], self.cap, self.den_eps):
+            a, b, e = ops.ms_exp_gates(zi, zf, self.b_i, self.b_f, self.cap, state["m"], batch)
+            y = torch.empty(T, HP, dtype=torch.float32, device=dev)
+            nq = torch.empty(T, H, dtype=torch.float32, device=dev)
+            ops.ms_walk(q, k, v, a, b, state["S"], batch, y, self.dim ** -0.5, nstate=state["n"], nq=nq)
+            ops.ms_finish(y, self.norm_w, g, "sigmoid", out, H, self.eps, nq, e, self.den_eps)
         planes.record(batch, "attention", out)
         ops.linear_into_stream(out, self.wo, x)
         return None

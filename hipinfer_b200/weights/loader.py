@@ -28,7 +28,7 @@ from .safetensors_io import ModelFiles, SafetensorsError, save_safetensors
 @dataclass(frozen=True)
 class ParamSpec:
     """One tensor a part needs. `init` tells the random-weights mode how to draw it:
-    "normal" (N(0, std)), "ones" (1, plus N(0, norm_std) when asked), "zeros"."""
+    "normal" (N(0, std)), "ones" (1, plus N(0, norm_std) when asked), "zeros", "average" (1 over the number of elements)."""
 
     name: str
     shape: Tuple[int, ...]
@@ -138,6 +138,8 @@ def random_weights(specs: Sequence[ParamSpec], seed: int, std: float = 0.02, nor
             t = torch.ones(s.shape, dtype=torch.float32, device=device)
             if norm_std:
                 t = t + torch.randn(s.shape, generator=g, dtype=torch.float32, device=device) * norm_std
+        elif s.init == "average":
+            t = torch.full(s.shape, 1.0 / max(1, torch.Size(s.shape).numel()), dtype=torch.float32, device=device)
         elif s.init == "zeros":
             t = torch.zeros(s.shape, dtype=torch.float32, device=device)
         else:

@@ -255,9 +255,9 @@ def sub(tensors, prefix):
 def forward(cfg, tensors, tokens, layers_out=None, round_to=None):
     """Logits [T, vocab] of one sequence from position 0. cfg: the config.json dictionary; tensors: name -> tensor.
     layers_out (a list): the residual rows after every layer (averaged over the depth) are appended.
-    round_to (a dtype): every sublayer's input and result are rounded to it; the difference to the exact logits measures
-    how sensitive each position is to rounding."""
-    rd = (lambda t: t) if round_to is None else (lambda t: t.to(round_to).to(F))
+    round_to (a dtype, or a function): every sublayer's input and result are rounded to it; the difference to the exact
+    logits measures how sensitive each position is to rounding."""
+    rd = (lambda t: t) if round_to is None else round_to if callable(round_to) else (lambda t: t.to(round_to).to(F))
     eps = cfg["norm"]["eps"]
     x = tensors["embed"].to(F)[torch.as_tensor(tokens, dtype=torch.long)]
     states = [x]
