@@ -68,14 +68,12 @@ class SideBySideMixer(Mixer):
     def forward_pair(self, xn, batch, cache, state):
         """The two raw results and how they are to be joined (an ops.NormedPair or ops.ScaledPair), for a caller that joins them on its own way over the row."""
         state = state or {}
-        out = []
-        for side, part in (("left.", self.left), ("right.", self.right)):
-            y = torch.zeros(xn.shape[0], self.hidden, dtype=torch.float32, device=xn.device)
+        out = torch.zeros(2, xn.shape[0], self.hidden, dtype=torch.float32, device=xn.device)
+        for y, side, part in ((out[0], "left.", self.left), (out[1], "right.", self.right)):
             own = {k[len(side):]: v for k, v in state.items() if k.startswith(side)}
             left = part.forward(xn, y, batch, cache if part.cache_need() is not None else None, own)
             if isinstance(left, ops.Pending):
                 left.finish()
-            out.append(y)
         if not self.normed:
             return ops.ScaledPair(out[0], out[1], *self.scales)
         return ops.NormedPair(out[0], out[1], self.w_left, self.w_right, self.mix, self.eps)
