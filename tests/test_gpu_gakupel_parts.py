@@ -159,26 +159,17 @@ def _paged(k, v, ps, dtype, seed):
     return kc.to(dtype).to(DEV), vc.to(dtype).to(DEV), order.to(torch.int32)
 
 
-@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H,G,D,E,ps", [(4, 2, 64, 64, 16), (8, 2, 96, 48, 16), (3, 1, 10, 6, 8), (20, 1, 32, 32, 16), (4, 4, 128, 64, 32),
-                                        (6, 2, 96, 96, 16), (2, 2, 48, 80, 16), (8, 2, 128, 128, 16), (1, 1, 64, 64, 64)])
-@pytest.mark.parametrize("bias,one", [(True, True), (False, False), (True, False), (False, True)])
-def test_attention_with_distance_bias_and_constant_sink(dtype, H, G, D, E, ps, bias, one):
-    """Requests of unequal portions (single rows, a few rows, more than a flash tile, after cached tokens that end at and around
-    page borders); one key far back in each request has a score that stands out, so that a lost or shifted key shows; the
-    bias falls steeply over the first keys, so that a distance that is off by one shows."""
-    from hipinfer_b200.kernels import ops
-
-    lengths, ctx = [1, 1, 5, 150, 70, 1, 16], [0, 333, 64, 0, 129, 64, 15]
+def _attention_case(dtype, H, G, D, E, ps, bias, one, lengths, ctx, r1, r2):
+    """(q, caches, batch, wanted): requests of `lengths` rows after `ctx` cached tokens. One key far back in each request has a
+    score that stands out for its last row, so that a lost or shifted key shows."""
     scale = D ** -0.5
-    r1, r2 = 0.4 + rnd(H, seed=1).abs(), 0.2 + rnd(H, seed=2).abs()
     qs, caches, tables, want = [], [], [], []
     for i, (n, c) in enumerate(zip(lengths, ctx)):
         tot = n + c
         q, k, v = rnd(n, H, D, seed=10 + i), rnd(tot, G, D, seed=30 + i), rnd(tot, G, E, seed=50 + i)
         far = max(0, tot // 3 - 1)
         k[far] = 3.0 * k[far]
-        q[-1] = 2.5 * k[far].repeat_interleave(H // G, 0)                   # the last row asks for the far key
+        q[-1] = 2.5 * k[far].repeat_interleave(H // G, 0)
         q, k, v = (t.to(dtype).float() for t in (q, k, v))
         out = torch.zeros(n, H, E, dtype=F)
         for h in range(H):
@@ -206,13 +197,48 @@ def test_attention_with_distance_bias_and_constant_sink(dtype, H, G, D, E, ps, b
         base += kc.shape[0]
     batch = batch_of(lengths, ctx)
     batch.block_tables = [torch.stack(tables).to(DEV)]
-    q, kc, vc = torch.cat(qs).to(dtype).to(DEV), torch.cat(kcs), torch.cat(vcs)
+    return torch.cat(qs).to(dtype).to(DEV), torch.cat(kcs), torch.cat(vcs), batch, torch.cat(want)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,D,E,ps", [(4, 2, 64, 64, 16), (8, 2, 96, 48, 16), (3, 1, 10, 6, 8), (20, 1, 32, 32, 16), (4, 4, 128, 64, 32),
+                                        (6, 2, 96, 96, 16), (2, 2, 48, 80, 16), (8, 2, 128, 128, 16), (1, 1, 64, 64, 64)])
+@pytest.mark.parametrize("bias,one", [(True, True), (False, False), (True, False), (False, True)])
+def test_attention_with_distance_bias_and_constant_sink(dtype, H, G, D, E, ps, bias, one):
+    """Unequal portions (single rows, a few rows, more than a flash tile, after cached tokens that end at and around page
+    borders); the bias falls steeply over the first keys, so that a distance that is off by one shows. The tensor-core
+    kernels, the warp-MMA kernels and the plain one."""
+    from hipinfer_b200.kernels import ops
+
+    r1, r2 = 0.4 + rnd(H, seed=1).abs(), 0.2 + rnd(H, seed=2).abs()
+    q, kc, vc, batch, want = _attention_case(dtype, H, G, D, E, ps, bias, one, [1, 1, 5, 150, 70, 1, 16], [0, 333, 64, 0, 129, 64, 15], r1, r2)
     kw = dict(sink=torch.zeros(H, device=DEV) if one else None, distance=ops.DistanceBias(r1.to(DEV), r2.to(DEV)) if bias else None)
-    plains = (False, True) if dtype == torch.bfloat16 else (False,)        # the tensor-core kernels, the warp-MMA kernels, the plain one
+    plains = (False, True) if dtype == torch.bfloat16 else (False,)
     for force_rows, force_plain in [(False, p) for p in plains] + ([(True, False)] if dtype == torch.bfloat16 else []):
-        att = torch.full((sum(lengths), H * E), float("nan"), dtype=dtype, device=DEV)
-        ops.attention_masked(q, kc, vc, batch, 0, att, H, G, D, E, ps, scale, force_rows=force_rows, force_plain=force_plain, **kw)
-        close(att, torch.cat(want), dtype, f"rows {force_rows} plain {force_plain}", 5e-5 if dtype == torch.float32 else None)
+        att = torch.full(want.shape, float("nan"), dtype=dtype, device=DEV)
+        ops.attention_masked(q, kc, vc, batch, 0, att, H, G, D, E, ps, D ** -0.5, force_rows=force_rows, force_plain=force_plain, **kw)
+        close(att, want, dtype, f"rows {force_rows} plain {force_plain}", 5e-5 if dtype == torch.float32 else None)
+
+
+@pytest.mark.parametrize("D,G,H", [(64, 2, 8), (64, 1, 3), (128, 2, 8), (128, 1, 1)])
+@pytest.mark.parametrize("rows", [2, 12, 40])
+@pytest.mark.parametrize("steep", [False, True])
+def test_single_rows_far_into_their_sequences(D, G, H, rows, steep):
+    """Decode steps of few and of many rows at unequal positions up to 1,300, at and around the key splits' edges, and portions
+    beside them. steep: a bias that falls by hundreds within a tile (the kernels that bound a tile's maximum by its nearest
+    key leave such a one to the others)."""
+    from hipinfer_b200.kernels import ops
+
+    ctx = ([0, 1299, 255, 256, 511, 512, 513, 767, 1023, 1024, 63, 64] + list(range(100, 1300, 43)))[:rows]
+    r1, r2 = (30.0 if steep else 0.3) + rnd(H, seed=1).abs(), 0.2 + rnd(H, seed=2).abs()
+    dist = ops.DistanceBias(r1.to(DEV), r2.to(DEV))
+    assert (dist.spread > 60) == steep
+    sink = torch.zeros(H, device=DEV)
+    for lengths, c in (([1] * rows, ctx), ([1] * (rows - 1) + [300], ctx[:-1] + [777])):
+        q, kc, vc, batch, want = _attention_case(torch.bfloat16, H, G, D, D, 16, True, True, lengths, c, r1, r2)
+        att = torch.full(want.shape, float("nan"), dtype=torch.bfloat16, device=DEV)
+        ops.attention_masked(q, kc, vc, batch, 0, att, H, G, D, D, 16, D ** -0.5, sink=sink, distance=dist)
+        close(att, want, torch.bfloat16, f"{lengths[-1]}")
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
