@@ -1447,6 +1447,7 @@ def moe_combine(ys: torch.Tensor, pos: torch.Tensor, y: torch.Tensor, top: int) 
 # normed (csrc/matrix_state.cu, depth_average.cu)
 # ------------------------------------------------------------------------------------------
 MS_PIECE_TOKENS = 64    # tokens a piece of the linear recurrence (ms_walk); 0: always one walk a request
+MS_PIECE_BLOCKS = 296   # a step whose long portions make more blocks than this walks them in one go (two a streaming multiprocessor)
 
 
 def _ms_rows(q, k, v, state, y):
@@ -1466,15 +1467,15 @@ def ms_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, 
     nq [T, heads] = n . q * q_scale. q, k float32 [T, groups * N], v float32 [T, heads * P] (views of wider rows are fine);
     a, b float32 [T, heads]; state float32 [slots, heads, N, P]; y float32 [T, heads * P].
 
-    A step whose longest portion has at least three times MS_PIECE_TOKENS rows runs in pieces of that many tokens; the
-    results differ from the walk in one go by rounding only."""
+    A step whose longest portion has at least three times MS_PIECE_TOKENS rows runs in pieces of that many tokens, unless its
+    long portions fill the GPU by themselves; the results differ from the walk in one go by rounding only."""
     _need_cuda(q, k, v, a, b, state, y, nstate, nq)
     T, H, G, N, P = _ms_rows(q, k, v, state, y)
     assert a.shape == b.shape == (T, H) and a.dtype == b.dtype == torch.float32 and a.is_contiguous() and b.is_contiguous()
     if nstate is not None:
         assert nstate.shape == (state.shape[0], H, N) and nstate.is_contiguous() and nq.shape == (T, H) and nq.is_contiguous()
     L, pieces, ps, pn, pd = int(MS_PIECE_TOKENS), 0, None, None, None
-    if L > 0 and batch.max_q_len >= 3 * L:
+    if L > 0 and batch.max_q_len >= 3 * L and T // batch.max_q_len * H * -(-P // 32) <= MS_PIECE_BLOCKS:
         pieces = -(-batch.max_q_len // L)
         room = T // L + batch.n_requests               # every request ends with at most one short piece
         ps = torch.empty(room, H, N, P, dtype=torch.float32, device=q.device)
