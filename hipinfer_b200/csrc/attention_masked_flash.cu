@@ -307,7 +307,7 @@ __global__ void __launch_bounds__(FM_THREADS) attn_masked_flash_kernel(FlashMask
 }
 
 // the (D, E) pairs that are instantiated
-#define FM_SIZES(X) X(6, 12) X(6, 6) X(3, 6) X(4, 8) X(4, 6) X(8, 16) X(6, 8) X(12, 16) X(2, 4) X(4, 4) X(8, 8) X(3, 4)
+#define FM_SIZES(X) X(6, 12) X(5, 10) X(3, 6) X(4, 8) X(4, 6) X(8, 16) X(6, 8) X(12, 16) X(2, 4) X(4, 4) X(8, 8) X(3, 4)
 
 HB_EXPORT int hb_attn_masked_flash_supported(int D, int E) {
 #define FM_CHECK(DK, EN) if (D == 16 * DK && E == 8 * EN) return 1;

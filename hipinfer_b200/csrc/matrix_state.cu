@@ -333,7 +333,7 @@ __global__ void __launch_bounds__(1024) ms_exp_gates_kernel(const float* __restr
   __shared__ float wF[32], wM[32], ms[1025];
   hb_pdl_launch();
   hb_pdl_wait();
-  const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthr = blockDim.x, nw = nthr >> 5;
+  const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthr = blockDim.x;
   const int t0 = q_start[r], len = q_len[r];
   float* mp = m_state + (size_t)slot[r] * H + h;
   float m0 = *mp;
@@ -371,7 +371,6 @@ __global__ void __launch_bounds__(1024) ms_exp_gates_kernel(const float* __restr
     m0 = ms[n];
     __syncthreads();
   }
-  (void)nw;
   if (tid == 0 && len > 0) *mp = m0;
 }
 

@@ -81,7 +81,7 @@ class MaskedAttentionMixer(Mixer):
         if self.q_temp and self.q_temp[1] <= 0:
             raise ValueError(f"attention: a query temperature every {self.q_temp[1]} positions")
         self.shared_values = p.get("values", "own") == "keys"
-        if self.shared_values and (self.vdim != self.dim or self.reads_cache_param(p)):
+        if self.shared_values and (self.vdim != self.dim or p.get("reads_cache")):
             raise ValueError(f"attention: values that are the keys need vdim = dim and a cache of their own ({self.vdim}, {self.dim})")
         self.distance_bias = bool(p.get("distance_bias", False))
         self.sink_one = p.get("sink") == "one"
@@ -98,10 +98,6 @@ class MaskedAttentionMixer(Mixer):
         self.w_in = self.wo = self.sink = self.table = self.norm_w = self.distance = None
         if not ctx.is_meta:
             self.table = ops.shared_rope_table(self.rot_dims, self.rot_base, ctx.max_model_len, ctx.device, p.get("rot_scaling"))
-
-    @staticmethod
-    def reads_cache_param(p):
-        return bool(p.get("reads_cache", False))
 
     @property
     def n_q(self):

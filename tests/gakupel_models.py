@@ -68,7 +68,7 @@ B = model(97, 48, [delta(3, 3, 8, 8, 1, mlp=moe(40, 1, 1)), attention(3, 3, 8, m
 # C: heads of 64, 96 and 128 (the tensor-core kernels, one of their sizes only in part); sixteen experts in four groups
 C = model(211, 128, [parallel((8, 2, 64, 64, 0.2, 100), (2, 64, 64, 15.0), mlp=moe(64, 16, 4, (4, 2), 1.3, 64)),
                      attention(4, 1, 128, rot_dims=64, mlp=dense(256)), delta(2, 2, 64, 128, 3, mlp=dense(96)),
-                     parallel((4, 4, 96, 96, 0.3, 64), (2, 96, 32, 15.0), mlp=moe(96, 4, 2, (2, 1), 1.0, 32)),
+                     parallel((4, 4, 96, 96, 0.25, 48), (2, 96, 32, 15.0), mlp=moe(96, 4, 2, (2, 1), 1.0, 32)),
                      attention(20, 1, 32, rot_dims=16)], max_positions=900)
 # D: sizes no vectorised kernel takes: a width that is no multiple of 4, heads of 10, 6 and 7
 D = model(90, 50, [attention(2, 1, 10, rot_dims=6, mlp=moe(30, 3, 2, None, 1.0, 10)),

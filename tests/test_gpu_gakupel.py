@@ -271,7 +271,7 @@ def _random_config(seed):
         else:
             left = (kv * pick([1, 2, 3, 5]), kv, dim, pick([16, 32, 48, 64, 96, 128])) + pick([(), (0.3, 50), (1.0, 7)])
             layers.append(tm.parallel(left, (pick([1, 2, 4, 6]), pick([16, 32, 48, 64, 128]), pick([16, 32, 48, 64, 128]), pick([2.0, 15.0, 30.0])),
-                                      pick([0.3, 0.6, 1.0]), pick([0.9, 1.0, -0.4]), mlp=mlp))
+                                      pick([0.3, 0.7, 1.0]), pick([0.8, 1.0, -0.4]), mlp=mlp))
     return tm.model(pick([64, 97, 300, 576]), width, layers, eps=pick([1e-5, 1e-6]), max_positions=512)
 
 
