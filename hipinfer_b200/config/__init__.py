@@ -9,6 +9,8 @@ from .mavinex import (MavinexConfig, MavinexLayerConfig, ScaledRotaryConfig, Sel
                       SinkLatentConfig, WindowAttentionConfig)
 from .gakupel import (DistanceAttentionConfig, GakupelConfig, GakupelLayerConfig, GatedDeltaConfig, GeluFFConfig, GroupedExpertsConfig,
                       MatrixMemoryConfig, ParallelMixerConfig, QueryTemperatureConfig, SharedKeyAttentionConfig)
+from .selovik import (IdentityExpertsConfig, LoopConfig, RotaryDiffAttentionConfig, SelovikConfig, SelovikLayerConfig,
+                      SquaredReluFFConfig)
 
 __all__ = ["Architecture", "ConfigError", "ModelConfig", "config_from_dict", "get_architecture", "load_config",
            "register_architecture", "registered_architectures", "save_config", "take", "Llama3RopeScaling",
@@ -17,4 +19,5 @@ __all__ = ["Architecture", "ConfigError", "ModelConfig", "config_from_dict", "ge
            "DenseFFConfig", "Mamba2Config", "RoutedFFConfig", "RunopelConfig", "RunopelLayerConfig", "WindowLatentConfig",
            "MavinexConfig", "MavinexLayerConfig", "ScaledRotaryConfig", "SelectiveScanConfig", "SideBySideConfig", "SinkLatentConfig",
            "WindowAttentionConfig", "DistanceAttentionConfig", "GakupelConfig", "GakupelLayerConfig", "GatedDeltaConfig", "GeluFFConfig",
-           "GroupedExpertsConfig", "MatrixMemoryConfig", "ParallelMixerConfig", "QueryTemperatureConfig", "SharedKeyAttentionConfig"]
+           "GroupedExpertsConfig", "MatrixMemoryConfig", "ParallelMixerConfig", "QueryTemperatureConfig", "SharedKeyAttentionConfig",
+           "IdentityExpertsConfig", "LoopConfig", "RotaryDiffAttentionConfig", "SelovikConfig", "SelovikLayerConfig", "SquaredReluFFConfig"]

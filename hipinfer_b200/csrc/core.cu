@@ -302,8 +302,8 @@ HB_EXPORT int hb_scale_add(float* x, const float* y, long ldy, const void* scale
 }
 
 // ---------------------------------------------------------------------------------------
-// y = act(x + bias) over columns [c0, c0 + n) of 32-bit rows, into a matrix of its own: act 0 nothing, 1 tanh.
-// (The small middle of a low-rank projection pair.)
+// y = act(x + bias) over columns [c0, c0 + n) of 32-bit rows, into a matrix of its own: act 0 nothing, 1 tanh (the small
+// middle of a low-rank projection pair), 2 the exact GELU, 3 the square of relu.
 // ---------------------------------------------------------------------------------------
 template <typename TB_, typename TO>
 __global__ void bias_act_kernel(const float* __restrict__ x, long ldx, const TB_* __restrict__ bias, TO* __restrict__ y,
@@ -316,13 +316,14 @@ __global__ void bias_act_kernel(const float* __restrict__ x, long ldx, const TB_
   float v = x[m * ldx + c] + (bias ? hb_to_float(bias[c]) : 0.f);
   if (act == 1) v = tanhf(v);
   else if (act == 2) v = 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  else if (act == 3) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
   y[m * ldy + c] = hb_from_float<TO>(v);
 }
 
 HB_EXPORT int hb_bias_act(const float* x, long ldx, const void* bias, int bias_dt, void* y, int y_dt, long ldy, int M,
                           int n, int act, cudaStream_t s) {
   if (M <= 0 || n <= 0) return 0;
-  if (act < 0 || act > 2) HB_FAIL("hb_bias_act: unknown activation %d", act);
+  if (act < 0 || act > 3) HB_FAIL("hb_bias_act: unknown activation %d", act);
   const size_t tot = (size_t)M * n;
   HB_DISPATCH_2(bias_dt, y_dt, "hb_bias_act",
                 (hb_launch(bias_act_kernel<TA, TB>, (unsigned)((tot + 255) / 256), 256, 0, s, x, ldx, (const TA*)bias,
@@ -605,7 +606,13 @@ HB_EXPORT int hb_rope_kv(const void* qkv, int qkv_dt, long ld, const int* pos, c
 // With pre_wq / pre_wk the q row (all H heads at once) and the k row are first divided by their own root mean square
 // (pre_eps inside the root) and multiplied by a weight per column, before the rotation.
 // No slot map (a layer that reads another layer's cache): q alone. A warp works on a head at a time.
+// With `maps` > 1 the k heads come in groups of that many which lie side by side in one plane row (G counts them all; the
+// planes are [page][G / maps][page_size][maps * D] and [page][G / maps][page_size][E]).
 // ---------------------------------------------------------------------------------------
+__device__ __forceinline__ size_t rn_key_row(int kh, int G, int maps, size_t page, size_t off, int page_size) {
+  return ((page * (G / maps) + kh / maps) * page_size + off) * maps + kh % maps;
+}
+
 template <typename TQ, typename TW>
 __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __restrict__ proj, long ld, int q_off, int k_off,
                                                               int v_off, const int* __restrict__ pos,
@@ -615,7 +622,7 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
                                                               TQ* __restrict__ kc, TQ* __restrict__ vc, int H, int G, int D,
                                                               int E, int page_size, const TW* __restrict__ pre_wq,
                                                               const TW* __restrict__ pre_wk, float pre_eps, int pre_head,
-                                                              float temp_coef, double temp_every) {
+                                                              float temp_coef, double temp_every, int maps) {
   extern __shared__ float rn_sh[];      // [8 warps][D], then 32 floats for the sums of a row norm
   hb_pdl_launch();
   hb_pdl_wait();
@@ -673,14 +680,54 @@ __global__ void __launch_bounds__(256) rope_norm_store_kernel(const float* __res
       f = rsqrtf(hb_warp_sum(ss) / (float)D + eps);
     }
     if (hh < H) f *= tq;
-    TQ* dst = hh < H ? q_out + ((size_t)t * H + hh) * D : kc + ((page * G + (hh - H)) * page_size + off) * D;
+    TQ* dst = hh < H ? q_out + ((size_t)t * H + hh) * D : kc + rn_key_row(hh - H, G, maps, page, off, page_size) * D;
     for (int d = lane; d < D; d += 32) dst[d] = hb_from_float<TQ>(buf[d] * f);
     __syncwarp();
   }
   if (slot < 0) return;
-  for (int i = blockIdx.y * 256 + threadIdx.x; i < G * E; i += 256 * gridDim.y) {
+  const int GV = G / maps;
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < GV * E; i += 256 * gridDim.y) {
     const int h = i / E, e = i - h * E;
-    vc[((page * G + h) * page_size + off) * E + e] = hb_from_float<TQ>(row[v_off + i]);
+    vc[((page * GV + h) * page_size + off) * E + e] = hb_from_float<TQ>(row[v_off + i]);
+  }
+}
+
+// Rotation and cache write alone (no norm, no temperature; halves paired from dimension 0 on), four columns an access: a
+// thread turns four pairs, or copies four columns that pass unchanged, or four values. The same products and sums.
+template <typename TQ>
+__global__ void __launch_bounds__(256) rope_store_vec_kernel(const float* __restrict__ proj, long ld, int q_off, int k_off, int v_off,
+                                                             const int* __restrict__ pos, const int* __restrict__ slot_map,
+                                                             const float2* __restrict__ table, int rot, TQ* __restrict__ q_out,
+                                                             TQ* __restrict__ kc, TQ* __restrict__ vc, int H, int G, int D, int E,
+                                                             int page_size, int maps) {
+  hb_pdl_launch();
+  const int t = blockIdx.x, half = rot >> 1, turns = half >> 2, per = turns + ((D - rot) >> 2);
+  const int slot = slot_map ? slot_map[t] : -1;
+  const float2* cs = table + (size_t)pos[t] * half;
+  hb_pdl_wait();
+  const float* row = proj + (size_t)t * ld;
+  const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot - page * page_size : 0;
+  const int GV = G / maps, n_qk = (H + (slot >= 0 ? G : 0)) * per, n = n_qk + (slot >= 0 ? GV * E / 4 : 0);
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < n; i += 256 * gridDim.y) {
+    if (i >= n_qk) {
+      const int c = (i - n_qk) * 4, h = c / E, e = c - h * E;
+      hb_store4(vc + (((size_t)page * GV + h) * page_size + off) * E + e, hb_load4(row + v_off + c));
+      continue;
+    }
+    const int hh = i / per, j = i - hh * per;
+    const float* src = hh < H ? row + q_off + (size_t)hh * D : row + k_off + (size_t)(hh - H) * D;
+    TQ* dst = hh < H ? q_out + ((size_t)t * H + hh) * D : kc + rn_key_row(hh - H, G, maps, page, off, page_size) * D;
+    if (j >= turns) {
+      const int d = rot + (j - turns) * 4;
+      hb_store4(dst + d, hb_load4(src + d));
+      continue;
+    }
+    const float4 u = hb_load4(src + 4 * j), v = hb_load4(src + half + 4 * j);
+    const float4 c0 = *(const float4*)(cs + 4 * j), c1 = *(const float4*)(cs + 4 * j + 2);     // (cos, sin) of pairs 4 j .. 4 j + 3
+    hb_store4(dst + 4 * j, make_float4(__fsub_rn(__fmul_rn(u.x, c0.x), __fmul_rn(v.x, c0.y)), __fsub_rn(__fmul_rn(u.y, c0.z), __fmul_rn(v.y, c0.w)),
+                                       __fsub_rn(__fmul_rn(u.z, c1.x), __fmul_rn(v.z, c1.y)), __fsub_rn(__fmul_rn(u.w, c1.z), __fmul_rn(v.w, c1.w))));
+    hb_store4(dst + half + 4 * j, make_float4(__fadd_rn(__fmul_rn(v.x, c0.x), __fmul_rn(u.x, c0.y)), __fadd_rn(__fmul_rn(v.y, c0.z), __fmul_rn(u.y, c0.w)),
+                                              __fadd_rn(__fmul_rn(v.z, c1.x), __fmul_rn(u.z, c1.y)), __fadd_rn(__fmul_rn(v.w, c1.z), __fmul_rn(u.w, c1.w))));
   }
 }
 
@@ -688,8 +735,9 @@ HB_EXPORT int hb_rope_norm_store(const float* proj, long ld, int q_off, int k_of
                                  const int* slot_map, const void* table, int rot, int rot_off, int pairing, int unit_norm,
                                  float eps, void* q_out, void* kc, void* vc, int q_dt, int T, int H, int G, int D, int E, int page_size,
                                  const void* pre_wq, const void* pre_wk, int pre_dt, float pre_eps, int pre_head, float temp_coef,
-                                 double temp_every, cudaStream_t s) {
+                                 double temp_every, int maps, cudaStream_t s) {
   if (T <= 0) return 0;
+  if (maps < 1 || G % maps) HB_FAIL("hb_rope_norm_store: %d key heads in groups of %d", G, maps);
   if (rot < 0 || rot_off < 0 || rot_off + rot > D || (rot & 1)) HB_FAIL("hb_rope_norm_store: %d rotated dimensions from %d on of a head of %d", rot, rot_off, D);
   if (slot_map && (!kc || !vc || G <= 0 || E <= 0 || page_size <= 0)) HB_FAIL("hb_rope_norm_store: a slot map without caches or sizes");
   const size_t smem = (size_t)(8 * D + 32) * sizeof(float);
@@ -704,10 +752,22 @@ HB_EXPORT int hb_rope_norm_store(const float* proj, long ld, int q_off, int k_of
     if (split > 8) split = 8;
     if (split < 1) split = 1;
   }
+  const uintptr_t bits = (uintptr_t)proj | (uintptr_t)table | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)vc;
+  if (!pre_wq && !unit_norm && temp_every <= 0.0 && pairing == 0 && rot_off == 0 && (rot & 7) == 0 && (D & 3) == 0 && (E & 3) == 0 &&
+      (ld & 3) == 0 && ((q_off | k_off | v_off) & 3) == 0 && !(bits & 15)) {
+    const int items = (H + G) * (rot / 8 + (D - rot) / 4) + G / maps * E / 4;
+    int blocks = 1;
+    while (blocks < 8 && blocks * 2 * T <= 1184 && blocks * 256 < items) blocks *= 2;
+    HB_DISPATCH_1(q_dt, "hb_rope_norm_store",
+                  (hb_launch(rope_store_vec_kernel<TA>, dim3(T, blocks), 256, 0, s, proj, ld, q_off, k_off, v_off, pos, slot_map,
+                             (const float2*)table, rot, (TA*)q_out, (TA*)kc, (TA*)vc, H, G, D, E, page_size, maps)));
+    HB_CHECK_LAUNCH("hb_rope_norm_store");
+    return 0;
+  }
   HB_DISPATCH_2(q_dt, pre_dt, "hb_rope_norm_store",
                 (hb_launch(rope_norm_store_kernel<TA, TB>, dim3(T, split), 256, smem, s, proj, ld, q_off, k_off, v_off, pos, slot_map,
                            (const float2*)table, rot, rot_off, pairing, unit_norm, eps, (TA*)q_out, (TA*)kc, (TA*)vc, H, G, D, E,
-                           page_size, (const TB*)pre_wq, (const TB*)pre_wk, pre_eps, pre_head, temp_coef, temp_every)));
+                           page_size, (const TB*)pre_wq, (const TB*)pre_wk, pre_eps, pre_head, temp_coef, temp_every, maps)));
   HB_CHECK_LAUNCH("hb_rope_norm_store");
   return 0;
 }

@@ -20,7 +20,7 @@
 
 HB_TL_DEFINE(stream)
 
-enum { ST_F32 = 0, ST_BF16 = 1, ST_ADD_F32 = 2, ST_SWIGLU_BF16 = 3, ST_SLICES = 4, ST_GEGLU_BF16 = 5, ST_GELU_BF16 = 6 };   // 5: as 3 with the tanh form of GELU; 6: as 1 after the exact GELU
+enum { ST_F32 = 0, ST_BF16 = 1, ST_ADD_F32 = 2, ST_SWIGLU_BF16 = 3, ST_SLICES = 4, ST_GEGLU_BF16 = 5, ST_GELU_BF16 = 6, ST_RELU2_BF16 = 7 };   // 5: as 3 with the tanh form of GELU; 6: as 1 after the exact GELU; 7: as 1 after the square of relu
 #define ST_IS_GLU(e) ((e) == ST_SWIGLU_BF16 || (e) == ST_GEGLU_BF16)
 constexpr int ST_ROWS = 128, ST_BK = 64, ST_W_BYTES = ST_ROWS * ST_BK * 2;
 
@@ -43,6 +43,7 @@ __device__ __forceinline__ void stream_store(int epi, void* C, long ldc, int m, 
   } else if (n < N) {
     if (epi == ST_BF16) ((__nv_bfloat16*)C)[(size_t)m * ldc + n] = __float2bfloat16_rn(v);
     else if (epi == ST_GELU_BF16) ((__nv_bfloat16*)C)[(size_t)m * ldc + n] = __float2bfloat16_rn(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+    else if (epi == ST_RELU2_BF16) ((__nv_bfloat16*)C)[(size_t)m * ldc + n] = __float2bfloat16_rn(fmaxf(v, 0.f) * fmaxf(v, 0.f));
     else if (epi == ST_ADD_F32) ((float*)C)[(size_t)m * ldc + n] += v;
     else ((float*)C)[(size_t)m * ldc + n] = v;
   }
@@ -313,7 +314,7 @@ HB_EXPORT int hb_gemm_stream(const void* A, long lda, const void* W, long ldw, v
   if (M <= 0 || N <= 0) return 0;
   if (M > 64) HB_FAIL("hb_gemm_stream: M = %d is beyond 64 rows", M);
   if (K <= 0 || (K & 7)) HB_FAIL("hb_gemm_stream: K = %d must be a positive multiple of 8 (16-byte rows for TMA)", K);
-  if (epi < 0 || epi > 6) HB_FAIL("hb_gemm_stream: unknown epilogue %d", epi);
+  if (epi < 0 || epi > 7) HB_FAIL("hb_gemm_stream: unknown epilogue %d", epi);
   if (ST_IS_GLU(epi) && (N & 31)) HB_FAIL("hb_gemm_stream: a gated epilogue needs N = %d to be a multiple of 32", N);
   if (!status) HB_FAIL("hb_gemm_stream: no status word");
   int kslice, ksplit, n_blocks;
@@ -346,7 +347,7 @@ HB_EXPORT int hb_gemm_stream(const void* A, long lda, const void* W, long ldw, v
 // Finish a product that was left as slices (epi 4): C per `epi` (0 to 3) from ws, for the same M, N, K.
 HB_EXPORT int hb_gemm_stream_finish(const float* ws, void* C, long ldc, int M, int N, int K, int epi, cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
-  if (epi < 0 || (epi > 3 && epi != ST_GEGLU_BF16 && epi != ST_GELU_BF16)) HB_FAIL("hb_gemm_stream_finish: unknown epilogue %d", epi);
+  if (epi < 0 || (epi > 3 && epi != ST_GEGLU_BF16 && epi != ST_GELU_BF16 && epi != ST_RELU2_BF16)) HB_FAIL("hb_gemm_stream_finish: unknown epilogue %d", epi);
   int kslice, ksplit, n_blocks;
   long per_token;
   hb_gemm_stream_plan(N, K, &kslice, &ksplit, &per_token, &n_blocks);

@@ -16,7 +16,7 @@
 // drains and returns.
 #include "tc_common.cuh"
 
-enum { EPI_F32 = 0, EPI_BF16 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_ROPE_KV = 4, EPI_GEGLU_BF16 = 5, EPI_GELU_BF16 = 6 };   // 6: bf16 after the exact (erf) GELU, no gate
+enum { EPI_F32 = 0, EPI_BF16 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_ROPE_KV = 4, EPI_GEGLU_BF16 = 5, EPI_GELU_BF16 = 6, EPI_RELU2_BF16 = 7 };   // 6: bf16 after the exact (erf) GELU, no gate; 7: after the square of relu
 
 // The gated epilogues: act(gate) * up over 16-interleaved columns, act = silu (3) or the tanh form of GELU (5), which is
 // g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)).
@@ -56,9 +56,10 @@ struct GemmSmem {
   static constexpr int TOTAL_TS = STAGING_OFFSET + 4 * 2 * 4096 + 1024;
 };
 
-#define EPI_IS_BF16(E) ((E) == EPI_BF16 || (E) == EPI_GELU_BF16)
+#define EPI_IS_BF16(E) ((E) == EPI_BF16 || (E) == EPI_GELU_BF16 || (E) == EPI_RELU2_BF16)
 template <int EPI> __device__ __forceinline__ float hb_bf16_act(float v) {
   if (EPI == EPI_GELU_BF16) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  if (EPI == EPI_RELU2_BF16) { const float r = fmaxf(v, 0.f); return r * r; }
   return v;
 }
 
@@ -611,6 +612,7 @@ static int dispatch_epi(int epi, const CUtensorMap& ma, const CUtensorMap& mw, v
     case EPI_SWIGLU_BF16: return launch_gemm_tc<BN, STAGES, EPI_SWIGLU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
     case EPI_GEGLU_BF16: return launch_gemm_tc<BN, STAGES, EPI_GEGLU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
     case EPI_GELU_BF16: return launch_gemm_tc<BN, STAGES, EPI_GELU_BF16>(ma, mw, C, ldc, M, N, K, status, s);
+    case EPI_RELU2_BF16: return launch_gemm_tc<BN, STAGES, EPI_RELU2_BF16>(ma, mw, C, ldc, M, N, K, status, s);
   }
   HB_FAIL("hb_gemm_tc: unknown epilogue %d", epi);
 }
@@ -652,6 +654,7 @@ HB_EXPORT int hb_gemm_tc(const void* A, long lda, const void* W, long ldw, void*
       case EPI_SWIGLU_BF16: r = launch_gemm_pair<EPI_SWIGLU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       case EPI_GEGLU_BF16: r = launch_gemm_pair<EPI_GEGLU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       case EPI_GELU_BF16: r = launch_gemm_pair<EPI_GELU_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
+      case EPI_RELU2_BF16: r = launch_gemm_pair<EPI_RELU2_BF16>(ma, W, ldw, C, ldc, M, N, K, status, s); break;
       default: HB_FAIL("hb_gemm_tc: unknown epilogue %d", epi);
     }
     if (r) return r;

@@ -8,7 +8,11 @@
 // the weight, silu(g) * u * s, again in 32-bit.
 // A third form (route mode 2): s = sigmoid(z); c = s + correction chooses, where the experts form equal groups of neighbours
 // only among the groups that rank best by the sum of their two largest c; the weights are the chosen s (without the
-// correction) divided by their sum, times a constant. Beside the router's rows one more row may give a number per token,
+// correction) divided by their sum, times a constant.
+// A fourth form (route mode 3): s = softmax(z) over all E; c = s + correction chooses, within the groups that rank best by their
+// largest c; the weights are the chosen s as they are.
+// Identity experts (any form): the last of the E router rows name experts without weights, whose result is the row itself:
+// their weights' sum goes to a number per token and what adds the results up adds the row times it. Beside the router's rows one more row may give a number per token,
 // sigmoid(w . h), that a shared expert's result is multiplied by.
 //
 // moe_route_kernel          scores and the chosen experts of every row: expert [T][top], weight [T][top]
@@ -38,7 +42,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
                                                                float* __restrict__ weight, int W, int E, int top, int mode,
                                                                const TW* __restrict__ correction, int groups, int keep, float scale,
                                                                const TW* __restrict__ shared_gate, float* __restrict__ shared_weight,
-                                                               int vec) {
+                                                               int vec, int n_real, float* __restrict__ identity_weight) {
   extern __shared__ float mr_sm[];     // [E] the scores, [E] those without the correction, [groups] the groups' sums
   float* sc = mr_sm;
   float* plain = sc + E;
@@ -69,13 +73,26 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
       continue;
     }
     if (bias) acc += hb_to_float(bias[e]);
-    const float v = mode == 1 ? acc : 1.f / (1.f + expf(-acc));
+    const float v = mode == 1 || mode == 3 ? acc : 1.f / (1.f + expf(-acc));
     sc[e] = mode == 2 ? v + hb_to_float(correction[e]) : v;
     plain[e] = v;
   }
   __syncthreads();
   if (warp != 0) return;
-  if (mode == 2 && groups > 1) {
+  if (mode == 3) {                       // the softmax over all E, then the corrections
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, plain[e]);
+    mx = hb_warp_max(mx);
+    for (int e = lane; e < E; e += 32) sum += expf(plain[e] - mx);
+    sum = hb_warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float v = expf(plain[e] - mx) / sum;
+      plain[e] = v;
+      sc[e] = v + (correction ? hb_to_float(correction[e]) : 0.f);
+    }
+    __syncwarp();
+  }
+  if (mode >= 2 && groups > 1) {
     const int span = E / groups;
     for (int q = lane; q < groups; q += 32) {
       float a = -INFINITY, b = -INFINITY;                  // the two largest
@@ -83,7 +100,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
         const float v = sc[e];
         if (v > a) { b = a; a = v; } else if (v > b) b = v;
       }
-      gs[q] = span > 1 ? a + b : a;
+      gs[q] = span > 1 && mode == 2 ? a + b : a;
     }
     __syncwarp();
     for (int q = lane; q < groups; q += 32) {
@@ -121,7 +138,13 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
     }
     __syncwarp();
   }
-  if (mode != 0 && lane == 0)
+  if (identity_weight && lane == 0) {
+    float w = 0.f;
+    for (int k = 0; k < top; k++)
+      if (expert[(size_t)t * top + k] >= n_real) w += weight[(size_t)t * top + k];
+    identity_weight[t] = w;
+  }
+  if ((mode == 1 || mode == 2) && lane == 0)
     for (int k = 0; k < top; k++) {
       const float w = weight[(size_t)t * top + k];
       weight[(size_t)t * top + k] = mode == 1 ? w / den : w / (den + 1e-20f) * scale;
@@ -131,12 +154,17 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
 // mode 0: the scores are sigmoid(z) and the chosen scores are the weights; mode 1: the largest logits z choose and the
 // weights are the softmax over the chosen logits alone; mode 2: sigmoid(z) + correction [E] chooses, within the `keep` best of
 // `groups` groups, and the weights are the chosen sigmoid(z) over their sum, times scale. bias (the router's element type, or
-// null) is added to z. shared_gate [W] (or null): shared_weight[t] = sigmoid(shared_gate . row).
+// null) is added to z. mode 3: softmax(z) + correction (or null) chooses, within the groups whose largest is largest, and the
+// weights are the chosen softmax(z). identity_weight [T] (or null; modes 0 and 3): the sum of the weights of the chosen experts
+// from n_real on. shared_gate [W] (or null): shared_weight[t] = sigmoid(shared_gate . row).
 HB_EXPORT int hb_moe_route(const void* xn, int x_dt, long ldx, const void* router, const void* bias, int w_dt, int* expert,
                            float* weight, int T, int W, int E, int top, int mode, const void* correction, int groups, int keep,
-                           float scale, const void* shared_gate, float* shared_weight, cudaStream_t s) {
+                           float scale, const void* shared_gate, float* shared_weight, int n_real, float* identity_weight, cudaStream_t s) {
   if (T <= 0) return 0;
   if (mode == 2 && !correction) HB_FAIL("hb_moe_route: the third form needs its corrections");
+  if (mode < 0 || mode > 3) HB_FAIL("hb_moe_route: unknown form %d", mode);
+  if (n_real < E && (!identity_weight || (mode != 0 && mode != 3)))
+    HB_FAIL("hb_moe_route: identity experts need a place for their weight and weights that are not normalised");
   if (groups > 1 && (E % groups || keep < 1 || keep > groups || (long)keep * (E / groups) < top))
     HB_FAIL("hb_moe_route: %d experts in %d groups of which %d stay, %d chosen", E, groups, keep, top);
   if (shared_gate && !shared_weight) HB_FAIL("hb_moe_route: a shared expert's gate needs a place for its result");
@@ -149,7 +177,7 @@ HB_EXPORT int hb_moe_route(const void* xn, int x_dt, long ldx, const void* route
     auto kern = moe_route_kernel<TA, TB>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     hb_launch(kern, dim3(T), dim3(threads), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert, weight,
-              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight, vec);
+              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight, vec, n_real, identity_weight);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_route");
   return 0;
@@ -181,11 +209,12 @@ template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(MG_THREADS) moe_gate_up_rows_kernel(const TA* __restrict__ xn, long ldx,
                                                                       const TW* __restrict__ wgu, const int* __restrict__ expert,
                                                                       const float* __restrict__ weight, TO* __restrict__ act,
-                                                                      int W, int F, int top, int vec, int at_output) {
+                                                                      int W, int F, int top, int vec, int at_output, int E) {
   extern __shared__ __align__(16) float mg_row[];      // [W]
   hb_pdl_launch();
   hb_pdl_wait();
   const int pair = blockIdx.y, t = pair / top, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  if (expert[pair] >= E) return;                       // an identity expert has no hidden rows
   for (int i = threadIdx.x; i < W; i += MG_THREADS) mg_row[i] = hb_to_float(xn[(size_t)t * ldx + i]);
   __syncthreads();
   const int e = expert[pair];
@@ -201,7 +230,7 @@ __global__ void __launch_bounds__(MG_THREADS) moe_gate_up_rows_kernel(const TA* 
 }
 
 HB_EXPORT int hb_moe_gate_up_rows(const void* xn, int x_dt, long ldx, const void* wgu, int w_dt, const int* expert,
-                                  const float* weight, void* act, int T, int W, int F, int top, int at_output, cudaStream_t s) {
+                                  const float* weight, void* act, int T, int W, int F, int top, int at_output, int E, cudaStream_t s) {
   if (T <= 0) return 0;
   const size_t smem = (size_t)W * sizeof(float);
   if (smem > 200 * 1024) HB_FAIL("hb_moe_gate_up_rows: a row of %d does not fit shared memory", W);
@@ -212,7 +241,7 @@ HB_EXPORT int hb_moe_gate_up_rows(const void* xn, int x_dt, long ldx, const void
   HB_DISPATCH_2(x_dt, w_dt, "hb_moe_gate_up_rows", do {
     auto kern = moe_gate_up_rows_kernel<TA, TB, TA>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)wgu, expert, weight, (TA*)act, W, F, top, vec, at_output);
+    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)wgu, expert, weight, (TA*)act, W, F, top, vec, at_output, E);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_gate_up_rows");
   return 0;
@@ -221,7 +250,8 @@ HB_EXPORT int hb_moe_gate_up_rows(const void* xn, int x_dt, long ldx, const void
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(MG_THREADS) moe_down_rows_kernel(const TA* __restrict__ act, const TW* __restrict__ wd,
                                                                    const int* __restrict__ expert, float* __restrict__ y, long ldy,
-                                                                   int W, int F, int top, int vec) {
+                                                                   int W, int F, int top, int vec, int E, const TA* __restrict__ xn,
+                                                                   long ldx, const float* __restrict__ identity_weight) {
   extern __shared__ __align__(16) float md_act[];      // [top][F4], F4 = F rounded up to four
   hb_pdl_launch();
   hb_pdl_wait();
@@ -229,7 +259,7 @@ __global__ void __launch_bounds__(MG_THREADS) moe_down_rows_kernel(const TA* __r
   const int F4 = (F + 3) & ~3;
   for (int i = threadIdx.x; i < top * F; i += MG_THREADS) {
     const int k = i / F, j = i - k * F;
-    md_act[k * F4 + j] = hb_to_float(act[((size_t)t * top + k) * F + j]);
+    md_act[k * F4 + j] = expert[(size_t)t * top + k] < E ? hb_to_float(act[((size_t)t * top + k) * F + j]) : 0.f;
   }
   __syncthreads();
   const int n1 = min(W, (int)(blockIdx.x + 1) * MG_ROWS);
@@ -237,14 +267,18 @@ __global__ void __launch_bounds__(MG_THREADS) moe_down_rows_kernel(const TA* __r
     float acc = 0.f;
     for (int k = 0; k < top; k++) {
       const int e = expert[(size_t)t * top + k];
+      if (e >= E) continue;
       acc += moe_warp_dot(wd + ((size_t)e * W + n) * F, md_act + k * F4, F, lane, vec);
     }
-    if (lane == 0) y[(size_t)t * ldy + n] += acc;
+    if (lane == 0) {
+      if (identity_weight) acc = fmaf(identity_weight[t], hb_to_float(xn[(size_t)t * ldx + n]), acc);
+      y[(size_t)t * ldy + n] += acc;
+    }
   }
 }
 
 HB_EXPORT int hb_moe_down_rows(const void* act, int a_dt, const void* wd, int w_dt, const int* expert, float* y, long ldy, int T,
-                               int W, int F, int top, cudaStream_t s) {
+                               int W, int F, int top, int E, const void* xn, long ldx, const float* identity_weight, cudaStream_t s) {
   if (T <= 0) return 0;
   const size_t smem = (size_t)top * ((F + 3) & ~3) * sizeof(float);
   if (smem > 200 * 1024) HB_FAIL("hb_moe_down_rows: %d x %d activations do not fit shared memory", top, F);
@@ -254,7 +288,8 @@ HB_EXPORT int hb_moe_down_rows(const void* act, int a_dt, const void* wd, int w_
   HB_DISPATCH_2(a_dt, w_dt, "hb_moe_down_rows", do {
     auto kern = moe_down_rows_kernel<TA, TB>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)act, (const TB*)wd, expert, y, ldy, W, F, top, vec);
+    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)act, (const TB*)wd, expert, y, ldy, W, F, top, vec, E,
+              (const TA*)xn, ldx, identity_weight);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_down_rows");
   return 0;
@@ -528,18 +563,19 @@ HB_EXPORT int hb_moe_sort(const int* expert, int* offsets, int* pos, int* src, i
 
 template <typename TA>
 __global__ void __launch_bounds__(128) moe_gather_kernel(const TA* __restrict__ xn, long ldx, const int* __restrict__ src,
-                                                         TA* __restrict__ xs, int W, int top) {
+                                                         TA* __restrict__ xs, int W, int top, const int* __restrict__ limit) {
   hb_pdl_launch();
   hb_pdl_wait();
+  if (limit && blockIdx.x >= *limit) return;
   const int r = blockIdx.x, t = src[r] / top;
   for (int i = threadIdx.x; i < W; i += 128) xs[(size_t)r * W + i] = xn[(size_t)t * ldx + i];
 }
 
 HB_EXPORT int hb_moe_gather(const void* xn, int x_dt, long ldx, const int* src, void* xs, int pairs, int W, int top,
-                            cudaStream_t s) {
+                            const int* limit, cudaStream_t s) {
   if (pairs <= 0) return 0;
   HB_DISPATCH_1(x_dt, "hb_moe_gather",
-                (hb_launch(moe_gather_kernel<TA>, dim3(pairs), dim3(128), 0, s, (const TA*)xn, ldx, src, (TA*)xs, W, top)));
+                (hb_launch(moe_gather_kernel<TA>, dim3(pairs), dim3(128), 0, s, (const TA*)xn, ldx, src, (TA*)xs, W, top, limit)));
   HB_CHECK_LAUNCH("hb_moe_gather");
   return 0;
 }
@@ -548,9 +584,10 @@ HB_EXPORT int hb_moe_gather(const void* xn, int x_dt, long ldx, const int* src, 
 template <typename TO>
 __global__ void __launch_bounds__(256) moe_act_kernel(const float* __restrict__ gu, const int* __restrict__ src,
                                                       const float* __restrict__ weight, TO* __restrict__ act, long n, int F,
-                                                      int at_output) {
+                                                      int at_output, const int* __restrict__ limit) {
   hb_pdl_launch();
   hb_pdl_wait();
+  if (limit) n = (long)*limit * F;
   for (long idx = (long)blockIdx.x * 256 + threadIdx.x; idx < n; idx += (long)gridDim.x * 256) {
     const long r = idx / F;
     const int j = (int)(idx - r * F);
@@ -565,10 +602,11 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const float* __restrict__ 
 template <typename TO>
 __global__ void __launch_bounds__(256) moe_act_vec_kernel(const float* __restrict__ gu, const int* __restrict__ src,
                                                           const float* __restrict__ weight, TO* __restrict__ act, long n4, int F,
-                                                          int at_output) {
+                                                          int at_output, const int* __restrict__ limit) {
   hb_pdl_launch();
   hb_pdl_wait();
   const int F4 = F >> 2;
+  if (limit) n4 = (long)*limit * F4;
   for (long idx = (long)blockIdx.x * 256 + threadIdx.x; idx < n4; idx += (long)gridDim.x * 256) {
     const long r = idx / F4;
     const int j = (int)(idx - r * F4) << 2;
@@ -582,41 +620,93 @@ __global__ void __launch_bounds__(256) moe_act_vec_kernel(const float* __restric
 }
 
 HB_EXPORT int hb_moe_act(const float* gu, const int* src, const float* weight, void* act, int o_dt, int pairs, int F,
-                         int at_output, cudaStream_t s) {
+                         int at_output, const int* limit, cudaStream_t s) {
   if (pairs <= 0) return 0;
   if (F % 4 == 0 && !(((uintptr_t)gu | (uintptr_t)act) & 15)) {
     const long n4 = (long)pairs * (F / 4);
     const int blocks4 = (int)((n4 + 255) / 256 < 148 * 16 ? (n4 + 255) / 256 : 148 * 16);
     HB_DISPATCH_1(o_dt, "hb_moe_act",
-                  (hb_launch(moe_act_vec_kernel<TA>, dim3(blocks4), dim3(256), 0, s, gu, src, weight, (TA*)act, n4, F, at_output)));
+                  (hb_launch(moe_act_vec_kernel<TA>, dim3(blocks4), dim3(256), 0, s, gu, src, weight, (TA*)act, n4, F, at_output, limit)));
     HB_CHECK_LAUNCH("hb_moe_act");
     return 0;
   }
   const long n = (long)pairs * F;
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  HB_DISPATCH_1(o_dt, "hb_moe_act", (hb_launch(moe_act_kernel<TA>, dim3(blocks), dim3(256), 0, s, gu, src, weight, (TA*)act, n, F, at_output)));
+  HB_DISPATCH_1(o_dt, "hb_moe_act", (hb_launch(moe_act_kernel<TA>, dim3(blocks), dim3(256), 0, s, gu, src, weight, (TA*)act, n, F, at_output, limit)));
   HB_CHECK_LAUNCH("hb_moe_act");
   return 0;
 }
 
+template <typename TA>
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ ys, const int* __restrict__ pos,
-                                                          float* __restrict__ y, long ldy, long n, int W, int top) {
+                                                          float* __restrict__ y, long ldy, long n, int W, int top,
+                                                          const int* __restrict__ limit, const TA* __restrict__ xn, long ldx,
+                                                          const float* __restrict__ identity_weight) {
   hb_pdl_launch();
   hb_pdl_wait();
+  const int lim = limit ? *limit : 0x7fffffff;
   for (long idx = (long)blockIdx.x * 256 + threadIdx.x; idx < n; idx += (long)gridDim.x * 256) {
     const long t = idx / W;
     const int c = (int)(idx - t * W);
     float acc = 0.f;
-    for (int k = 0; k < top; k++) acc += ys[(size_t)pos[t * top + k] * W + c];
+    for (int k = 0; k < top; k++) {
+      const int p = pos[t * top + k];
+      if (p < lim) acc += ys[(size_t)p * W + c];
+    }
+    if (identity_weight) acc = fmaf(identity_weight[t], hb_to_float(xn[t * ldx + c]), acc);
     y[t * ldy + c] += acc;
   }
 }
 
-HB_EXPORT int hb_moe_combine(const float* ys, const int* pos, float* y, long ldy, int T, int W, int top, cudaStream_t s) {
+// Four columns a thread: the same sums.
+template <typename TA>
+__global__ void __launch_bounds__(256) moe_combine_vec_kernel(const float* __restrict__ ys, const int* __restrict__ pos,
+                                                              float* __restrict__ y, long ldy, long n4, int W4, int top,
+                                                              const int* __restrict__ limit, const TA* __restrict__ xn, long ldx,
+                                                              const float* __restrict__ identity_weight) {
+  hb_pdl_launch();
+  hb_pdl_wait();
+  const int lim = limit ? *limit : 0x7fffffff;
+  for (long idx = (long)blockIdx.x * 256 + threadIdx.x; idx < n4; idx += (long)gridDim.x * 256) {
+    const long t = idx / W4;
+    const int c = (int)(idx - t * W4) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k = 0; k < top; k++) {
+      const int p = pos[t * top + k];
+      if (p >= lim) continue;
+      const float4 v = hb_load4(ys + (size_t)p * W4 * 4 + c);
+      acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    if (identity_weight) {
+      const float w = identity_weight[t];
+      const float4 v = hb_load4(xn + t * ldx + c);
+      acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
+    }
+    float4 o = hb_load4(y + t * ldy + c);
+    o.x += acc.x; o.y += acc.y; o.z += acc.z; o.w += acc.w;
+    hb_store4(y + t * ldy + c, o);
+  }
+}
+
+// limit (or null): sorted rows from *limit on belong to identity experts and hold nothing; y also gets identity_weight[t] xn[t].
+HB_EXPORT int hb_moe_combine(const float* ys, const int* pos, float* y, long ldy, int T, int W, int top, const int* limit,
+                             const void* xn, int x_dt, long ldx, const float* identity_weight, cudaStream_t s) {
   if (T <= 0) return 0;
+  if (identity_weight && !xn) HB_FAIL("hb_moe_combine: identity experts need their input rows");
+  if (W % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && !(((uintptr_t)ys | (uintptr_t)y | (uintptr_t)xn) & 15)) {
+    const long n4 = (long)T * (W / 4);
+    const int blocks4 = (int)((n4 + 255) / 256 < 148 * 16 ? (n4 + 255) / 256 : 148 * 16);
+    HB_DISPATCH_1(x_dt, "hb_moe_combine",
+                  (hb_launch(moe_combine_vec_kernel<TA>, dim3(blocks4), dim3(256), 0, s, ys, pos, y, ldy, n4, W / 4, top, limit,
+                             (const TA*)xn, ldx, identity_weight)));
+    HB_CHECK_LAUNCH("hb_moe_combine");
+    return 0;
+  }
   const long n = (long)T * W;
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  hb_launch(moe_combine_kernel, dim3(blocks), dim3(256), 0, s, ys, pos, y, ldy, n, W, top);
+  HB_DISPATCH_1(x_dt, "hb_moe_combine",
+                (hb_launch(moe_combine_kernel<TA>, dim3(blocks), dim3(256), 0, s, ys, pos, y, ldy, n, W, top, limit, (const TA*)xn, ldx,
+                           identity_weight)));
   HB_CHECK_LAUNCH("hb_moe_combine");
   return 0;
 }

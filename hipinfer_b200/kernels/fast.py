@@ -43,7 +43,8 @@ _fns = {}
 _LAUNCHES = {"hb_rows_scaled_qkv_rope": 1, "hb_rows_scaled_swiglu": 1, "hb_rows_norm_qkv_rope": 1, "hb_rows_add": 1, "hb_rows_norm_swiglu": 1, "hb_gemm_tc_rope_kv": 1, "hb_gemm_stream_finish": 1, "hb_add_rmsnorm_slices": 1, "hb_rope_kv_slices": 1, "hb_gemm_tc": 1, "hb_gemm_stream": 1, "hb_attn_decode": 1, "hb_flash_prefill": 1, "hb_flash_prefill_tc": 1}
 _status = None
 
-EPI_F32, EPI_BF16, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_SLICES, EPI_GEGLU_BF16, EPI_GELU_BF16 = 0, 1, 2, 3, 4, 5, 6
+EPI_F32, EPI_BF16, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_SLICES, EPI_GEGLU_BF16, EPI_GELU_BF16, EPI_RELU2_BF16 = 0, 1, 2, 3, 4, 5, 6, 7
+ACT_EPILOGUES = {"gelu": EPI_GELU_BF16, "relu2": EPI_RELU2_BF16}
 
 
 class KernelTimeout(RuntimeError):
@@ -287,10 +288,11 @@ def linear_gated(a, w, act_out, group, act) -> bool:
 
 
 def linear_act(a, w, out, act) -> bool:
-    """out (bf16) = act(a @ w.T), act "gelu" (the exact form), in the product's epilogue (csrc/gemm_tc.cu, gemm_stream.cu)."""
-    if act != "gelu" or out.dtype != torch.bfloat16 or not _tc_ok(a, w.t):
+    """out (bf16) = act(a @ w.T), act "gelu" (the exact form) or "relu2" (the square of relu), in the product's epilogue
+    (csrc/gemm_tc.cu, gemm_stream.cu)."""
+    if act not in ACT_EPILOGUES or out.dtype != torch.bfloat16 or not _tc_ok(a, w.t):
         return False
-    _gemm(a, w.t, out, EPI_GELU_BF16)
+    _gemm(a, w.t, out, ACT_EPILOGUES[act])
     return True
 
 

@@ -29,7 +29,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 
 # library name -> sources (relative to csrc/); headers every library depends on
 LIBRARIES: Dict[str, List[str]] = {
-    "core": ["core.cu"],
+    "core": ["core.cu", "residual_rows.cu"],
     "mixers": ["mixers_entry.cu", "delta_rule.cu", "attention_window.cu", "attention_window_flash.cu"],
     "seqmix": ["seqmix_entry.cu", "attention_masked.cu", "attention_masked_flash.cu", "attention_masked_heads.cu", "latent.cu", "gla.cu"],
     "hybrid": ["hybrid_entry.cu", "hyper_streams.cu", "ssd.cu", "moe.cu", "selective_scan.cu"],

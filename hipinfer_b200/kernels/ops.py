@@ -36,7 +36,9 @@ _SIGS = {
         "hb_layernorm": [_p, _p, _p, _i, _p, _i, _p, _i, _i, _f, _p],
         "hb_gated_act": [_p, _i, _l, _p, _i, _l, _i, _i, _i, _i, _p],
         "hb_rope_norm_store": [_p, _l, _i, _i, _i, _p, _p, _p, _i, _i, _i, _i, _f, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _p, _i,
-                               _f, _i, _f, C.c_double, _p],
+                               _f, _i, _f, C.c_double, _i, _p],
+        "hb_embed_rows": [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _l, _l, _f, _f, _p],
+        "hb_two_norms": [_p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _p],
         "hb_polynorm": [_p, _l, _p, _i, _l, _i, _i, _f, _f, _f, _f, _f, _p],
         "hb_scale_add": [_p, _p, _l, _p, _i, _i, _i, _p],
         "hb_bias_act": [_p, _l, _p, _i, _p, _i, _l, _i, _i, _i, _p],
@@ -71,14 +73,14 @@ _SIGS = {
                               _p],
         "hb_split_rounded": [_p, _l, _p, _p, _i, _i, _p],
         "hb_residual_norm": [_p, _p, _p, _p, _p, _p, _i, _f, _f, _f, _p, _f, _p, _i, _i, _i, _p],
-        "hb_moe_route": [_p, _i, _l, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _f, _p, _p, _p],
-        "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p],
-        "hb_moe_down_rows": [_p, _i, _p, _i, _p, _p, _l, _i, _i, _i, _i, _p],
+        "hb_moe_route": [_p, _i, _l, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _f, _p, _p, _i, _p, _p],
+        "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p],
+        "hb_moe_down_rows": [_p, _i, _p, _i, _p, _p, _l, _i, _i, _i, _i, _i, _p, _l, _p, _p],
         "hb_moe_sort": [_p, _p, _p, _p, _i, _i, _p],
         "hb_moe_grouped": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _i, _i, _i, _p],
-        "hb_moe_gather": [_p, _i, _l, _p, _p, _i, _i, _i, _p],
-        "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p],
-        "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p],
+        "hb_moe_gather": [_p, _i, _l, _p, _p, _i, _i, _i, _p, _p],
+        "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
+        "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p, _p, _i, _l, _p, _p],
     },
     "memory": {
         "hb_ms_walk": [_p, _l, _p, _l, _p, _l, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p],
@@ -196,6 +198,47 @@ def embedding_scaled(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tenso
     return out
 
 
+def embedding_rows(table: torch.Tensor, batch, out: torch.Tensor, scale: float = 1.0, bigram=None,
+                   norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[i] = norm(table[token] * scale + bigram row) into the float32 residual stream, the same rows once more into `copy`
+    where one is given. bigram: (table [buckets + 1, H], buckets, mul_prev, mul_cur, previous tokens int32 [slots]): the row
+    (previous * mul_prev + token * mul_cur) mod buckets, `buckets` for a sequence's first token; the previous token of a
+    portion's first row is read from the request's state slot, which is left holding the portion's last token.
+    norm_weight (float32 [H]): weight * x / sqrt(mean(x^2) + eps); absent: no norm."""
+    tokens = batch.tokens
+    _need_cuda(table, tokens, out, norm_weight, copy)
+    T, H = out.shape
+    assert out.dtype == torch.float32 and out.is_contiguous() and tokens.dtype == torch.int32 and tokens.numel() == T
+    assert table.is_contiguous() and table.shape[1] == H
+    assert norm_weight is None or (norm_weight.dtype == torch.float32 and norm_weight.numel() == H and norm_weight.is_contiguous())
+    assert copy is None or (copy.dtype == torch.float32 and copy.shape == out.shape and copy.is_contiguous())
+    bt, buckets, mp, mc, prev = bigram if bigram is not None else (None, 0, 0, 0, None)
+    if bt is not None:
+        _need_cuda(bt, prev)
+        assert bt.dtype == table.dtype and bt.is_contiguous() and bt.shape == (buckets + 1, H) and prev.dtype == torch.int32
+    _call("core", "hb_embed_rows", table.data_ptr(), _ptr(bt), _dt(table), tokens.data_ptr(), batch.positions.data_ptr(),
+          batch.row_request.data_ptr(), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_state_slot.data_ptr(),
+          _ptr(prev), _ptr(norm_weight), out.data_ptr(), _ptr(copy), T, H, int(buckets), int(mp), int(mc), float(scale), float(eps),
+          _stream())
+    return out
+
+
+def two_norms(x: torch.Tensor, w1: Optional[torch.Tensor], w2: Optional[torch.Tensor], eps: float, dtype: torch.dtype,
+              add: Optional[torch.Tensor] = None, vec: Optional[torch.Tensor] = None):
+    """x += add + vec where they are given (add float32 [T, H], vec float32 [H]), then the RMS norms of x with the weights w1
+    and w2 (float32 [H]) as rows of `dtype`, from one sum of squares: (y1, y2), None for a weight that is None."""
+    _need_cuda(x, w1, w2, add, vec)
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    for w in (w1, w2, vec):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == H and w.is_contiguous())
+    assert add is None or (add.dtype == torch.float32 and add.shape == x.shape and add.is_contiguous())
+    y1, y2 = (None if w is None else torch.empty(T, H, dtype=dtype, device=x.device) for w in (w1, w2))
+    _call("core", "hb_two_norms", x.data_ptr(), _ptr(add), _ptr(vec), _ptr(w1), _ptr(w2), _ptr(y1), _ptr(y2), _DT[dtype], T, H,
+          float(eps), _stream())
+    return y1, y2
+
+
 def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
               rows: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[i] = weight * (x[r] - mean) / sqrt(var + eps) (+ bias), r = rows[i] or i; x float32 [*, H]."""
@@ -238,14 +281,15 @@ def scale_add(x: torch.Tensor, y: torch.Tensor, scale: torch.Tensor) -> torch.Te
 
 
 def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, act: str = "none") -> torch.Tensor:
-    """out = act(x + bias) for float32 rows x (a view of some columns is fine); act "none", "tanh" or "gelu" (the exact form, z Phi(z))."""
+    """out = act(x + bias) for float32 rows x (a view of some columns is fine); act "none", "tanh", "gelu" (the exact form, z Phi(z)) or
+    "relu2" (the square of relu)."""
     _need_cuda(x, bias, out)
     _rows_contiguous(x, "bias_act in")
     _rows_contiguous(out, "bias_act out")
     assert x.dtype == torch.float32 and x.shape == out.shape
     M, n = x.shape
     _call("core", "hb_bias_act", x.data_ptr(), x.stride(0), _ptr(bias), _dt(bias) if bias is not None else 0,
-          out.data_ptr(), _dt(out), out.stride(0), M, n, {"none": 0, "tanh": 1, "gelu": 2}[act], _stream())
+          out.data_ptr(), _dt(out), out.stride(0), M, n, {"none": 0, "tanh": 1, "gelu": 2, "relu2": 3}[act], _stream())
     return out
 
 
@@ -782,7 +826,7 @@ def linear_gated(a: torch.Tensor, w_gate_up: "Weight", act_out: torch.Tensor, gr
 
 
 def linear_act(a: torch.Tensor, w: "Weight", out: torch.Tensor, act: str) -> torch.Tensor:
-    """out = act(a @ w.T), act "gelu" (the exact form): the activation in the product's epilogue where one takes these
+    """out = act(a @ w.T), act "gelu" (the exact form) or "relu2" (the square of relu): the activation in the product's epilogue where one takes these
     sizes, else the product's 32-bit rows through `bias_act`."""
     from . import fast
 
@@ -847,14 +891,16 @@ def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_m
                     table: torch.Tensor, rot: int, pairing: str, unit_norm: bool, eps: float, q_out: torch.Tensor,
                     k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], n_heads: int, n_kv_heads: int,
                     dim: int, vdim: int, page_size: int, rot_off: int = 0, row_norm=None, row_norm_eps: float = 0.0,
-                    head_norm=None, q_temp=None) -> torch.Tensor:
+                    head_norm=None, q_temp=None, maps: int = 1) -> torch.Tensor:
     """From a float32 projection result whose rows hold q, k, v at the column `offsets` (q, k, v): q and k rotated on
     the `rot` dimensions from `rot_off` on (pairing "half": (i, i + rot/2); "interleaved": (2i, 2i + 1)) and, with unit_norm,
     divided by their root mean square over `dim`; q to q_out [T, n_heads * dim], k and v (vdim wide, raw) to their page
     slots. slot_map None: q alone. row_norm (wq [n_heads * dim], wk [n_kv_heads * dim]): before the rotation the whole
     q row and the whole k row are divided by their root mean square (row_norm_eps inside the root) and multiplied by the
     weights, column by column. head_norm (wq [dim], wk [dim]) instead: each head by itself, with weights the heads share.
-    q_temp (coef, every): q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    q_temp (coef, every): q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1). maps > 1: heads with
+    several score maps; n_heads and n_kv_heads count every map's (side by side in the projection's rows), a kv head's maps lie
+    side by side in its key row, [page, n_kv_heads / maps, page_size, maps * dim], and there are n_kv_heads / maps values."""
     _need_cuda(proj, positions, slot_map, table, q_out, k_cache, v_cache)
     _rows_contiguous(proj, "rope_norm_store in")
     T = proj.shape[0]
@@ -862,7 +908,7 @@ def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_m
     assert table.dtype == torch.float32 and table.is_contiguous() and table.shape[1] * 2 == rot
     if slot_map is not None:
         assert k_cache.dtype == v_cache.dtype == q_out.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
-        assert k_cache.shape[-1] == dim and v_cache.shape[-1] == vdim
+        assert k_cache.shape[-1] == maps * dim and v_cache.shape[-1] == vdim and k_cache.shape[1] * maps == n_kv_heads
     q_off, k_off, v_off = (int(o) for o in offsets)
     assert row_norm is None or head_norm is None
     per_head = head_norm is not None
@@ -876,7 +922,8 @@ def rope_norm_store(proj: torch.Tensor, offsets, positions: torch.Tensor, slot_m
           _ptr(slot_map), table.data_ptr(), int(rot), int(rot_off), PAIRINGS[pairing], 1 if unit_norm else 0, float(eps), q_out.data_ptr(),
           _ptr(k_cache) if slot_map is not None else None, _ptr(v_cache) if slot_map is not None else None, _dt(q_out), T,
           n_heads, n_kv_heads, dim, vdim, page_size, _ptr(wq_pre), _ptr(wk_pre), _dt(wq_pre) if wq_pre is not None else 0,
-          float(row_norm_eps), 1 if per_head else 0, float(coef), float(every), _stream())
+          float(row_norm_eps), 1 if per_head else 0, float(coef), float(every), int(maps),
+          _stream())
     return q_out
 
 
@@ -1338,19 +1385,24 @@ def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, pair: Optio
     return x
 
 
-MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "sigmoid_normed": 2}
+MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "sigmoid_normed": 2, "softmax": 3}
 
 
 def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[torch.Tensor] = None, score: str = "sigmoid",
               correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
-              shared_gate: Optional[torch.Tensor] = None, shared_weight: Optional[torch.Tensor] = None):
+              shared_gate: Optional[torch.Tensor] = None, shared_weight: Optional[torch.Tensor] = None, identity: int = 0,
+              identity_weight: Optional[torch.Tensor] = None):
     """(expert int32 [T, top], weight float32 [T, top]): the `top` experts with the largest z = router @ row (+ bias), 32-bit
     sums; the largest first, ties to the lower index. score "sigmoid": the weights are sigmoid(z) of the chosen ones;
     "softmax_chosen": the softmax over the chosen logits alone. "sigmoid_normed": sigmoid(z) + correction chooses, with
     groups > 1 only among the experts of the `keep` groups (of neighbours) whose two largest sums are largest; the weights are
-    the chosen sigmoid(z), without the correction, over their sum (+ 1e-20), times scale. shared_gate [1, W] or [W]: also
+    the chosen sigmoid(z), without the correction, over their sum (+ 1e-20), times scale. "softmax": softmax(z) over all +
+    correction chooses, with groups > 1 only among the experts of the groups whose largest is largest; the weights are the
+    chosen softmax(z). The last `identity` router rows are identity experts: identity_weight[t] (float32 [T]) = the sum of the
+    weights of the chosen ones. shared_gate [1, W] or [W]: also
     shared_weight[t] (float32 [T]) = sigmoid(shared_gate . row)."""
-    _need_cuda(xn, router, bias, correction, shared_gate, shared_weight)
+    _need_cuda(xn, router, bias, correction, shared_gate, shared_weight, identity_weight)
+    assert not identity or (identity_weight.dtype == torch.float32 and identity_weight.numel() == xn.shape[0])
     assert correction is None or (correction.dtype == router.dtype and correction.numel() == router.shape[0] and correction.is_contiguous())
     assert shared_gate is None or (shared_gate.dtype == router.dtype and shared_gate.numel() == router.shape[1]
                                    and shared_weight.dtype == torch.float32 and shared_weight.numel() == xn.shape[0])
@@ -1362,16 +1414,17 @@ def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[t
     weight = torch.empty(T, top, dtype=torch.float32, device=xn.device)
     _call("hybrid", "hb_moe_route", xn.data_ptr(), _dt(xn), xn.stride(0), router.data_ptr(), _ptr(bias), _dt(router),
           expert.data_ptr(), weight.data_ptr(), T, W, E, int(top), MOE_SCORES[score], _ptr(correction), int(groups), int(keep), float(scale),
-          _ptr(shared_gate), _ptr(shared_weight), _stream())
+          _ptr(shared_gate), _ptr(shared_weight), E - int(identity), _ptr(identity_weight) if identity else None, _stream())
     return expert, weight
 
 
 def moe_rows(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor, expert: torch.Tensor, score: torch.Tensor,
-             y: torch.Tensor, at_output: bool = False) -> torch.Tensor:
+             y: torch.Tensor, at_output: bool = False, identity_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y += sum over a row's chosen experts of Wd_e (silu(s Wg_e h) * (s Wu_e h)), row by row with nothing sorted and
     nothing on the host. wgu [E, 2F, W] (gate rows, then up rows), wdown [E, W, F], y float32 [T, W]. at_output: the
-    weight multiplies the expert's result instead of its input, Wd_e (s silu(Wg_e h) * (Wu_e h))."""
-    _need_cuda(xn, wgu, wdown, expert, score, y)
+    weight multiplies the expert's result instead of its input, Wd_e (s silu(Wg_e h) * (Wu_e h)). Choices from E on are
+    identity experts: y also gets identity_weight[t] * xn[t]."""
+    _need_cuda(xn, wgu, wdown, expert, score, y, identity_weight)
     _rows_contiguous(xn, "moe_rows in")
     _rows_contiguous(y, "moe_rows out")
     T, top = expert.shape
@@ -1380,9 +1433,9 @@ def moe_rows(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor, expert: t
     assert wgu.is_contiguous() and wdown.is_contiguous() and wdown.shape == (E, W, F) and y.dtype == torch.float32
     act = torch.empty(T * top, F, dtype=xn.dtype, device=xn.device)
     _call("hybrid", "hb_moe_gate_up_rows", xn.data_ptr(), _dt(xn), xn.stride(0), wgu.data_ptr(), _dt(wgu), expert.data_ptr(),
-          score.data_ptr(), act.data_ptr(), T, W, F, top, 1 if at_output else 0, _stream())
+          score.data_ptr(), act.data_ptr(), T, W, F, top, 1 if at_output else 0, E, _stream())
     _call("hybrid", "hb_moe_down_rows", act.data_ptr(), _dt(act), wdown.data_ptr(), _dt(wdown), expert.data_ptr(), y.data_ptr(),
-          y.stride(0), T, W, F, top, _stream())
+          y.stride(0), T, W, F, top, E, xn.data_ptr(), xn.stride(0), _ptr(identity_weight), _stream())
     return y
 
 
@@ -1403,42 +1456,48 @@ def moe_grouped(a: torch.Tensor, src: Optional[torch.Tensor], top: int, w: torch
                 out: torch.Tensor) -> torch.Tensor:
     """out[r] = w[e] a[row(r)] for the sorted rows r of every expert e (offsets[e] <= r < offsets[e + 1]); row(r) is
     src[r] // top where src is given (the step's input rows), else r. w [E, Nout, K]; out float32 [sorted rows, Nout].
-    An expert's weights are read once for all of its rows; nothing is read by the host."""
+    An expert's weights are read once for all of its rows; nothing is read by the host. Sorted rows of experts beyond E
+    (identity experts) are left alone."""
     _need_cuda(a, w, offsets, out)
     _rows_contiguous(a, "moe_grouped in")
     E, Nout, K = w.shape
     assert w.is_contiguous() and a.shape[1] == K and out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == Nout
-    assert offsets.numel() == E + 1 and offsets.dtype == torch.int32 and (src is None or src.dtype == torch.int32)
+    assert offsets.numel() >= E + 1 and offsets.dtype == torch.int32 and (src is None or src.dtype == torch.int32)
     _call("hybrid", "hb_moe_grouped", a.data_ptr(), _dt(a), a.stride(0), _ptr(src), int(top), w.data_ptr(), _dt(w),
           offsets.data_ptr(), out.data_ptr(), E, Nout, K, _stream())
     return out
 
 
-def moe_gather(xn: torch.Tensor, src: torch.Tensor, top: int) -> torch.Tensor:
-    """The input rows in sorted order: out[r] = xn[src[r] // top]."""
+def moe_gather(xn: torch.Tensor, src: torch.Tensor, top: int, limit: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The input rows in sorted order: out[r] = xn[src[r] // top]. limit (int32 [1] on the device): only rows below it."""
     _rows_contiguous(xn, "moe_gather in")
     out = torch.empty(src.numel(), xn.shape[1], dtype=xn.dtype, device=xn.device)
     _call("hybrid", "hb_moe_gather", xn.data_ptr(), _dt(xn), xn.stride(0), src.data_ptr(), out.data_ptr(), src.numel(),
-          xn.shape[1], int(top), _stream())
+          xn.shape[1], int(top), _ptr(limit), _stream())
     return out
 
 
-def moe_act(gu: torch.Tensor, src: torch.Tensor, score: torch.Tensor, out: torch.Tensor, at_output: bool = False) -> torch.Tensor:
+def moe_act(gu: torch.Tensor, src: torch.Tensor, score: torch.Tensor, out: torch.Tensor, at_output: bool = False,
+            limit: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[r] = silu(s g) * (s u) of the sorted rows' float32 [g | u], s the score of the row's pair; with at_output
-    s silu(g) * u (the weight of the expert's result, brought in before the linear down product)."""
+    s silu(g) * u (the weight of the expert's result, brought in before the linear down product). limit (int32 [1] on the
+    device): only rows below it."""
     pairs, F = out.shape
     assert gu.dtype == torch.float32 and gu.is_contiguous() and gu.shape == (pairs, 2 * F) and out.is_contiguous()
     _call("hybrid", "hb_moe_act", gu.data_ptr(), src.data_ptr(), score.data_ptr(), out.data_ptr(), _dt(out), pairs, F,
-          1 if at_output else 0, _stream())
+          1 if at_output else 0, _ptr(limit), _stream())
     return out
 
 
-def moe_combine(ys: torch.Tensor, pos: torch.Tensor, y: torch.Tensor, top: int) -> torch.Tensor:
-    """y[t] += the sorted results of row t's choices, added in the order of the choices."""
+def moe_combine(ys: torch.Tensor, pos: torch.Tensor, y: torch.Tensor, top: int, limit: Optional[torch.Tensor] = None,
+                xn: Optional[torch.Tensor] = None, identity_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[t] += the sorted results of row t's choices, added in the order of the choices. With identity experts: the sorted rows
+    from limit (int32 [1] on the device) on are theirs and hold nothing, and y[t] += identity_weight[t] * xn[t]."""
     _rows_contiguous(y, "moe_combine out")
     T, W = y.shape
     assert ys.dtype == y.dtype == torch.float32 and ys.is_contiguous() and ys.shape == (T * top, W)
-    _call("hybrid", "hb_moe_combine", ys.data_ptr(), pos.data_ptr(), y.data_ptr(), y.stride(0), T, W, int(top), _stream())
+    _call("hybrid", "hb_moe_combine", ys.data_ptr(), pos.data_ptr(), y.data_ptr(), y.stride(0), T, W, int(top), _ptr(limit), _ptr(xn),
+          _dt(xn) if xn is not None else 0, xn.stride(0) if xn is not None else 0, _ptr(identity_weight), _stream())
     return y
 
 

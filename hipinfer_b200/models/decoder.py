@@ -19,6 +19,9 @@ from ..parts.registry import BuildContext, build_part
 from ..parts.spec import ModelSpec, PartSpec
 
 
+EMBEDDING_STATE = -1      # where the embedding's per-request state is kept, beside the run order's indices
+
+
 @dataclass(frozen=True)
 class StepCachePlan:
     group: int   # cache group of the step's mixer
@@ -47,6 +50,8 @@ class DecoderModel:
         self.layers = [build_part("block", PartSpec(ls.block, {**ls.params, "layer": ls}), ctx, ls.prefix) for ls in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm, ctx)
         self.head = build_part("head", spec.head, ctx)
+        self.pass_entry = build_part("pass_entry", spec.pass_entry, ctx) if spec.pass_entry is not None else None
+        self.parts = [self.embedding] + self.layers + [self.final_norm, self.head] + ([self.pass_entry] if self.pass_entry else [])
         self._plan_cache()
 
     # ---------------------------------------------------------------- what the cache must provide
@@ -55,6 +60,8 @@ class DecoderModel:
         counts: List[int] = []
         self.cache_plan: List[Optional[StepCachePlan]] = []
         self.state_specs: Dict[Tuple[int, str], Tuple[Tuple[int, ...], torch.dtype]] = {}
+        for name, (shape, dtype) in getattr(self.embedding, "state_need", dict)().items():
+            self.state_specs[(EMBEDDING_STATE, name)] = (tuple(shape), dtype)
         for i, st in enumerate(self.spec.order):
             mixer = self.layers[st.layer].mixer
             need = mixer.cache_need()
@@ -86,7 +93,7 @@ class DecoderModel:
     # ---------------------------------------------------------------- weights
     def param_specs(self):
         seen, out = set(), []
-        for part in [self.embedding] + self.layers + [self.final_norm, self.head]:
+        for part in self.parts:
             for s in part.param_specs():
                 if s.name not in seen:
                     seen.add(s.name)
@@ -94,7 +101,7 @@ class DecoderModel:
         return out
 
     def load(self, tensors) -> None:
-        for part in [self.embedding] + self.layers + [self.final_norm, self.head]:
+        for part in self.parts:
             part.load(tensors)
 
     def step_weight_bytes(self) -> int:
@@ -107,15 +114,24 @@ class DecoderModel:
     # ---------------------------------------------------------------- forward
     def forward(self, batch, storage) -> torch.Tensor:
         """Run the batch's tokens from the cache; logits float32 [len(batch.want_rows), vocab]."""
-        if getattr(self.embedding, "takes_positions", False):
+        order = self.spec.order
+        # a pass after the first starts with the embedding rows added once more: they are kept for it
+        again = self.pass_entry is not None and any((st.enters_pass or 0) > 0 for st in order)
+        first = None
+        if getattr(self.embedding, "takes_batch", False):
+            if again:
+                first = torch.empty(batch.tokens.numel(), self.spec.hidden_size, dtype=torch.float32, device=batch.tokens.device)
+            x = self.embedding.forward(batch, storage.layer_state(EMBEDDING_STATE), copy=first)
+        elif getattr(self.embedding, "takes_positions", False):
             x = self.embedding.forward(batch.tokens, batch.positions)
         else:
             x = self.embedding.forward(batch.tokens)
+        if again and first is None:
+            first = x.clone()
         planes.record(batch, "embedding", x)
         # what a layer leaves for the next reader of x: a sum not yet added (kernels.ops.Pending: the next norm adds
         # it), or that next norm already prepared by the layer's last product (kernels.fast.NormFeed); else None
         carry = None
-        order = self.spec.order
         keeps = any(getattr(layer, "takes_history", False) for layer in self.layers)
         history = DepthHistory(len(order) + 1, x) if keeps else None
         for i, st in enumerate(order):
@@ -128,7 +144,15 @@ class DecoderModel:
             kw = {}
             if carry is not None:
                 kw["pending"] = carry
-            if getattr(layer, "takes_next_norm", False) and i + 1 < len(order):
+            if st.enters_pass is not None:
+                if isinstance(carry, ops.Pending):
+                    carry.finish()
+                kw.pop("pending", None)
+                if getattr(layer, "takes_entry", False):
+                    kw["entry"] = self.pass_entry.addends(first, st.enters_pass)
+                else:
+                    self.pass_entry.forward(x, first, st.enters_pass)
+            if getattr(layer, "takes_next_norm", False) and i + 1 < len(order) and order[i + 1].enters_pass is None:
                 kw["next_norm"] = getattr(self.layers[order[i + 1].layer], "mixer_norm", None)
             if history is not None:
                 if getattr(layer, "takes_history", False):

@@ -218,6 +218,85 @@ class ParallelBlock(Part):
         return None
 
 
+class ParallelTwoNormBlock(Part):
+    """Two norms of the same rows, one reader each: x <- x + (mixer(norm1(x)) + feed_forward(norm2(x))). The norms are one pass
+    over the row (one sum of squares, two weights), which also adds what a pass of looped layers starts with (`entry`); both
+    sublayers then add into the 32-bit residual stream. The feed-forward with its norm is optional. Norms of another kind than
+    the RMS norm, or with different eps, are run one by one.
+
+    params: layer (the LayerSpec)."""
+
+    SLOTS = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
+    OPTIONAL = ("feed_forward_norm", "feed_forward")
+    takes_entry = True      # forward() accepts entry=(rows or None, vector): added to x before the norms
+
+    def __init__(self, params, ctx, prefix=""):
+        super().__init__(params, ctx, prefix)
+        layer = params["layer"]
+        has_ff = "feed_forward" in layer.parts
+        self.parts = build_slots(self, layer, {n: r for n, r in self.SLOTS.items() if has_ff or n not in self.OPTIONAL}, ctx, prefix)
+        if not has_ff:
+            self.feed_forward = self.feed_forward_norm = None
+        self.weights = None
+
+    def param_specs(self):
+        return [s for p in self.parts for s in p.param_specs()]
+
+    def load(self, tensors):
+        for p in self.parts:
+            p.load(tensors)
+        norms = [n for n in (self.mixer_norm, self.feed_forward_norm) if n is not None]
+        if all(isinstance(n, RMSNorm) and n.eps == norms[0].eps for n in norms):
+            self.weights = [n.weight.to(torch.float32).contiguous() for n in norms] + [None] * (2 - len(norms))
+
+    def weight_bytes(self):
+        return sum(p.weight_bytes() for p in self.parts)
+
+    def _norms(self, x, entry):
+        if self.weights is not None:
+            return ops.two_norms(x, self.weights[0], self.weights[1], self.mixer_norm.eps, self.ctx.dtype, *(entry or (None, None)))
+        if entry is not None:
+            ops.two_norms(x, None, None, 0.0, self.ctx.dtype, *entry)
+        return self.mixer_norm.forward(x), None if self.feed_forward_norm is None else self.feed_forward_norm.forward(x)
+
+    def forward(self, x, batch, cache, state, entry=None):
+        h1, h2 = self._norms(x, entry)
+        planes.record(batch, "mixer_norm", h1)
+        left = self.mixer.forward(h1, x, batch, cache, state)
+        if isinstance(left, ops.Pending):
+            left.finish()
+        planes.record(batch, "after_mixer", x)
+        if self.feed_forward is not None:
+            planes.record(batch, "feed_forward_norm", h2)
+            left = self.feed_forward.forward(h2, x, batch)
+            if isinstance(left, ops.Pending):
+                left.finish()
+        planes.record(batch, "after_feed_forward", x)
+        return None
+
+
+class LoopEntry(Part):
+    """What is added to the residual stream ahead of pass t of layers that run several times in a row: a vector step[t], and
+    from the second pass on the embedding rows. params: name (a tensor [passes, hidden_size]), passes, hidden_size."""
+
+    def __init__(self, params, ctx, prefix=""):
+        super().__init__(params, ctx, prefix)
+        self.name, self.passes, self.hidden = prefix + params["name"], int(params["passes"]), int(params["hidden_size"])
+        self.step = None
+
+    def param_specs(self):
+        return [ParamSpec(self.name, (self.passes, self.hidden))]
+
+    def load(self, tensors):
+        self.step = tensors[self.name].to(torch.float32).contiguous()
+
+    def addends(self, first, t):
+        return first if t > 0 else None, self.step[t]
+
+    def forward(self, x, first, t):
+        ops.two_norms(x, None, None, 0.0, torch.float32, *self.addends(first, t))
+
+
 class PreparedNorm:
     """The rows of `norm` over the residual rows as a layer left them: the layer's last write-back computed them on its
     way, so the layer that owns `norm` need not read the residual rows again."""
@@ -512,5 +591,7 @@ register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "post_norm", PostNormBlock)
 register_part("block", "parallel", ParallelBlock)
+register_part("block", "parallel_two_norms", ParallelTwoNormBlock)
+register_part("pass_entry", "loop", LoopEntry)
 register_part("block", "pre_norm_scaled", ScaledPreNormBlock)
 register_part("block", "hyper_connections", HyperConnectionBlock)

@@ -3,7 +3,9 @@
 A head has TWO score maps: its query is [map 1 (dim) | map 2 (dim)] and so are the keys of its kv head (query head h
 reads kv head h // (heads / kv_heads)); both maps are ordinary softmax attention over the same values (vdim wide):
 
-    q, k, v = Wq h + bq, Wk h + bk, Wv h + bv          no position encoding: positions enter through the mask alone
+    q, k, v = Wq h + bq, Wk h + bk, Wv h + bv          (the biases by choice)
+    q, k rotated on the first `rot_dims` dimensions of each map (pairs (i, i + rot_dims / 2)); 0: no position encoding,
+        positions enter through the mask alone
     a_m = softmax(scale * q_m k_m^T over the visible keys) v,   m = 1, 2
     o = a_1 - lambda * a_2,   lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff      (one number for the layer)
     o <- o / sqrt(mean(o^2) + eps) * (1 - diff)        over the head's vdim values, no weight
@@ -16,10 +18,10 @@ model's run order names. What the cache retains is given apart from the mask (`c
 because the layers that share a cache may look back differently far: the model gives all of them the widest.
 
 lambda depends on the weights alone and is computed when they are loaded. Scores, softmax, the combination and the
-head norm are 32-bit (csrc/attention_window.cu); q, k, v are rounded once, after their bias.
+head norm are 32-bit (csrc/attention_window.cu); q, k, v are rounded once, after their bias and rotation.
 
 params: hidden_size, heads, kv_heads, dim, vdim, scale, diff, eps, window (None or 0: none), keep_first, cache_window,
-cache_keep_first, reads_cache, and tensor names (`<key>_name`): q, k, v, g, o, q_bias, k_bias, v_bias, lq1, lk1, lq2, lk2.
+cache_keep_first, reads_cache, biases (default True), rot_dims, rot_base, rot_scaling (ops.rope_frequencies), and tensor names (`<key>_name`): q, k, v, g, o, q_bias, k_bias, v_bias, lq1, lk1, lq2, lk2.
 With `out_scale=` the output projection's result is multiplied by that vector before it is added into the residual stream.
 """
 from __future__ import annotations
@@ -55,6 +57,15 @@ class DifferentialAttentionMixer(Mixer):
         if self.cache_window and (not self.window or self.window > self.cache_window or self.keep_first > self.cache_keep_first):
             raise ValueError("differential attention: the cache retains less than the mask sees")
         self.reads_cache = bool(p.get("reads_cache", False))
+        self.biases = bool(p.get("biases", True))
+        self.rot_dims, self.rot_base = int(p.get("rot_dims") or 0), float(p.get("rot_base") or 10000.0)
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
+            raise ValueError(f"differential attention: {self.rot_dims} rotated dimensions of a map of {self.dim}")
+        if self.rot_dims and self.biases:
+            raise ValueError("differential attention: a rotation of queries and keys with biases is not implemented")
+        self.table = None
+        if not ctx.is_meta and not self.biases:
+            self.table = ops.shared_rope_table(self.rot_dims, self.rot_base, ctx.max_model_len, ctx.device, p.get("rot_scaling"))
         self.names = {k: prefix + p.get(k + "_name", d) for k, d in _DEFAULT_NAMES.items()}
         self.w_in = self.wo = None
         self.lam = 0.0
@@ -69,11 +80,12 @@ class DifferentialAttentionMixer(Mixer):
 
     def param_specs(self):
         n, W = self.names, self.hidden
-        specs = [ParamSpec(n["q"], (self.n_q, W)), ParamSpec(n["q_bias"], (self.n_q,), init="zeros")]
-        if not self.reads_cache:
-            specs += [ParamSpec(n["k"], (self.n_k, W)), ParamSpec(n["k_bias"], (self.n_k,), init="zeros"),
-                      ParamSpec(n["v"], (self.kv_heads * self.vdim, W)),
-                      ParamSpec(n["v_bias"], (self.kv_heads * self.vdim,), init="zeros")]
+        rows = [("q", self.n_q)] + ([] if self.reads_cache else [("k", self.n_k), ("v", self.kv_heads * self.vdim)])
+        specs = []
+        for key, size in rows:
+            specs.append(ParamSpec(n[key], (size, W)))
+            if self.biases:
+                specs.append(ParamSpec(n[key + "_bias"], (size,), init="zeros"))
         specs += [ParamSpec(n[k], (self.dim,)) for k in ("lq1", "lk1", "lq2", "lk2")]
         specs += [ParamSpec(n["g"], (self.heads * self.vdim, W)), ParamSpec(n["o"], (W, self.heads * self.vdim))]
         return specs
@@ -84,10 +96,12 @@ class DifferentialAttentionMixer(Mixer):
         dt = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
         self.w_in = ops.Weight(torch.cat([m.to(dt) for m in mats], 0).contiguous())     # rows [q | k | v | g] or [q | g]
         self.wo = ops.Weight(t["o"])
-        bdt = t["q_bias"].dtype
-        self.bq = t["q_bias"]
-        self.bk = None if self.reads_cache else t["k_bias"].to(bdt)
-        self.bv = None if self.reads_cache else t["v_bias"].to(bdt)
+        self.bq = self.bk = self.bv = None
+        if self.biases:
+            bdt = t["q_bias"].dtype
+            self.bq = t["q_bias"]
+            self.bk = None if self.reads_cache else t["k_bias"].to(bdt)
+            self.bv = None if self.reads_cache else t["v_bias"].to(bdt)
         dot = lambda a, b: float((t[a].double().cpu() * t[b].double().cpu()).sum())
         self.lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.diff
 
@@ -105,11 +119,17 @@ class DifferentialAttentionMixer(Mixer):
         T = xn.shape[0]
         n_kv = 0 if self.reads_cache else self.n_k + self.kv_heads * self.vdim
         proj = torch.empty(T, self.n_q + n_kv + self.heads * self.vdim, dtype=torch.float32, device=xn.device)
-        ops.linear(xn, self.w_in, proj)
+        ops.linear_rows32(xn, self.w_in, proj)
         q = torch.empty(T, self.n_q, dtype=self.ctx.dtype, device=xn.device)
         write = cache.write and not self.reads_cache
-        ops.qkv_bias_store(proj[:, :self.n_q + n_kv], self.bq, self.bk, self.bv, batch.slot_maps[cache.group] if write else None,
-                           q, cache.k, cache.v, self.n_q, self.kv_heads, self.MAPS * self.dim, self.vdim, self.ctx.page_size)
+        slot_map = batch.slot_maps[cache.group] if write else None
+        if self.biases:
+            ops.qkv_bias_store(proj[:, :self.n_q + n_kv], self.bq, self.bk, self.bv, slot_map, q, cache.k, cache.v, self.n_q,
+                               self.kv_heads, self.MAPS * self.dim, self.vdim, self.ctx.page_size)
+        else:
+            ops.rope_norm_store(proj, (0, self.n_q, self.n_q + self.n_k), batch.positions, slot_map, self.table, self.rot_dims, "half",
+                                False, 0.0, q, cache.k, cache.v, self.heads * self.MAPS, self.kv_heads * self.MAPS, self.dim,
+                                self.vdim, self.ctx.page_size, maps=self.MAPS)
         att = torch.empty(T, self.heads * self.vdim, dtype=self.ctx.dtype, device=xn.device)
         ops.attention_window(q, cache.k, cache.v, batch, cache.group, att, self.heads, self.kv_heads, self.dim, self.vdim,
                              self.MAPS, self.ctx.page_size, self.window, self.keep_first, self.scale, self.lam,
@@ -117,7 +137,7 @@ class DifferentialAttentionMixer(Mixer):
         planes.record(batch, "q", q)
         planes.record(batch, "attention", att)
         if out_scale is None:
-            ops.linear(att, self.wo, x, accumulate=True)
+            ops.linear_into_stream(att, self.wo, x)
         else:
             ops.linear_scaled_add(att, self.wo, x, out_scale)
         return None

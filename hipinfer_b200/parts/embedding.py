@@ -7,6 +7,7 @@ import torch
 
 from ..kernels import ops
 from ..weights import ParamSpec
+from .norm import RMSNorm
 from .registry import Part, build_part, register_part, to_compute
 
 
@@ -84,6 +85,53 @@ class NormedTokenEmbedding(Part):
         return self.norm.forward(raw, out=torch.empty_like(raw))
 
 
+class BigramTokenEmbedding(Part):
+    """x = norm(table[token] * scale + bigram[row]): a scaled token embedding, a second table addressed by the token and the one
+    before it, and a norm whose result stays 32-bit. The row is (previous * mul_prev + token * mul_cur) mod buckets, and row
+    `buckets` (the last) for a sequence's first token. The previous token is state of the request: a step's first row of a
+    request finds it in the request's slot. All of it is one kernel (csrc/residual_rows.cu).
+
+    params: name, vocab_size, hidden_size, scale (default 1), bigram (buckets, mul_prev, mul_cur) or None, bigram_name (default
+    "bigram"), norm (the PartSpec of an RMS norm over hidden_size) or None."""
+
+    takes_batch = True
+
+    def __init__(self, params, ctx, prefix=""):
+        super().__init__(params, ctx, prefix)
+        self.name, self.vocab, self.hidden = params["name"], int(params["vocab_size"]), int(params["hidden_size"])
+        self.scale = float(params.get("scale", 1.0))
+        self.bigram = tuple(int(v) for v in params["bigram"]) if params.get("bigram") else None
+        if self.bigram and (self.bigram[0] < 1 or min(self.bigram[1:]) < 0):
+            raise ValueError(f"bigram embedding: {self.bigram[0]} buckets, multipliers {self.bigram[1:]}")
+        self.bigram_name = params.get("bigram_name", "bigram")
+        self.norm = build_part("norm", params["norm"], ctx, prefix) if params.get("norm") else None
+        if self.norm is not None and not isinstance(self.norm, RMSNorm):
+            raise ValueError("bigram embedding: the norm must be an RMS norm")
+        self.table = self.bigram_table = self.norm_weight = None
+
+    def param_specs(self):
+        specs = [ParamSpec(self.name, (self.vocab, self.hidden))]
+        if self.bigram:
+            specs.append(ParamSpec(self.bigram_name, (self.bigram[0] + 1, self.hidden)))
+        return specs + (self.norm.param_specs() if self.norm else [])
+
+    def state_need(self):
+        return {"previous": ((), torch.int32)} if self.bigram else {}
+
+    def load(self, tensors):
+        self.table = to_compute(tensors[self.name], self.ctx)
+        if self.bigram:
+            self.bigram_table = to_compute(tensors[self.bigram_name], self.ctx).to(self.table.dtype)
+        if self.norm:
+            self.norm.load(tensors)
+            self.norm_weight = self.norm.weight.to(torch.float32).contiguous()
+
+    def forward(self, batch, state, copy=None):
+        x = torch.empty(batch.tokens.numel(), self.hidden, dtype=torch.float32, device=batch.tokens.device)
+        bigram = (self.bigram_table, *self.bigram, state["previous"]) if self.bigram else None
+        return ops.embedding_rows(self.table, batch, x, self.scale, bigram, self.norm_weight, self.norm.eps if self.norm else 0.0, copy)
+
+
 class StreamsTokenEmbedding(Part):
     """A token embedding into `streams` residual streams: every token's row of the 32-bit stream tensor holds `streams`
     copies of its embedding, [T, streams * hidden_size]. params: name, vocab_size, hidden_size, streams."""
@@ -142,5 +190,6 @@ class LMHead(Part):
 register_part("embedding", "token", TokenEmbedding)
 register_part("embedding", "token_position", ScaledPositionEmbedding)
 register_part("embedding", "token_normed", NormedTokenEmbedding)
+register_part("embedding", "token_bigram", BigramTokenEmbedding)
 register_part("embedding", "token_streams", StreamsTokenEmbedding)
 register_part("head", "linear", LMHead)

@@ -108,8 +108,8 @@ class GatedFF(Part):
 
 
 class ActivatedFF(Part):
-    """A dense feed-forward without a gate and without biases: out = Wdown act(Wup h), act "gelu" (the exact form, z Phi(z)),
-    computed on the product's 32-bit result and rounded once.
+    """A dense feed-forward without a gate and without biases: out = Wdown act(Wup h), act "gelu" (the exact form, z Phi(z))
+    or "relu2" (the square of relu), computed on the product's 32-bit result and rounded once.
 
     params: hidden_size, intermediate_size, activation (default "gelu"), up_name, down_name."""
 
@@ -117,8 +117,8 @@ class ActivatedFF(Part):
         super().__init__(params, ctx, prefix)
         self.hidden, self.inter = int(params["hidden_size"]), int(params["intermediate_size"])
         self.act = params.get("activation", "gelu")
-        if self.act != "gelu":
-            raise ValueError(f"feed-forward: activation {self.act!r} is not known (known: 'gelu')")
+        if self.act not in ("gelu", "relu2"):
+            raise ValueError(f"feed-forward: activation {self.act!r} is not known (known: 'gelu', 'relu2')")
         self.names = {k: prefix + params.get(k + "_name", f"mlp.{k}") for k in ("up", "down")}
         self.wup = self.wdown = None
 

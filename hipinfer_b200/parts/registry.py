@@ -15,7 +15,10 @@ Interfaces (duck-typed; the base classes below give the defaults):
                   {name: tensor [slots, *shape]} it declared (index with batch.req_state_slot)
   feed_forward    forward(xn, x, batch): adds its output into x
   block           forward(x, batch, cache, state): one layer in its arrangement
-  embedding       forward(tokens int32 [T]) -> x float32 [T, H]
+  embedding       forward(tokens int32 [T]) -> x float32 [T, H]; with `takes_batch` forward(batch, state, copy=None), where
+                  state holds what its state_need() declared (as a mixer's) and copy, if given, gets the same rows once more
+  pass_entry      forward(x, first, t): what is added to x ahead of pass t of layers that run several times, `first` being the
+                  embedding rows; addends(first, t) -> (rows or None, vector): the same for a block that adds them itself
   head            forward(xn [W, H]) -> logits float32 [W, V]
 """
 from __future__ import annotations
@@ -90,7 +93,7 @@ class Mixer(Part):
 
 
 _REGISTRIES: Dict[str, Dict[str, Callable]] = {k: {} for k in
-                                               ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head")}
+                                               ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "pass_entry")}
 
 
 def register_part(role: str, kind: str, cls: Callable) -> None:

@@ -14,6 +14,11 @@ A third: `score` "sigmoid_normed" chooses by sigmoid(z) + a correction per exper
 only within the `keep` groups of neighbouring experts that rank best by the sum of their two largest; the weights are the
 chosen sigmoid(z), without the correction, over their sum, times `weight_scale`.
 
+A fourth: `score` "softmax" chooses by softmax(z) over all experts + the correction, where `groups` is given only within the
+`keep` groups that rank best by their LARGEST; the weights are the chosen softmax(z) as they are.
+With `identity` the last that many of the experts + identity router rows are experts without tensors whose result is h itself
+(times the weight; kinds of score that are not normalised). Groups are formed over all of them together.
+
 With `shared_size` a shared expert of the same form and that size runs for every token and is added; with `shared_gate` its
 result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits).
 Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: a few rows one
@@ -22,7 +27,7 @@ portions sorts its (row, choice) pairs by expert and gives each expert's block o
 tensor-core kernels in bfloat16), for which the host reads the experts' row counts once a layer.
 
 params: hidden_size, experts, top, expert_size, score (default "sigmoid"), weight_at (default "input"), router_bias
-(default False), groups (count, keep) (default none), weight_scale (default 1), shared_size (default none), shared_gate (default
+(default False), groups (count, keep) (default none), identity (default 0), weight_scale (default 1), shared_size (default none), shared_gate (default
 False), router_name (default "mlp.router"), router_bias_name (default "mlp.router.b"), correction_name (default
 "mlp.correction"), expert_prefix (default "mlp.e": expert i's tensors are <expert_prefix><i>.gate / .up / .down),
 shared_prefix (default "mlp.shared": .gate / .up / .down, and .sg for its gate).
@@ -46,8 +51,10 @@ class RoutedFF(Part):
         super().__init__(params, ctx, prefix)
         self.hidden, self.experts, self.top = int(params["hidden_size"]), int(params["experts"]), int(params["top"])
         self.inter = int(params["expert_size"])
-        if not 1 <= self.top <= self.experts:
-            raise ValueError(f"routed feed-forward: top {self.top} of {self.experts} experts")
+        self.identity = int(params.get("identity") or 0)
+        self.choices = self.experts + self.identity          # what the router chooses from
+        if not 1 <= self.top <= self.choices:
+            raise ValueError(f"routed feed-forward: top {self.top} of {self.choices} experts")
         self.score, self.weight_at = params.get("score", "sigmoid"), params.get("weight_at", "input")
         if self.score not in ops.MOE_SCORES or self.weight_at not in ("input", "output"):
             raise ValueError(f"routed feed-forward: score {self.score!r} (known: {sorted(ops.MOE_SCORES)}), weight_at "
@@ -58,14 +65,17 @@ class RoutedFF(Part):
         self.router_bias = None
         self.expert_prefix = prefix + params.get("expert_prefix", "mlp.e")
         self.router = self.wgu = self.wdown = self.correction = None
-        self.correction_name = (prefix + params.get("correction_name", "mlp.correction")) if self.score == "sigmoid_normed" else None
+        corrected = self.score in ("sigmoid_normed", "softmax")
+        self.correction_name = (prefix + params.get("correction_name", "mlp.correction")) if corrected else None
         self.groups, self.keep = (int(g) for g in (params.get("groups") or (1, 1)))
         self.weight_scale = float(params.get("weight_scale", 1.0))
-        if self.experts % self.groups or not 1 <= self.keep <= self.groups or self.keep * (self.experts // self.groups) < self.top:
-            raise ValueError(f"routed feed-forward: {self.experts} experts in {self.groups} groups of which {self.keep} stay, "
+        if self.choices % self.groups or not 1 <= self.keep <= self.groups or self.keep * (self.choices // self.groups) < self.top:
+            raise ValueError(f"routed feed-forward: {self.choices} experts in {self.groups} groups of which {self.keep} stay, "
                              f"{self.top} chosen")
-        if self.groups > 1 and self.score != "sigmoid_normed":
-            raise ValueError(f"routed feed-forward: groups go with score 'sigmoid_normed', not {self.score!r}")
+        if self.groups > 1 and not corrected:
+            raise ValueError(f"routed feed-forward: groups go with scores 'sigmoid_normed' and 'softmax', not {self.score!r}")
+        if self.identity and (self.score not in ("sigmoid", "softmax") or not self.at_output):
+            raise ValueError("routed feed-forward: identity experts go with weights that are not normalised, on the experts' results")
         self.shared = int(params.get("shared_size") or 0)
         self.shared_gated = bool(params.get("shared_gate", False)) and self.shared > 0
         self.shared_prefix = prefix + params.get("shared_prefix", "mlp.shared")
@@ -75,11 +85,11 @@ class RoutedFF(Part):
         return f"{self.expert_prefix}{i}.{key}"
 
     def param_specs(self):
-        specs = [ParamSpec(self.router_name, (self.experts, self.hidden))]
+        specs = [ParamSpec(self.router_name, (self.choices, self.hidden))]
         if self.router_bias_name:
-            specs.append(ParamSpec(self.router_bias_name, (self.experts,), init="zeros"))
+            specs.append(ParamSpec(self.router_bias_name, (self.choices,), init="zeros"))
         if self.correction_name:
-            specs.append(ParamSpec(self.correction_name, (self.experts,), init="zeros"))
+            specs.append(ParamSpec(self.correction_name, (self.choices,), init="zeros"))
         if self.shared:
             s = self.shared_prefix
             specs += [ParamSpec(s + ".gate", (self.shared, self.hidden)), ParamSpec(s + ".up", (self.shared, self.hidden)),
@@ -146,25 +156,28 @@ class RoutedFF(Part):
     def forward(self, xn, x, batch):
         T, top, F = xn.shape[0], self.top, self.inter
         shared_weight = torch.empty(T, dtype=torch.float32, device=xn.device) if self.shared_gated else None
+        idw = torch.empty(T, dtype=torch.float32, device=xn.device) if self.identity else None
         expert, score = ops.moe_route(xn, self.router, top, self.router_bias, self.score, self.correction, self.groups, self.keep,
-                                      self.weight_scale, self.shared_gate, shared_weight)
+                                      self.weight_scale, self.shared_gate, shared_weight, self.identity, idw)
         if self.shared:
             self._add_shared(xn, x, shared_weight)
         if T * top < GROUPED_MIN_PAIRS:
-            ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output)
+            ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output, idw)
             return None
-        offsets, pos, src = ops.moe_sort(expert, self.experts)
+        offsets, pos, src = ops.moe_sort(expert, self.choices)
+        # identity experts come last in the order: their sorted rows hold nothing
+        limit, rows_in = (offsets[self.experts:], xn) if self.identity else (None, None)
         if getattr(batch, "max_q_len", 1) <= 1 or T * top < SORTED_MIN_PAIRS:
             gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
             ops.moe_grouped(xn, src, top, self.wgu, offsets, gu)
             act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
-            ops.moe_act(gu, src, score, act, self.at_output)
+            ops.moe_act(gu, src, score, act, self.at_output, limit)
             planes.record(batch, "activation", act)
             ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
             ops.moe_grouped(act, None, 1, self.wdown, offsets, ys)
-            ops.moe_combine(ys, pos, x, top)
+            ops.moe_combine(ys, pos, x, top, limit, rows_in, idw)
             return None
-        xs = ops.moe_gather(xn, src, top)
+        xs = ops.moe_gather(xn, src, top, limit)
         bounds = offsets.tolist()                      # the one read by the host: how many rows each expert has
         gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
         for e in range(self.experts):
@@ -172,14 +185,14 @@ class RoutedFF(Part):
             if hi > lo:
                 ops.linear(xs[lo:hi], self.w_gu_e[e], gu[lo:hi])
         act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
-        ops.moe_act(gu, src, score, act, self.at_output)
+        ops.moe_act(gu, src, score, act, self.at_output, limit)
         planes.record(batch, "activation", act)
         ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
                 ops.linear(act[lo:hi], self.w_down_e[e], ys[lo:hi])
-        ops.moe_combine(ys, pos, x, top)
+        ops.moe_combine(ys, pos, x, top, limit, rows_in, idw)
         return None
 
 

@@ -11,7 +11,9 @@ and knows nothing else about the architecture.
   with other slots and needs no change here). Chosen layer by layer: layers of one model may differ.
 - `order` is the list of steps in which layers run. A step may name a layer that an earlier
   step named (its weights are used again, with a cache of its own), or say that its mixer
-  reads the cache of an earlier step instead of keeping one.
+  reads the cache of an earlier step instead of keeping one. A step that starts another pass of
+  layers that run several times may say so (`enters_pass`): what the model adds to the residual
+  stream there is its `pass_entry` part.
 
 The reference has one hard-wired graph (src/api.cu:1728-1765, 1891-1952).
 """
@@ -46,6 +48,7 @@ class LayerSpec:
 class RunStep:
     layer: int
     reads_cache_of: Optional[int] = None  # index into `order` of the earlier step whose cache is read
+    enters_pass: Optional[int] = None     # the step is the first of this pass: the model's pass_entry part runs ahead of it
 
 
 @dataclass(frozen=True)
@@ -60,6 +63,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     eos_token_ids: Tuple[int, ...] = ()
+    pass_entry: Optional[PartSpec] = None   # what steps that enter a pass add to the residual stream
 
     def validate(self) -> None:
         if not self.order:
@@ -67,6 +71,8 @@ class ModelSpec:
         for i, st in enumerate(self.order):
             if not (0 <= st.layer < len(self.layers)):
                 raise ValueError(f"order[{i}] names layer {st.layer}; there are {len(self.layers)} layers")
+            if st.enters_pass is not None and self.pass_entry is None:
+                raise ValueError(f"order[{i}] enters a pass; the model has no pass_entry part")
             if st.reads_cache_of is not None:
                 j = st.reads_cache_of
                 if not (0 <= j < i):
