@@ -572,8 +572,33 @@ def gakupel_configs(size: dict, window: int):
     return gakupel, mavinex_configs(size, window)[0]
 
 
-DESIGNS = {"gakupel": gakupel_configs, "torirax": design_configs, "vegodra": vegodra_configs, "runopel": runopel_configs, "mavinex": mavinex_configs}
-BESIDE = {"gakupel": "mavinex", "torirax": "llama", "vegodra": "llama", "runopel": "vegodra", "mavinex": "runopel"}
+def selovik_configs(size: dict, window: int):
+    """(Selovik config, Gakupel config, Torirax config) of equal width, layer runs, head counts and feed-forward width: Gakupel
+    is the closest of the other designs in its feed-forwards (a dense one without a gate, grouped routing with a shared
+    expert), Torirax in its attention (two score maps a head). Selovik's attention has maps of head_dim / 2 with values of
+    head_dim, as Torirax's, rotated whole (YaRN), in a window of `window` positions. Feed-forwards alternate between the dense one
+    and eight experts of half its width beside four identity experts in four groups, two per token, with a shared expert of
+    a quarter. The layers in the middle (three eighths of the layer runs) are gone through twice."""
+    W, L, H, G, D = size["width"], size["layers"], size["heads"], size["kv"], size["head_dim"]
+    start, span = L // 8, 3 * L // 8
+    m = dict(heads=H, kv_heads=G, dim=D // 2, vdim=D, scale=(D // 2) ** -0.5, diff=0.5, mask=dict(size=window),
+             rot=dict(base=500000.0, dims=D // 2, scaling=dict(factor=4.0, original=CONTEXT_LEN // 4, fast=32.0, slow=1.0)))
+    layers = []
+    for i in range(L - span):
+        if i % 2 == 0:
+            mlp = dict(kind="dense", ff=size["ff"])
+        else:
+            mlp = dict(kind="moe", expert=dict(ff=size["ff"] // 2), router=dict(experts=8, identity=4, top=2, groups=dict(count=4, keep=2)),
+                       shared=dict(ff=size["ff"] // 4))
+        layers.append(dict(type="attention", mixer=m, mlp=mlp))
+    selovik = dict(architecture="Selovik", vocab=size["vocab"], width=W, max_positions=CONTEXT_LEN, norm=dict(eps=1e-5),
+                   embedding=dict(scale=1.0, bigram=dict(buckets=65521, mul_prev=31, mul_cur=17)), logit_scale=0.5,
+                   loop=dict(start=start, stop=start + span, times=2), layers=layers)
+    return selovik, gakupel_configs(size, window)[0], design_configs(size, window)[0]
+
+
+DESIGNS = {"selovik": selovik_configs, "gakupel": gakupel_configs, "torirax": design_configs, "vegodra": vegodra_configs, "runopel": runopel_configs, "mavinex": mavinex_configs}
+BESIDE = {"selovik": "gakupel,torirax", "gakupel": "mavinex", "torirax": "llama", "vegodra": "llama", "runopel": "vegodra", "mavinex": "runopel"}
 
 
 def kernel_table(one, reps: int = 3):
@@ -618,7 +643,7 @@ def kernel_table(one, reps: int = 3):
 
 def design_bench(a) -> int:
     """Prefill and decode throughput of the chosen design and of the model beside it (the Llama decoder for Torirax and
-    Vegodra, Vegodra for Runopel, Runopel for Mavinex, Mavinex for Gakupel) at equal layer sizes, with each step's kernels by name; one JSON line. The default run
+    Vegodra, Vegodra for Runopel, Runopel for Mavinex, Mavinex for Gakupel, Gakupel and Torirax for Selovik) at equal layer sizes, with each step's kernels by name; one JSON line. The default run
     of this file is untouched by this option."""
     import torch
 
@@ -639,7 +664,7 @@ def design_bench(a) -> int:
             size["layers"] = a.layers
         MODEL["vocab_size"] = size["vocab"]
         res = {}
-        for which, cfg in zip((a.design, BESIDE[a.design]), DESIGNS[a.design](size, a.window)):
+        for which, cfg in zip([a.design] + BESIDE[a.design].split(","), DESIGNS[a.design](size, a.window)):
             pages_per_seq = -(-(PROMPT_LEN + a.steps + a.warmup + 16 + 4 * PAGE) // PAGE)
             eng = Engine(config=cfg, random_weights=0, std=0.02, dtype="bfloat16", max_batch=max(batches), max_seq=CONTEXT_LEN,
                          max_prefill=max(PREFILL_TOKENS, PROMPT_LEN), page_size=PAGE,
@@ -769,7 +794,7 @@ def main() -> int:
                     help="prefill and decode of this design beside its closest other model at equal layer sizes (see --sizes); "
                          "the default run is not changed by it")
     ap.add_argument("--sizes", default="1b", help="with --design: layer sizes, of " + ", ".join(sorted(DESIGN_SIZES)) + " (commas between)")
-    ap.add_argument("--window", type=int, default=1024, help="with --design: the attention window (torirax: the first 4 tokens are kept; runopel; mavinex) or chunk size (vegodra)")
+    ap.add_argument("--window", type=int, default=1024, help="with --design: the attention window (torirax: the first 4 tokens are kept; runopel; mavinex; selovik) or chunk size (vegodra)")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)

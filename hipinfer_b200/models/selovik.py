@@ -33,7 +33,7 @@ def _ff_spec(c: SelovikConfig, ff) -> PartSpec:
 
 def selovik_spec(c: SelovikConfig) -> ModelSpec:
     W = c.width
-    norm = lambda name: PartSpec("rmsnorm", dict(name=name, size=W, eps=c.norm_eps, one_plus=True))
+    norm = lambda name, **kw: PartSpec("rmsnorm", dict(name=name, size=W, eps=c.norm_eps, one_plus=True, **kw))
     layers = []
     for i, L in enumerate(c.layers):
         parts = dict(mixer_norm=norm("norm1"), mixer=_mixer_spec(c, L.mixer))
@@ -44,8 +44,9 @@ def selovik_spec(c: SelovikConfig) -> ModelSpec:
         architecture=c.architecture, hidden_size=W, vocab_size=c.vocab, max_position=c.max_positions,
         embedding=PartSpec("token_bigram", dict(name="embed", vocab_size=c.vocab, hidden_size=W, scale=c.embedding_scale,
                                                 bigram=c.bigram, norm=norm("embed.norm"))),
-        layers=tuple(layers), order=tuple(RunStep(i, enters_pass=t) for i, t in c.run_order()), final_norm=norm("final.norm"),
-        head=PartSpec("linear", dict(tied_to="embed", vocab_size=c.vocab, hidden_size=W, scale=c.logit_scale)),
+        layers=tuple(layers), order=tuple(RunStep(i, enters_pass=t) for i, t in c.run_order()),
+        # the head is linear: the logits' scale multiplies its input, in the norm's 32-bit weight
+        final_norm=norm("final.norm", gain=c.logit_scale), head=PartSpec("linear", dict(tied_to="embed", vocab_size=c.vocab, hidden_size=W)),
         pass_entry=None if c.loop is None else PartSpec("loop", dict(name="loop.step", passes=c.loop.times, hidden_size=W)),
         eos_token_ids=c.eos_token_ids)
 

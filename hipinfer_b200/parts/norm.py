@@ -13,21 +13,21 @@ from .registry import Part, register_part, to_compute
 class RMSNorm(Part):
     """params: name (tensor name relative to the prefix), size, eps, one_plus (default False: the weight multiplies as it is
     stored; True: the tensor is stored around zero and the row is multiplied by 1 + w, a sum made in 32-bit at load and kept
-    in 32-bit)."""
+    in 32-bit), gain (default 1: a constant that multiplies the result; it is folded into the weight, in 32-bit)."""
 
     def __init__(self, params, ctx, prefix=""):
         super().__init__(params, ctx, prefix)
         self.size, self.eps = int(params["size"]), float(params["eps"])
         self.name = prefix + params["name"]
-        self.one_plus = bool(params.get("one_plus", False))
+        self.one_plus, self.gain = bool(params.get("one_plus", False)), float(params.get("gain", 1.0))
         self.weight = None
 
     def param_specs(self):
         return [ParamSpec(self.name, (self.size,), init="zeros" if self.one_plus else "ones")]
 
     def load(self, tensors):
-        if self.one_plus:
-            self.weight = (tensors[self.name].to(torch.float32) + 1.0).contiguous()
+        if self.one_plus or self.gain != 1.0:
+            self.weight = ((tensors[self.name].to(torch.float32) + (1.0 if self.one_plus else 0.0)) * self.gain).contiguous()
             return
         self.weight = to_compute(tensors[self.name], self.ctx)
 

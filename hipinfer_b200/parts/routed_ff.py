@@ -20,7 +20,8 @@ With `identity` the last that many of the experts + identity router rows are exp
 (times the weight; kinds of score that are not normalised). Groups are formed over all of them together.
 
 With `shared_size` a shared expert of the same form and that size runs for every token and is added; with `shared_gate` its
-result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits).
+result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits). One without a gate is a gated
+feed-forward like any other and runs on its kernels (parts/feed_forward.py).
 Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: a few rows one
 by one, more of them sorted by expert so that an expert's weights are read once for all of its rows. A step with prompt
 portions sorts its (row, choice) pairs by expert and gives each expert's block of rows to the ordinary products (the
@@ -39,6 +40,7 @@ import torch
 from ..kernels import ops
 from ..weights import ParamSpec
 from . import planes
+from .feed_forward import GatedFF
 from .registry import Part, register_part, to_compute
 
 SORTED_MIN_PAIRS = 64     # fewer (row, choice) pairs than this never go to the ordinary products
@@ -79,7 +81,11 @@ class RoutedFF(Part):
         self.shared = int(params.get("shared_size") or 0)
         self.shared_gated = bool(params.get("shared_gate", False)) and self.shared > 0
         self.shared_prefix = prefix + params.get("shared_prefix", "mlp.shared")
-        self.shared_gate = self.s_gu = self.s_down = self.ones = self.index = None
+        self.shared_gate = self.s_gu = self.s_down = self.index = self.shared_ff = None
+        if self.shared and not self.shared_gated:
+            self.shared_ff = GatedFF(dict(hidden_size=self.hidden, intermediate_size=self.shared, activation="silu",
+                                          **{k + "_name": f"{params.get('shared_prefix', 'mlp.shared')}.{k}" for k in ("gate", "up", "down")}),
+                                     ctx, prefix)
 
     def _expert(self, i, key):
         return f"{self.expert_prefix}{i}.{key}"
@@ -90,12 +96,13 @@ class RoutedFF(Part):
             specs.append(ParamSpec(self.router_bias_name, (self.choices,), init="zeros"))
         if self.correction_name:
             specs.append(ParamSpec(self.correction_name, (self.choices,), init="zeros"))
-        if self.shared:
+        if self.shared_ff is not None:
+            specs += self.shared_ff.param_specs()
+        elif self.shared:
             s = self.shared_prefix
             specs += [ParamSpec(s + ".gate", (self.shared, self.hidden)), ParamSpec(s + ".up", (self.shared, self.hidden)),
                       ParamSpec(s + ".down", (self.hidden, self.shared))]
-            if self.shared_gated:
-                specs.append(ParamSpec(s + ".sg", (1, self.hidden)))
+            specs.append(ParamSpec(s + ".sg", (1, self.hidden)))
         for i in range(self.experts):
             specs += [ParamSpec(self._expert(i, "gate"), (self.inter, self.hidden)),
                       ParamSpec(self._expert(i, "up"), (self.inter, self.hidden)),
@@ -109,13 +116,14 @@ class RoutedFF(Part):
             self.router_bias = t(self.router_bias_name).to(self.router.dtype).contiguous()
         if self.correction_name:
             self.correction = t(self.correction_name).to(self.router.dtype).contiguous()
-        if self.shared:
+        if self.shared_ff is not None:
+            self.shared_ff.load(tensors)
+        elif self.shared:
             g, u, d = (t(f"{self.shared_prefix}.{k}") for k in ("gate", "up", "down"))
             sdt = g.dtype if g.dtype == u.dtype == d.dtype else torch.float32
             self.s_gu = ops.Weight(torch.cat([g.to(sdt), u.to(sdt)], 0).contiguous())        # gate rows, then up rows
             self.s_down = ops.Weight(d.to(sdt).contiguous())
-            if self.shared_gated:
-                self.shared_gate = t(self.shared_prefix + ".sg").to(self.router.dtype).reshape(-1).contiguous()
+            self.shared_gate = t(self.shared_prefix + ".sg").to(self.router.dtype).reshape(-1).contiguous()
         mats = [t(self._expert(i, k)) for i in range(self.experts) for k in ("gate", "up", "down")]
         dt = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
         E, F, W = self.experts, self.inter, self.hidden
@@ -128,22 +136,20 @@ class RoutedFF(Part):
     def weight_bytes(self):
         """What a single row reads: the router and `top` experts."""
         per = (self.wgu.numel() + self.wdown.numel()) * self.wgu.element_size() // self.experts
-        shared = self.s_gu.nbytes + self.s_down.nbytes if self.shared else 0
+        shared = self.shared_ff.weight_bytes() if self.shared_ff else self.s_gu.nbytes + self.s_down.nbytes if self.shared else 0
         return self.router.numel() * self.router.element_size() + self.top * per + shared
 
     def _row_index(self, T, dev):
-        """(0 .. T-1, zeros, ones): a shared expert as the one expert of every row."""
+        """(0 .. T-1, zeros): a shared expert as the one expert of every row."""
         if self.index is None or self.index[0].numel() < T:
             n = max(T, 2048)
-            self.index = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, 1, dtype=torch.int32, device=dev),
-                          torch.ones(n, dtype=torch.float32, device=dev))
+            self.index = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, 1, dtype=torch.int32, device=dev))
         return tuple(t[:T] for t in self.index)
 
     def _add_shared(self, xn, x, weight):
         """x += weight * shared expert: the weight enters at the activation in 32-bit (the down product is linear)."""
         T, F = xn.shape[0], self.shared
-        rows, zeros, ones = self._row_index(T, xn.device)
-        weight = ones if weight is None else weight
+        rows, zeros = self._row_index(T, xn.device)
         if T < SHARED_MIN_ROWS:
             ops.moe_rows(xn, self.s_gu.t.unsqueeze(0), self.s_down.t.unsqueeze(0), zeros, weight, x, True)
             return
@@ -159,7 +165,9 @@ class RoutedFF(Part):
         idw = torch.empty(T, dtype=torch.float32, device=xn.device) if self.identity else None
         expert, score = ops.moe_route(xn, self.router, top, self.router_bias, self.score, self.correction, self.groups, self.keep,
                                       self.weight_scale, self.shared_gate, shared_weight, self.identity, idw)
-        if self.shared:
+        if self.shared_ff is not None:
+            self.shared_ff.forward(xn, x, None)
+        elif self.shared:
             self._add_shared(xn, x, shared_weight)
         if T * top < GROUPED_MIN_PAIRS:
             ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output, idw)

@@ -142,6 +142,23 @@ def route(h, router, correction, r):
     return chosen, torch.gather(s, 1, chosen)
 
 
+def closest_call(h, router, correction, r):
+    """Per token, how far the closest of the router's calls is from going the other way (the last group kept against the first
+    one dropped, the last expert chosen against the next)."""
+    c = torch.softmax(h @ router.T, -1) + correction
+    T, E = c.shape
+    g, margin = r.get("groups"), torch.full((T,), float("inf"), dtype=F)
+    if g and g["keep"] < g["count"]:
+        best = torch.sort(c.reshape(T, g["count"], -1).amax(-1), dim=-1, descending=True)
+        margin = best.values[:, g["keep"] - 1] - best.values[:, g["keep"]]
+        stay = torch.zeros(T, g["count"], dtype=torch.bool).scatter_(1, best.indices[:, :g["keep"]], True)
+        c = c.masked_fill(~stay.repeat_interleave(E // g["count"], 1), float("-inf"))
+    c = torch.sort(c, dim=-1, descending=True).values
+    if r["top"] < E:
+        margin = torch.minimum(margin, c[:, r["top"] - 1] - c[:, r["top"]])
+    return margin
+
+
 def experts(h, w, r):
     """w: router, correction, e<i>.gate / up / down, shared.gate / up / down; r also: experts, identity."""
     chosen, weight = route(h, w["router"], w["correction"], r)
@@ -174,10 +191,11 @@ def sub(tensors, prefix):
     return {k[len(prefix):]: v.to(F) for k, v in tensors.items() if k.startswith(prefix)}
 
 
-def forward(cfg, tensors, tokens, layers_out=None, round_to=None):
+def forward(cfg, tensors, tokens, layers_out=None, round_to=None, calls=None):
     """Logits [T, vocab] of one sequence from position 0. cfg: the config.json dictionary; tensors: name -> tensor.
     layers_out (a list): the residual rows after every layer run are appended. round_to (a function): every sublayer's input
-    and result go through it; the difference to the exact logits measures how sensitive each position is to rounding."""
+    and result go through it; the difference to the exact logits measures how sensitive each position is to rounding. calls (a
+    list): every router's closest call per position is appended."""
     rd = round_to or (lambda t: t)
     eps = cfg["norm"]["eps"]
     x = x0 = embedding(tokens, tensors, cfg)
@@ -190,7 +208,10 @@ def forward(cfg, tensors, tokens, layers_out=None, round_to=None):
         L, w = cfg["layers"][i], layers[i]
         y = rd(attention(rd(norm(x, w["norm1"], eps)), sub(w, "mix."), L["mixer"], eps))
         if L.get("mlp") is not None:
-            y = y + rd(feed_forward(rd(norm(x, w["norm2"], eps)), sub(w, "mlp."), L["mlp"]))
+            h = rd(norm(x, w["norm2"], eps))
+            if calls is not None and L["mlp"]["kind"] == "moe":
+                calls.append(closest_call(h, w["mlp.router"], w["mlp.correction"], L["mlp"]["router"]))
+            y = y + rd(feed_forward(h, sub(w, "mlp."), L["mlp"]))
         x = x + y
         if layers_out is not None:
             layers_out.append(x.clone())
