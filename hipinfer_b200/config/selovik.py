@@ -54,7 +54,7 @@ class RotaryDiffAttentionConfig:
         if rot.dims < 0 or rot.dims % 2 or rot.dims > dim:
             raise ConfigError(f"config.json: {where}rot.dims = {rot.dims} must be even and at most dim = {dim}")
         mask = _optional(m, "mask", where)
-        c = cls(pos("heads"), pos("kv_heads"), dim, pos("vdim"), take(m, "scale", float), take(m, "diff", float), rot,
+        c = cls(pos("heads"), pos("kv_heads"), dim, pos("vdim"), take(m, "scale", float, positive=True), take(m, "diff", float), rot,
                 take(mask, "size", int, None, positive=True) if mask else None)
         if c.heads % c.kv_heads:
             raise ConfigError(f"config.json: {where}{c.heads} heads are not a multiple of {c.kv_heads} kv_heads")

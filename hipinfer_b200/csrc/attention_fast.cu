@@ -98,7 +98,19 @@ __device__ __forceinline__ void ad_load_rows(const __nv_bfloat16* __restrict__ k
 // layer's 11 us at 8 requests) become two cluster barriers. Blocks without keys only pass the barriers.
 // EX: a distance bias, r1 ln(1 + r2 (p - j)) off the score of key j, and a sink, exp(sink) in the denominator (a number
 // per head each; the sink joins in the block of the row's first chunk).
-template <int D, int G, bool TMA, int RW, int KW, int SR, bool CL, bool EX>
+// DIFF (TMA only): differential attention. A head has two score maps of D / 2 dimensions that lie side by side in its query
+// and key rows; the G rows of the tile are (head, map) pairs, a row holding its map's half of the query and zeros in the other
+// half, so that one product over the whole key row gives both maps' scores. The block that finishes a (row, kv head) combines
+// the maps, o = a_0 - lambda a_1, divides by the root mean square over the D values, multiplies by post and by sigmoid(gate). A
+// window is allowed: chunks are counted from the row's first one, pages are read whole from the one that holds the window's
+// first key, and the keys before it are masked.
+struct AdDiff {
+  const float* gate;         // [T][ld_gate] at column gate_off, or null
+  long ld_gate;
+  int gate_off;
+  float lambda, post, eps;
+};
+template <int D, int G, bool TMA, int RW, int KW, int SR, bool CL, bool EX, bool DIFF>
 __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, int* __restrict__ status,
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
@@ -106,7 +118,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     __nv_bfloat16* __restrict__ out, float* __restrict__ part_acc, float* __restrict__ part_ml, int Hq, int Hkv,
     int page_size, int window, float scale_log2, int chunk, int S, const int* __restrict__ q_len, int row_limit,
     const int* __restrict__ ctx_len, int* __restrict__ counters, const float* __restrict__ r1p,
-    const float* __restrict__ r2p, const float* __restrict__ sink) {
+    const float* __restrict__ r2p, const float* __restrict__ sink, AdDiff df) {
+  static_assert(!DIFF || (TMA && !EX && G % 2 == 0), "two score maps: by TMA, no extras");
   constexpr int CH = D / 8, KS = D / 16, NT_O = D / 8, WK = 64;  // WK: keys per warp pass
   extern __shared__ __align__(128) uint8_t smem_dyn[];
   uint8_t* smem_raw = TMA ? (uint8_t*)(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023) : smem_dyn;   // the swizzle wants 1 KB
@@ -123,21 +136,23 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
   __shared__ int abort_flag;
   __shared__ __align__(16) float cl_acc[CL ? G * D : 1];     // CL: this block's partial result, read by the merging block
   __shared__ __align__(8) float cl_ml[CL ? G * 2 : 2];
+  __shared__ float fin[DIFF ? G * D : 1];                    // DIFF: the maps' results, before they are combined
   hb_pdl_launch();
   HB_TL_MARK(0, 0);
-  const int t = blockIdx.z, h = blockIdx.y, s = blockIdx.x;
+  const int t = blockIdx.z, h = blockIdx.y;
   // row_req null: a step of single decode rows, row t being request t (and its position the length its request had):
   // one round trip to memory less before the keys can be asked for
   const int rq = row_req ? row_req[t] : t;
   const int p = pos[t];
   const int lo = window > 0 ? max(0, p - window + 1) : 0;
   const int s_lo = lo / chunk, s_hi = p / chunk;
+  const int s_off = DIFF && window > 0 ? s_lo : 0, s = (int)blockIdx.x + s_off;      // the chunk of the grid's first block
   if ((q_len && q_len[rq] >= row_limit) || s < s_lo || s > s_hi) {  // a long portion (the flash kernel's), or no keys here
     if ((blockIdx.x | blockIdx.y | blockIdx.z) == 0) hb_pdl_wait();  // the grid never ends before the one ahead of it
     if constexpr (CL) { hb_cluster_sync(); hb_cluster_sync(); }      // the cluster's two barriers, as every block of it
     return;
   }
-  const int k0 = max(s * chunk, lo), k1 = min((s + 1) * chunk, p + 1), nk = k1 - k0;
+  const int k0 = max(s * chunk, DIFF ? lo / page_size * page_size : lo), k1 = min((s + 1) * chunk, p + 1), nk = k1 - k0;
   const int n_old = ctx_len ? max(0, min(k1, row_req ? ctx_len[rq] : p) - k0) : 0;   // rows of the tile from earlier steps
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
   const int* table = bt + (size_t)rq * bt_stride;
@@ -203,10 +218,45 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
   for (int i = tid; i < 16 * CH; i += AD_THREADS) {
     const int r = i / CH, c = i - r * CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < G) v = *(const uint4*)(q + ((size_t)t * Hq + (size_t)h * G + r) * D + c * 8);
+    if constexpr (DIFF) {
+      if (r < G && c / (CH / 2) == (r & 1)) v = *(const uint4*)(q + ((size_t)t * (Hq / 2) + (size_t)h * (G / 2) + r / 2) * D + c * 8);
+    } else {
+      if (r < G) v = *(const uint4*)(q + ((size_t)t * Hq + (size_t)h * G + r) * D + c * 8);
+    }
     asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};" ::"r"(sQ + ad_swz<D>(r, c)), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
   }
   if constexpr (!TMA) hb_cp_async_wait<0>();
+  // DIFF: the gates of head `warp` (the heads of a kv head are at most four), asked for long before they are needed
+  float gate_v[DIFF ? D / 32 : 1];
+  if constexpr (DIFF) {
+#pragma unroll
+    for (int i = 0; i < D / 32; i++)
+      gate_v[i] = df.gate && warp < G / 2 ? df.gate[(size_t)t * df.ld_gate + df.gate_off + (h * (G / 2) + warp) * D + i * 32 + lane] : 0.f;
+  }
+  // the row's result, a value at a time (DIFF: of one map, to be combined)
+  auto put = [&](size_t head, int gg, int d, float v) {
+    if constexpr (DIFF) fin[gg * D + d] = v;
+    else out[head * D + d] = __float2bfloat16_rn(v);
+  };
+  auto combine = [&]() {
+    if constexpr (DIFF) {
+      static_assert(G / 2 <= AD_WARPS, "a warp a head");
+      __syncthreads();
+      if (warp < G / 2) {
+        float o[D / 32], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < D / 32; i++) {
+          o[i] = fin[2 * warp * D + i * 32 + lane] - df.lambda * fin[(2 * warp + 1) * D + i * 32 + lane];
+          ss = fmaf(o[i], o[i], ss);
+        }
+        const float f = rsqrtf(hb_warp_sum(ss) / (float)D + df.eps) * df.post;
+        __nv_bfloat16* dst = out + ((size_t)t * (Hq / 2) + (size_t)h * (G / 2) + warp) * D;
+#pragma unroll
+        for (int i = 0; i < D / 32; i++)
+          dst[i * 32 + lane] = __float2bfloat16_rn(df.gate ? o[i] * f / (1.f + expf(-gate_v[i])) : o[i] * f);
+      }
+    }
+  };
   __syncthreads();
   if constexpr (TMA) {
     if (warp * KW < nk) loaded = hb_mbar_wait(&bars[warp], 0, &abort_flag);
@@ -285,7 +335,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     for (int i = 0; i < RW / 8; i++)
 #pragma unroll
       for (int e = 0; e < 2; e++) {
-        if (kb + i * 8 + 2 * tq + e >= nk) sc[i][e] = -INFINITY;
+        if (kb + i * 8 + 2 * tq + e >= nk || (DIFF && k0 + kb + i * 8 + 2 * tq + e < lo)) sc[i][e] = -INFINITY;
         mx = fmaxf(mx, sc[i][e]);
       }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -352,18 +402,20 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     }
     const size_t head = (size_t)t * Hq + (size_t)h * G + gg;
     if (whole) {
-      out[head * D + d] = __float2bfloat16_rn(a / l);
+      put(head, gg, d, a / l);
     } else if constexpr (CL) {
       cl_acc[i] = a;
       if (d == 0) { cl_ml[gg * 2] = m * 0.6931471805599453f; cl_ml[gg * 2 + 1] = l; }
     } else {
-      part_acc[(head * S + s) * D + d] = a;
+      const int sb = s - s_off;
+      part_acc[(head * S + sb) * D + d] = a;
       if (d == 0) {
-        part_ml[(head * S + s) * 2] = m * 0.6931471805599453f;
-        part_ml[(head * S + s) * 2 + 1] = l;
+        part_ml[(head * S + sb) * 2] = m * 0.6931471805599453f;
+        part_ml[(head * S + sb) * 2 + 1] = l;
       }
     }
   }
+  if (DIFF && whole) combine();
   HB_TL_MARK(1, 3);   // slot 1: the end of the chunk work; slot 0: the end of the merge
   if constexpr (CL) {
     hb_cluster_sync();                                     // every block's partial is in its shared memory, visible cluster-wide
@@ -377,8 +429,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
         for (int c = 0; c < 8; c++)
           if (c < nc) {
             uint32_t ra, rm;
-            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(acc_l + (uint32_t)i * 4), "r"((uint32_t)(s_lo + c)));
-            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(rm) : "r"(ml_l + (uint32_t)gg * 8), "r"((uint32_t)(s_lo + c)));
+            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(acc_l + (uint32_t)i * 4), "r"((uint32_t)(s_lo - s_off + c)));
+            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(rm) : "r"(ml_l + (uint32_t)gg * 8), "r"((uint32_t)(s_lo - s_off + c)));
             asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(av[c]) : "r"(ra) : "memory");
             asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(mv[c]), "=f"(lv[c]) : "r"(rm) : "memory");
           }
@@ -393,8 +445,9 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
             l += lv[c] * f;
             a += av[c] * f;
           }
-        out[((size_t)t * Hq + (size_t)h * G + gg) * D + (i - gg * D)] = __float2bfloat16_rn(a / l);
+        put((size_t)t * Hq + (size_t)h * G + gg, gg, i - gg * D, a / l);
       }
+      combine();
     }
     hb_cluster_sync();                                     // no block leaves while its partial may still be read
     HB_TL_MARK(0, 3);
@@ -424,8 +477,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
       const int i = i0 + k * AD_THREADS, gg = i / D, d = i - gg * D;
       if (i < G * D) {
         const size_t head = (size_t)t * Hq + (size_t)h * G + gg;
-        const float2* ml = (const float2*)part_ml + head * S + s_lo;
-        const float* pa = part_acc + (head * S + s_lo) * D + d;
+        const float2* ml = (const float2*)part_ml + head * S + s_lo - s_off;
+        const float* pa = part_acc + (head * S + s_lo - s_off) * D + d;
 #pragma unroll
         for (int c = 0; c < 16; c++)
           if (c < nc) { v[k][c] = __ldcg(ml + c); acc[k][c] = __ldcg(pa + (size_t)c * D); }
@@ -446,7 +499,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
             l += v[k][c].y * f;
             a += acc[k][c] * f;
           }
-        out[((size_t)t * Hq + (size_t)h * G + gg) * D + d] = __float2bfloat16_rn(a / l);
+        put((size_t)t * Hq + (size_t)h * G + gg, gg, d, a / l);
       }
     }
    }
@@ -454,8 +507,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
     for (int i = tid; i < G * D; i += AD_THREADS) {
       const int gg = i / D, d = i - gg * D;
       const size_t head = (size_t)t * Hq + (size_t)h * G + gg;
-      const float2* ml = (const float2*)part_ml + head * S + s_lo;
-      const float* pa = part_acc + (head * S + s_lo) * D + d;
+      const float2* ml = (const float2*)part_ml + head * S + s_lo - s_off;
+      const float* pa = part_acc + (head * S + s_lo - s_off) * D + d;
       float m = -INFINITY, a = 0.f, l = 0.f;
       for (int c = 0; c < nc; c++) m = fmaxf(m, __ldcg(ml + c).x);
       for (int c = 0; c < nc; c++) {
@@ -464,37 +517,42 @@ __global__ void __launch_bounds__(AD_THREADS) attn_decode_kernel(
         l += v.y * f;
         a += __ldcg(pa + (size_t)c * D) * f;
       }
-      out[head * D + d] = __float2bfloat16_rn(a / l);
+      put(head, gg, d, a / l);
     }
   }
+  combine();
   HB_TL_MARK(0, 3);
 }
 
-template <int D, bool TMA, int RW, int KW, int SR, bool CL, bool EX>
+template <int D, bool TMA, int RW, int KW, int SR, bool CL, bool EX, bool DIFF = false>
 static int launch_decode(int G, dim3 grid, size_t smem, cudaStream_t st, const CUtensorMap& mk, const CUtensorMap& mv,
                          int* status, const __nv_bfloat16* q, const __nv_bfloat16* kc, const __nv_bfloat16* vc,
                          const int* bt, int bt_stride, const int* row_req, const int* pos, __nv_bfloat16* out, float* pa,
                          float* pm, int Hq, int Hkv, int page_size, int window, float scale, int chunk, int S,
                          const int* q_len, int row_limit, const int* ctx_len, int* counters, const float* r1, const float* r2,
-                         const float* sink) {
+                         const float* sink, const AdDiff& df = AdDiff{}) {
 #define HB_AD_CASE(GG)                                                                                              \
   case GG:                                                                                                          \
     {                                                                                                               \
       static bool configured = false;                                                                               \
       if (!configured) {                                                                                            \
-        cudaFuncSetAttribute(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+        cudaFuncSetAttribute(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX, DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
         configured = true;                                                                                          \
       }                                                                                                             \
     }                                                                                                               \
     if (CL)                                                                                                         \
-      hb_launch_cluster(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, grid, AD_THREADS, smem, st, dim3(grid.x, 1, 1), mk, mv, status, \
+      hb_launch_cluster(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX, DIFF>, grid, AD_THREADS, smem, st, dim3(grid.x, 1, 1), mk, mv, status, \
                         q, kc, vc, bt, bt_stride, row_req, pos, out, pa, pm, Hq, Hkv, page_size, window, scale, chunk, S,    \
-                        q_len, row_limit, ctx_len, counters, r1, r2, sink);                                         \
+                        q_len, row_limit, ctx_len, counters, r1, r2, sink, df);                                         \
     else                                                                                                            \
-      hb_launch(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX>, grid, AD_THREADS, smem, st, mk, mv, status, q, kc, vc, bt, bt_stride, \
+      hb_launch(attn_decode_kernel<D, GG, TMA, RW, KW, SR, CL, EX, DIFF>, grid, AD_THREADS, smem, st, mk, mv, status, q, kc, vc, bt, bt_stride, \
                 row_req, pos, out, pa, pm, Hq, Hkv, page_size, window, scale, chunk, S, q_len, row_limit, ctx_len,  \
-                counters, r1, r2, sink);                                                                            \
+                counters, r1, r2, sink, df);                                                                            \
     return 0;
+  if constexpr (DIFF) {
+    switch (G) { HB_AD_CASE(2) HB_AD_CASE(4) HB_AD_CASE(6) HB_AD_CASE(8) }
+    return 1;
+  } else
   switch (G) {
     HB_AD_CASE(1) HB_AD_CASE(2) HB_AD_CASE(3) HB_AD_CASE(4) HB_AD_CASE(5) HB_AD_CASE(6) HB_AD_CASE(7) HB_AD_CASE(8)
   }
@@ -586,5 +644,58 @@ HB_EXPORT int hb_attn_decode(const void* q, const void* kc, const void* vc, long
 #undef HB_AD_ARGS
   if (r) HB_FAIL("hb_attn_decode: no kernel for group %d", G);
   HB_CHECK_LAUNCH("hb_attn_decode");
+  return 0;
+}
+
+// Differential attention of single rows (DIFF above): q [T, H, D] with D = both maps' dimensions together (64 or 128), planes [page, G,
+// page_size, D] for keys and values (values are as wide as the two maps), out [T, H, D]; at most four heads a kv head, pages of
+// 8 to 64 tokens (32 at D = 128). max_pos: the largest position among the rows. The workspace holds T * 2 H * S * (D + 2) floats,
+// S = hb_attn_diff_decode_splits(...); counters as for hb_attn_decode.
+HB_EXPORT int hb_attn_diff_decode_supported(int H, int G, int D, int page_size) {
+  return G > 0 && H % G == 0 && H / G <= 4 && (D == 64 || D == 128) && page_size >= 8 && page_size <= (D == 64 ? 64 : 32) && 64 % page_size == 0;
+}
+HB_EXPORT int hb_attn_diff_decode_splits(int D, int window, int max_pos) {
+  const int chunk = D == 64 ? AD_WARPS * 128 : AD_WARPS * 64, all = max_pos / chunk + 1;
+  return window > 0 && (window - 1) / chunk + 2 < all ? (window - 1) / chunk + 2 : all;
+}
+HB_EXPORT int hb_attn_diff_decode(const void* q, const void* kc, const void* vc, long n_pages, const int* bt, int bt_stride,
+                                  const int* row_req, const int* pos, const float* gate, long ld_gate, int gate_off, void* out,
+                                  float* workspace, int* counters, int T, int H, int G, int D, int page_size, int window, float scale,
+                                  float lambda, float post, float eps, int max_pos, const int* q_len, int row_limit, const int* ctx_len,
+                                  int* status, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (!hb_attn_diff_decode_supported(H, G, D, page_size)) HB_FAIL("hb_attn_diff_decode: %d/%d heads of %d with pages of %d are not supported", H, G, D, page_size);
+  const int chunk = D == 64 ? AD_WARPS * 128 : AD_WARPS * 64, S = hb_attn_diff_decode_splits(D, window, max_pos), Hq = 2 * H;
+  const long cache_rows = n_pages * G * page_size;
+  if (T > 65535 || G > 65535 || S > 65535) HB_FAIL("hb_attn_diff_decode: %d rows / %d kv heads / %d chunks are beyond the grid limit", T, G, S);
+  if (!status || n_pages <= 0 || cache_rows >= (1L << 31)) HB_FAIL("hb_attn_diff_decode: no status word, or %ld cache rows", cache_rows);
+  if (S > 1 && (!workspace || !counters)) HB_FAIL("hb_attn_diff_decode: rows that span %d chunks need a workspace and counters", S);
+  if (((uintptr_t)q | (uintptr_t)out) & 15) HB_FAIL("hb_attn_diff_decode: q and out must be 16-byte aligned");
+  static int n_sm = 0;
+  if (!n_sm) {
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&n_sm, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) n_sm = 1;
+  }
+  const bool resident = D == 64 && (long)S * G * T <= n_sm;
+  const int rw = D == 128 ? 32 : resident ? 128 : 64;
+  const size_t smem = 2 * (size_t)(AD_WARPS * rw) * D * 2 + 16 * (size_t)D * 2 + 1024;
+  CUtensorMap mk, mv;
+  if (hb_make_tensor_map_bf16(&mk, kc, (uint64_t)cache_rows, (uint64_t)D, (uint64_t)D, (uint32_t)page_size)) return -1;
+  if (hb_make_tensor_map_bf16(&mv, vc, (uint64_t)cache_rows, (uint64_t)D, (uint64_t)D, (uint32_t)page_size)) return -1;
+  float* pa = workspace;
+  float* pm = workspace ? workspace + (size_t)T * Hq * S * D : nullptr;
+  const AdDiff df{gate, ld_gate, gate_off, lambda, post, eps};
+  const bool cl = S >= 2 && S <= 8 && T <= g_ad_cluster_rows;
+  const float sl2 = scale * 1.4426950408889634f;
+  int r;
+#define HB_AD_ARGS 2 * (H / G), dim3(S, G, T), smem, st, mk, mv, status, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, \
+                   bt, bt_stride, row_req, pos, (__nv_bfloat16*)out, pa, pm, Hq, G, page_size, window, sl2, chunk, S, q_len, row_limit, ctx_len, \
+                   counters, nullptr, nullptr, nullptr, df
+  if (D == 128) r = cl ? launch_decode<128, true, 32, 64, 32, true, false, true>(HB_AD_ARGS) : launch_decode<128, true, 32, 64, 32, false, false, true>(HB_AD_ARGS);
+  else if (resident) r = cl ? launch_decode<64, true, 64, 128, 128, true, false, true>(HB_AD_ARGS) : launch_decode<64, true, 64, 128, 128, false, false, true>(HB_AD_ARGS);
+  else r = cl ? launch_decode<64, true, 64, 128, 64, true, false, true>(HB_AD_ARGS) : launch_decode<64, true, 64, 128, 64, false, false, true>(HB_AD_ARGS);
+#undef HB_AD_ARGS
+  if (r) HB_FAIL("hb_attn_diff_decode: no kernel for %d heads a kv head", H / G);
+  HB_CHECK_LAUNCH("hb_attn_diff_decode");
   return 0;
 }

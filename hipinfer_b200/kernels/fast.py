@@ -29,6 +29,11 @@ _SIGS = {
     "hb_flash_prefill_supported": [_i, _i, _i],
     "hb_flash_prefill_tc": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p, _p, _p],
     "hb_flash_prefill_tc_supported": [_i, _i, _i, _i],
+    "hb_attn_diff_decode": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _l, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _f, _f, _f, _i, _p, _i, _p, _p, _p],
+    "hb_attn_diff_decode_supported": [_i, _i, _i, _i],
+    "hb_attn_diff_decode_splits": [_i, _i, _i],
+    "hb_flash_diff_tc": [_p, _p, _p, _l, _p, _i, _p, _p, _p, _p, _l, _i, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _f, _f, _i, _p, _p],
+    "hb_flash_diff_tc_supported": [_i, _i, _i, _i, _i],
     "hb_gemm_tc_rope_kv": [_p, _l, _p, _l, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
     "hb_attn_decode_supported": [_i, _i, _i],
     "hb_wait_selftest": [_p, _i, _p, _p],
@@ -40,7 +45,7 @@ _SIGS = {
     "hb_rows_norm_supported": [_i, _i],
 }
 _fns = {}
-_LAUNCHES = {"hb_rows_scaled_qkv_rope": 1, "hb_rows_scaled_swiglu": 1, "hb_rows_norm_qkv_rope": 1, "hb_rows_add": 1, "hb_rows_norm_swiglu": 1, "hb_gemm_tc_rope_kv": 1, "hb_gemm_stream_finish": 1, "hb_add_rmsnorm_slices": 1, "hb_rope_kv_slices": 1, "hb_gemm_tc": 1, "hb_gemm_stream": 1, "hb_attn_decode": 1, "hb_flash_prefill": 1, "hb_flash_prefill_tc": 1}
+_LAUNCHES = {"hb_rows_scaled_qkv_rope": 1, "hb_rows_scaled_swiglu": 1, "hb_rows_norm_qkv_rope": 1, "hb_rows_add": 1, "hb_rows_norm_swiglu": 1, "hb_gemm_tc_rope_kv": 1, "hb_gemm_stream_finish": 1, "hb_add_rmsnorm_slices": 1, "hb_rope_kv_slices": 1, "hb_gemm_tc": 1, "hb_gemm_stream": 1, "hb_attn_decode": 1, "hb_flash_prefill": 1, "hb_flash_prefill_tc": 1, "hb_flash_diff_tc": 1, "hb_attn_diff_decode": 1}
 _status = None
 
 EPI_F32, EPI_BF16, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_SLICES, EPI_GEGLU_BF16, EPI_GELU_BF16, EPI_RELU2_BF16 = 0, 1, 2, 3, 4, 5, 6, 7
@@ -502,6 +507,49 @@ def flash_prefill_tc(q, k_cache, v_cache, block_table, q_start, q_len, ctx_len, 
           out.data_ptr(), q.shape[0], q_len.numel(), int(max_q_len), n_heads, n_kv_heads, head_dim, page_size, int(window),
           float(scale), int(min_rows), status_word().data_ptr(), *_extras(distance, sink), _stream())
     return out
+
+
+DIFF_TC_MIN_ROWS = 65    # a step with a portion of at least this many rows gives its differential attention to the tcgen05 kernel
+
+
+def flash_diff_tc(q, k_cache, v_cache, batch, block_table, out, n_heads, n_kv_heads, dim, vdim, page_size, window, scale, lam, post, eps,
+                  gate, gate_offset, min_rows) -> bool:
+    """The tcgen05 flash kernel with two score maps a head for prompt portions (csrc/attention_diff_tc.cu); False where it does not
+    take the sizes or the step's portions are short."""
+    if (PLAIN_ONLY or q.dtype != torch.bfloat16 or batch.max_q_len < DIFF_TC_MIN_ROWS or not scale > 0
+            or not _fn("hb_flash_diff_tc_supported")(n_heads, n_kv_heads, dim, vdim, page_size)):
+        return False
+    ld = 0 if gate is None else gate.stride(0)
+    if gate is not None and (ld % 2 or gate_offset % 2 or gate.data_ptr() % 8):
+        return False
+    _call("hb_flash_diff_tc", q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[0], block_table.data_ptr(),
+          block_table.stride(0), batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_ctx_len.data_ptr(),
+          None if gate is None else gate.data_ptr(), ld, int(gate_offset), out.data_ptr(), q.shape[0], batch.n_requests,
+          batch.max_q_len, n_heads, n_kv_heads, dim, vdim, page_size, int(window), float(scale), float(lam), float(post), float(eps),
+          int(min_rows), status_word().data_ptr(), _stream())
+    return True
+
+
+def attention_diff_decode(q, k_cache, v_cache, batch, block_table, out, n_heads, n_kv_heads, dim, vdim, page_size, window, scale, lam, post,
+                          eps, gate, gate_offset, max_pos, q_len=None, row_limit=0) -> bool:
+    """Differential attention of single rows by the TMA decode kernel (csrc/attention_fast.cu, DIFF): values as wide as the two maps
+    together (64 or 128), at most four heads a kv head. False where it does not take the sizes."""
+    D = 2 * dim
+    if (PLAIN_ONLY or q.dtype != torch.bfloat16 or vdim != D or not scale > 0 or (k_cache.data_ptr() | v_cache.data_ptr()) % 16
+            or not _fn("hb_attn_diff_decode_supported")(n_heads, n_kv_heads, D, page_size)):
+        return False
+    T = q.shape[0]
+    splits = _fn("hb_attn_diff_decode_splits")(D, int(window), int(max_pos))
+    ws = torch.empty(T * 2 * n_heads * splits * (D + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+    cnt = _decode_counters(q.device, T * n_kv_heads) if splits > 1 else None
+    p = lambda t: None if t is None else t.data_ptr()
+    rows_are_requests = batch.max_q_len == 1 and T == batch.n_requests
+    _call("hb_attn_diff_decode", q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[0], block_table.data_ptr(),
+          block_table.stride(0), None if rows_are_requests else batch.row_request.data_ptr(), batch.positions.data_ptr(), p(gate),
+          0 if gate is None else gate.stride(0), int(gate_offset), out.data_ptr(), p(ws), p(cnt), T, n_heads, n_kv_heads, D, page_size,
+          int(window), float(scale), float(lam), float(post), float(eps), int(max_pos), p(q_len), int(row_limit),
+          batch.req_ctx_len.data_ptr(), status_word().data_ptr(), _stream())
+    return True
 
 
 FLASH_MIN_ROWS = 16     # portions of at least this many rows go to the flash kernel, shorter ones to the row kernel

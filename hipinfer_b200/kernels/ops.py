@@ -365,7 +365,11 @@ def attention_window(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
              and getattr(batch, "max_q_len", 0) >= WINDOW_FLASH_MIN_ROWS
              and _fn("mixers", "hb_attn_window_flash_supported")(n_heads, n_kv_heads, dim, vdim, maps) == 1
              and (gate is None or (gate_ld % 2 == 0 and gate_offset % 2 == 0)))
-    if flash:
+    if flash and keep_first == 0 and fast.flash_diff_tc(q, k_cache, v_cache, batch, bt, out, n_heads, n_kv_heads, dim, vdim, page_size, window,
+                                                        scale, lam, post, eps, gate, gate_offset, WINDOW_FLASH_MIN_ROWS):
+        if min(batch.h_q_len) >= WINDOW_FLASH_MIN_ROWS:
+            return out
+    elif flash:
         _call("mixers", "hb_attn_window_flash", q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), bt.data_ptr(), bt.stride(0),
               batch.req_q_start.data_ptr(), batch.req_q_len.data_ptr(), batch.req_ctx_len.data_ptr(), _ptr(gate), gate_ld,
               int(gate_offset), out.data_ptr(), batch.n_requests, batch.max_q_len, n_heads, n_kv_heads, dim, vdim, page_size,
@@ -378,6 +382,11 @@ def attention_window(q, k_cache, v_cache, batch, group: int, out, n_heads: int, 
     lib.hb_attn_window_rows_mma_workspace.restype = C.c_long
     max_pos = int(getattr(batch, "max_pos", 0)) or int(bt.shape[1]) * page_size - 1
     q_len_ptr = batch.req_q_len.data_ptr() if flash else None
+    # values as wide as both maps, no kept first tokens: the TMA decode kernel, with the maps of the group's heads as its rows
+    if (maps == 2 and norm and keep_first == 0 and not force_plain and not force_simt and hasattr(batch, "req_ctx_len")
+            and fast.attention_diff_decode(q, k_cache, v_cache, batch, bt, out, n_heads, n_kv_heads, dim, vdim, page_size, window, scale, lam,
+                                           post, eps, gate, gate_offset, max_pos, batch.req_q_len if flash else None, WINDOW_FLASH_MIN_ROWS)):
+        return out
     if (maps == 2 and norm and q.dtype == torch.bfloat16 and not fast.PLAIN_ONLY and not force_plain and not force_simt
             and _fn("mixers", "hb_attn_window_rows_mma_supported")(n_heads, n_kv_heads, dim, vdim, maps) == 1):
         # the heads of a kv head as the rows of a warp MMA tile
