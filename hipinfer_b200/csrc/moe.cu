@@ -23,7 +23,7 @@
 //   moe_grouped_kernel      a block per (expert, tile of output features): the expert's weights are read once for all of
 //   moe_grouped_mma_kernel  its rows (a round of them at a time), for the gate/up product and for the down product;
 //                           nothing on the host, so the step replays from a CUDA graph. The second is the bfloat16 form on
-//                           warp MMAs, the first takes any element types and sizes
+//                           warp MMAs, with the activation in the gate/up product; the first takes any element types and sizes
 // Many rows (prompt portions): the (row, choice) pairs are sorted by expert, so that each expert's rows are one
 // contiguous block that an ordinary product takes
 //   moe_sort_kernel         offsets [E + 1], pos [pair] -> sorted row, src [sorted row] -> pair
@@ -304,6 +304,13 @@ HB_EXPORT int hb_moe_down_rows(const void* act, int a_dt, const void* wd, int w_
 // ---------------------------------------------------------------------------------------------------------------------
 constexpr int MX_THREADS = 256, MX_RB = 8, MX_NW = 4, MX_TILE = (MX_THREADS / 32) * MX_NW;
 
+// 16 bytes of a weight: read once a step, so not kept in L1, which the rows share.
+__device__ __forceinline__ uint4 hb_ldg_once(const uint4* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+
 template <typename T> struct MxVec4;
 template <> struct MxVec4<float> { using type = float4; };
 template <> struct MxVec4<__nv_bfloat16> { using type = uint2; };
@@ -405,13 +412,17 @@ __global__ void __launch_bounds__(MX_THREADS) moe_grouped_kernel(const TA* __res
   }
 }
 
-// The same product on warp MMAs (bfloat16 rows and weights, K a multiple of 32). The weights are the MMA's row operand,
-// 16 output features a warp, and come straight from memory: a lane reads 8 consecutive k of feature g and of feature
-// g + 8 (16 bytes each) per block of 32 k; the rows are the column operand, 8 a tile, up to 4 tiles a round, from shared
-// memory in segments of MM_KS k (twice and four times as many where a round has at most 16 or 8 rows). Inside a block of 32 k the lanes' k are dealt to the MMA's k slots in another order than
-// memory's, the same for both operands, which a sum over k does not see. 32-bit accumulation; a (row, feature) sum does
-// not depend on the other rows of the round.
-constexpr int MM_THREADS = 128, MM_KS = 1024, MM_LD = MM_KS + 32, MM_ROWS = 32, MM_TILE = 16 * (MM_THREADS / 32);
+// The same product on warp MMAs (bfloat16 rows and weights, K a multiple of 32), and the gate/up product with its activation. A
+// warp owns 16 weight rows, the MMA's row operand, over one of KW equal parts of K; the rows are the column operand, 8 a tile, up
+// to 4 tiles a round. Both come straight from memory (the rows from L1 and L2: every warp of a block reads the same ones): a lane
+// reads 8 consecutive k (16 bytes) of weight rows g and g + 8 and of row g of every tile per block of 32 k. Inside a block of 32 k
+// the lanes' k are dealt to the MMA's k slots in another order than memory's, the same for both operands, which a sum over k does
+// not see. The loads of the next MU blocks are under way while this one's products run: no shared memory and no barrier between
+// a warp and its weights. The parts of K are added in their order through shared memory. 32-bit accumulation; a (row, feature) sum
+// does not depend on the other rows of the round.
+// ACT: the 16 weight rows are 8 gate rows and the 8 up rows that go with them, so that a thread holds both halves of its hidden
+// units: it applies the activation and the pair's weight and writes bfloat16.
+constexpr int MM_THREADS = 128, MM_WARPS = MM_THREADS / 32, MM_ROWS = 32;
 
 __device__ __forceinline__ void mm_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -419,84 +430,158 @@ __device__ __forceinline__ void mm_mma(float (&c)[4], uint32_t a0, uint32_t a1, 
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <int NT>
-__device__ __forceinline__ void mm_round(const __nv_bfloat16* __restrict__ a, long lda, const int* mm_row, int nr,
-                                         const __nv_bfloat16* __restrict__ we, float* __restrict__ out, __nv_bfloat16* rows, int g0,
-                                         int n0, int Nout, int K) {
-  constexpr int KS = MM_KS * 4 / NT, LD = KS + 32;           // the same shared memory holds fewer rows of more k
-  const int tid = threadIdx.x, lane = tid & 31, g = lane >> 2, t = lane & 3;
+struct MmArgs {
+  const __nv_bfloat16* a;      // the rows
+  long lda;
+  const int* src;              // sorted row -> pair, or null: the rows are sorted already
+  int top;
+  const __nv_bfloat16* w;      // [E][Nw][K]
+  const int* offsets;          // [E + 1]
+  const float* weight;         // ACT: [pairs]
+  __nv_bfloat16* act;          // ACT: [sorted rows][Nout]
+  float* out;                  // else: [sorted rows][Nout]
+  int Nout, Nw, K, at_output;
+};
+
+template <int NT, int KW, bool ACT>
+__device__ __forceinline__ void mm_round(const MmArgs& A, const __nv_bfloat16* __restrict__ we, int g0, int nr, float* red) {
+  constexpr int MU = NT == 4 ? 2 : 4, FT = ACT ? 8 : 16, TILES = MM_WARPS / KW;     // blocks of 32 k a stage; features and tiles
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int tile = warp / KW, part = warp % KW, n0 = (blockIdx.x * TILES + tile) * FT;
+  const int nb = A.K >> 5, b0 = nb * part / KW, b1 = nb * (part + 1) / KW;
+  // features past the end read the last one's weights, rows past the round's end its first row: their sums are not stored
+  const int ra = min(n0 + g, A.Nout - 1), rb = ACT ? A.Nout + ra : min(n0 + g + 8, A.Nout - 1);
+  const uint4* wa = (const uint4*)(we + (size_t)ra * A.K) + t;
+  const uint4* wb = (const uint4*)(we + (size_t)rb * A.K) + t;
+  const uint4* row[NT];
+#pragma unroll
+  for (int nt = 0; nt < NT; nt++) {
+    const int r = g0 + (nt * 8 + g < nr ? nt * 8 + g : 0);
+    row[nt] = (const uint4*)(A.a + (size_t)(A.src ? A.src[r] / A.top : r) * A.lda) + t;
+  }
   float acc[NT][4];
 #pragma unroll
   for (int nt = 0; nt < NT; nt++)
 #pragma unroll
     for (int i = 0; i < 4; i++) acc[nt][i] = 0.f;
-  // features past the end read the last feature's weights; their sums are not stored
-  const __nv_bfloat16* wa = we + (size_t)min(n0 + g, Nout - 1) * K + t * 8;
-  const __nv_bfloat16* wb = we + (size_t)min(n0 + g + 8, Nout - 1) * K + t * 8;
-  for (int k0 = 0; k0 < K; k0 += KS) {
-    const int kn = min(KS, K - k0), per = kn >> 3;
-    __syncthreads();                                        // the segment before has been read; mm_row is written
-    for (int r = 0; r < nr; r++) {
-      const __nv_bfloat16* ar = a + (size_t)mm_row[r] * lda + k0;
-#pragma unroll 4
-      for (int i = tid; i < per; i += MM_THREADS) *(uint4*)(rows + (size_t)r * LD + 8 * i) = *(const uint4*)(ar + 8 * i);
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  uint4 A0[MU], A1[MU], B[MU][NT];
+  auto load = [&](int b, uint4 (&x0)[MU], uint4 (&x1)[MU], uint4 (&y)[MU][NT]) {
+#pragma unroll
+    for (int u = 0; u < MU; u++) {
+      const bool in = b + u < b1;
+      x0[u] = in ? hb_ldg_once(wa + (b + u) * 4) : zero;
+      x1[u] = in ? hb_ldg_once(wb + (b + u) * 4) : zero;
     }
-    __syncthreads();
-#pragma unroll 4
-    for (int kb = 0; kb < kn; kb += 32) {
-      const uint4 A0 = *(const uint4*)(wa + k0 + kb), A1 = *(const uint4*)(wb + k0 + kb);
+#pragma unroll
+    for (int u = 0; u < MU; u++)
+#pragma unroll
+      for (int nt = 0; nt < NT; nt++) y[u][nt] = b + u < b1 ? row[nt][(b + u) * 4] : zero;
+  };
+  load(b0, A0, A1, B);
+  for (int b = b0; b < b1; b += MU) {
+    uint4 N0[MU], N1[MU], NB[MU][NT];
+    load(b + MU, N0, N1, NB);
+#pragma unroll
+    for (int u = 0; u < MU; u++)
 #pragma unroll
       for (int nt = 0; nt < NT; nt++) {
-        // rows past nr hold whatever shared memory held: a row is a column of the MMA, and its sums are not stored
-        const uint4 B = *(const uint4*)(rows + (size_t)(nt * 8 + g) * LD + kb + t * 8);
-        mm_mma(acc[nt], A0.x, A1.x, A0.y, A1.y, B.x, B.y);
-        mm_mma(acc[nt], A0.z, A1.z, A0.w, A1.w, B.z, B.w);
+        mm_mma(acc[nt], A0[u].x, A1[u].x, A0[u].y, A1[u].y, B[u][nt].x, B[u][nt].y);
+        mm_mma(acc[nt], A0[u].z, A1[u].z, A0[u].w, A1[u].w, B[u][nt].z, B[u][nt].w);
       }
+#pragma unroll
+    for (int u = 0; u < MU; u++) {
+      A0[u] = N0[u];
+      A1[u] = N1[u];
+#pragma unroll
+      for (int nt = 0; nt < NT; nt++) B[u][nt] = NB[u][nt];
     }
+  }
+  if constexpr (KW > 1) {
+    __syncthreads();                                        // the round before has read its sums
+    if (part > 0) {
+#pragma unroll
+      for (int nt = 0; nt < NT; nt++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) red[((warp * NT + nt) * 4 + i) * 32 + lane] = acc[nt][i];
+    }
+    __syncthreads();
+    if (part > 0) return;
+#pragma unroll
+    for (int q = 1; q < KW; q++)
+#pragma unroll
+      for (int nt = 0; nt < NT; nt++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) acc[nt][i] += red[(((warp + q) * NT + nt) * 4 + i) * 32 + lane];
   }
 #pragma unroll
   for (int nt = 0; nt < NT; nt++)
 #pragma unroll
-    for (int i = 0; i < 4; i++) {
-      const int r = nt * 8 + 2 * t + (i & 1), n = n0 + g + (i >> 1) * 8;
-      if (r < nr && n < Nout) out[(size_t)(g0 + r) * Nout + n] = acc[nt][i];
+    for (int i = 0; i < 2; i++) {
+      const int r = nt * 8 + 2 * t + i;
+      if (r >= nr) continue;
+      if constexpr (ACT) {
+        if (n0 + g >= A.Nout) continue;
+        const float sw = A.weight[A.src[g0 + r]], s = A.at_output ? 1.f : sw, so = A.at_output ? sw : 1.f;
+        const float gt = s * acc[nt][i], up = s * acc[nt][2 + i];
+        A.act[(size_t)(g0 + r) * A.Nout + n0 + g] = __float2bfloat16_rn(gt / (1.f + expf(-gt)) * up * so);
+      } else {
+        if (n0 + g < A.Nout) A.out[(size_t)(g0 + r) * A.Nout + n0 + g] = acc[nt][i];
+        if (n0 + g + 8 < A.Nout) A.out[(size_t)(g0 + r) * A.Nout + n0 + g + 8] = acc[nt][2 + i];
+      }
     }
 }
 
-__global__ void __launch_bounds__(MM_THREADS) moe_grouped_mma_kernel(const __nv_bfloat16* __restrict__ a, long lda,
-                                                                     const int* __restrict__ src, int top,
-                                                                     const __nv_bfloat16* __restrict__ w,
-                                                                     const int* __restrict__ offsets, float* __restrict__ out,
-                                                                     int Nout, int K) {
-  extern __shared__ __align__(16) unsigned char mx_raw[];
-  __shared__ int mm_row[MM_ROWS];
-  __nv_bfloat16* rows = (__nv_bfloat16*)mx_raw;             // [MM_ROWS][MM_LD], or half the rows of twice the k, or a quarter of four times
+template <int KW, bool ACT>
+__global__ void __launch_bounds__(MM_THREADS, 3) moe_grouped_mma_kernel(MmArgs A) {
+  __shared__ float red[KW > 1 ? MM_WARPS * 4 * 4 * 32 : 1];
   hb_pdl_launch();
   hb_pdl_wait();
-  const int e = blockIdx.y, lo = offsets[e], hi = offsets[e + 1];
-  if (lo >= hi) return;
-  const int tid = threadIdx.x, warp = tid >> 5;
-  const int n0 = blockIdx.x * MM_TILE + warp * 16;
-  const __nv_bfloat16* we = w + (size_t)e * Nout * K;
+  const int e = blockIdx.y, lo = A.offsets[e], hi = A.offsets[e + 1];
+  const __nv_bfloat16* we = A.w + (size_t)e * A.Nw * A.K;
   for (int g0 = lo; g0 < hi; g0 += MM_ROWS) {
     const int nr = min(MM_ROWS, hi - g0);
-    __syncthreads();                                        // the round before has read its row numbers
-    if (tid < nr) mm_row[tid] = src ? src[g0 + tid] / top : g0 + tid;
-    if (nr <= 8) mm_round<1>(a, lda, mm_row, nr, we, out, rows, g0, n0, Nout, K);
-    else if (nr <= 16) mm_round<2>(a, lda, mm_row, nr, we, out, rows, g0, n0, Nout, K);
-    else mm_round<4>(a, lda, mm_row, nr, we, out, rows, g0, n0, Nout, K);
+    if (nr <= 8) mm_round<1, KW, ACT>(A, we, g0, nr, red);
+    else if (nr <= 16) mm_round<2, KW, ACT>(A, we, g0, nr, red);
+    else mm_round<4, KW, ACT>(A, we, g0, nr, red);
   }
 }
 
+static bool mm_ok(const void* a, int a_dt, long lda, const void* w, int w_dt, int K) {
+  return a_dt == HB_BF16 && w_dt == HB_BF16 && K % 32 == 0 && lda % 8 == 0 && !(((uintptr_t)a | (uintptr_t)w) & 15);
+}
+
+template <bool ACT>
+static void mm_launch(const MmArgs& A, int E, int parts, cudaStream_t s) {
+  // the parts of K follow from K alone: short walks, and enough warps to fill the machine when only a few experts have rows
+  constexpr int FT = ACT ? 8 : 16;
+  const int tiles = (A.Nout + FT - 1) / FT, kw = parts ? parts : A.K >= 512 ? 4 : A.K >= 256 ? 2 : 1;
+  const dim3 grid((tiles * kw + MM_WARPS - 1) / MM_WARPS, E);
+  if (kw == 1) hb_launch(moe_grouped_mma_kernel<1, ACT>, grid, dim3(MM_THREADS), 0, s, A);
+  else if (kw == 2) hb_launch(moe_grouped_mma_kernel<2, ACT>, grid, dim3(MM_THREADS), 0, s, A);
+  else hb_launch(moe_grouped_mma_kernel<4, ACT>, grid, dim3(MM_THREADS), 0, s, A);
+}
+
+// act[r] (bfloat16, sorted rows) = silu(s g) * (s u) times the rest of the pair's weight, [g | u] = w[e] row: the gate/up product
+// with its activation in one kernel. parts: of K, 1, 2 or 4 (0: what suits the sizes). Returns 1 (nothing done) where the sizes or element types are not its.
+HB_EXPORT int hb_moe_grouped_act(const void* a, int a_dt, long lda, const int* src, int top, const void* w, int w_dt, const int* offsets,
+                                 const float* weight, void* act, int E, int F, int K, int at_output, int parts, cudaStream_t s) {
+  if (parts != 0 && parts != 1 && parts != 2 && parts != 4) HB_FAIL("hb_moe_grouped_act: %d parts of K", parts);
+  if (E <= 0 || F <= 0 || K <= 0) return 0;
+  if (!mm_ok(a, a_dt, lda, w, w_dt, K) || !src || E > 65535) return 1;
+  mm_launch<true>(MmArgs{(const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, weight, (__nv_bfloat16*)act, nullptr, F, 2 * F,
+                         K, at_output}, E, parts, s);
+  HB_CHECK_LAUNCH("hb_moe_grouped_act");
+  return 0;
+}
+
 HB_EXPORT int hb_moe_grouped(const void* a, int a_dt, long lda, const int* src, int top, const void* w, int w_dt,
-                             const int* offsets, float* out, int E, int Nout, int K, cudaStream_t s) {
+                             const int* offsets, float* out, int E, int Nout, int K, int parts, cudaStream_t s) {
+  if (parts != 0 && parts != 1 && parts != 2 && parts != 4) HB_FAIL("hb_moe_grouped: %d parts of K", parts);
   if (E <= 0 || Nout <= 0 || K <= 0) return 0;
   if (E > 65535) HB_FAIL("hb_moe_grouped: %d experts are too many for this kernel", E);
-  if (a_dt == HB_BF16 && w_dt == HB_BF16 && K % 32 == 0 && lda % 8 == 0 && !(((uintptr_t)a | (uintptr_t)w) & 15)) {
-    const size_t smem = (size_t)MM_ROWS * MM_LD * sizeof(__nv_bfloat16);
-    cudaFuncSetAttribute(moe_grouped_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(moe_grouped_mma_kernel, dim3((Nout + MM_TILE - 1) / MM_TILE, E), dim3(MM_THREADS), smem, s,
-              (const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, out, Nout, K);
+  if (mm_ok(a, a_dt, lda, w, w_dt, K)) {
+    mm_launch<false>(MmArgs{(const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, nullptr, nullptr, out, Nout, Nout, K, 0}, E, parts, s);
     HB_CHECK_LAUNCH("hb_moe_grouped");
     return 0;
   }

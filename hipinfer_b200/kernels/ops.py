@@ -77,7 +77,8 @@ _SIGS = {
         "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p],
         "hb_moe_down_rows": [_p, _i, _p, _i, _p, _p, _l, _i, _i, _i, _i, _i, _p, _l, _p, _p],
         "hb_moe_sort": [_p, _p, _p, _p, _i, _i, _p],
-        "hb_moe_grouped": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _i, _i, _i, _p],
+        "hb_moe_grouped": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p],
+        "hb_moe_grouped_act": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p],
         "hb_moe_gather": [_p, _i, _l, _p, _p, _i, _i, _i, _p, _p],
         "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
         "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p, _p, _i, _l, _p, _p],
@@ -1462,7 +1463,7 @@ def moe_sort(expert: torch.Tensor, n_experts: int):
 
 
 def moe_grouped(a: torch.Tensor, src: Optional[torch.Tensor], top: int, w: torch.Tensor, offsets: torch.Tensor,
-                out: torch.Tensor) -> torch.Tensor:
+                out: torch.Tensor, parts: int = 0) -> torch.Tensor:
     """out[r] = w[e] a[row(r)] for the sorted rows r of every expert e (offsets[e] <= r < offsets[e + 1]); row(r) is
     src[r] // top where src is given (the step's input rows), else r. w [E, Nout, K]; out float32 [sorted rows, Nout].
     An expert's weights are read once for all of its rows; nothing is read by the host. Sorted rows of experts beyond E
@@ -1473,8 +1474,34 @@ def moe_grouped(a: torch.Tensor, src: Optional[torch.Tensor], top: int, w: torch
     assert w.is_contiguous() and a.shape[1] == K and out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == Nout
     assert offsets.numel() >= E + 1 and offsets.dtype == torch.int32 and (src is None or src.dtype == torch.int32)
     _call("hybrid", "hb_moe_grouped", a.data_ptr(), _dt(a), a.stride(0), _ptr(src), int(top), w.data_ptr(), _dt(w),
-          offsets.data_ptr(), out.data_ptr(), E, Nout, K, _stream())
+          offsets.data_ptr(), out.data_ptr(), E, Nout, K, int(parts), _stream())
     return out
+
+
+def moe_grouped_fast(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor) -> bool:
+    """Whether moe_grouped_act and moe_grouped run on warp MMAs for these rows and weights."""
+    return (xn.dtype == wgu.dtype == wdown.dtype == torch.bfloat16 and wgu.shape[2] % 32 == 0 and wdown.shape[2] % 32 == 0
+            and xn.stride(0) % 8 == 0 and (xn.data_ptr() | wgu.data_ptr() | wdown.data_ptr()) % 16 == 0)
+
+
+def moe_grouped_act(xn: torch.Tensor, src: torch.Tensor, top: int, wgu: torch.Tensor, offsets: torch.Tensor, score: torch.Tensor,
+                    act: torch.Tensor, at_output: bool = False, parts: int = 0) -> bool:
+    """moe_grouped of the gate/up weights [E, 2F, W] and moe_act as one kernel: act [sorted rows, F] (bfloat16). False where it does
+    not take the sizes or element types (nothing was done). parts (here and in moe_grouped): K is summed in 1, 2 or 4 parts by
+    warps of their own (0: what suits the sizes)."""
+    _need_cuda(xn, src, wgu, offsets, score, act)
+    _rows_contiguous(xn, "moe_grouped_act in")
+    E, F2, W = wgu.shape
+    assert wgu.is_contiguous() and xn.shape[1] == W and offsets.numel() >= E + 1 and act.is_contiguous() and act.shape[1] * 2 == F2
+    if act.dtype != torch.bfloat16:
+        return False
+    r = _fn("hybrid", "hb_moe_grouped_act")(xn.data_ptr(), _dt(xn), xn.stride(0), src.data_ptr(), int(top), wgu.data_ptr(), _dt(wgu),
+                                            offsets.data_ptr(), score.data_ptr(), act.data_ptr(), E, F2 // 2, W, 1 if at_output else 0,
+                                            int(parts), _stream())
+    if r < 0:
+        raise KernelError(library.load("hybrid").hb_last_error().decode())
+    library.launches[0] += r == 0
+    return r == 0
 
 
 def moe_gather(xn: torch.Tensor, src: torch.Tensor, top: int, limit: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -22,8 +22,9 @@ With `identity` the last that many of the experts + identity router rows are exp
 With `shared_size` a shared expert of the same form and that size runs for every token and is added; with `shared_gate` its
 result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits). One without a gate is a gated
 feed-forward like any other and runs on its kernels (parts/feed_forward.py).
-Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: a few rows one
-by one, more of them sorted by expert so that an expert's weights are read once for all of its rows. A step with prompt
+Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: sorted by expert so
+that an expert's weights are read once for all of its rows (in 32-bit, and at sizes the warp-MMA kernels do not take, a few
+rows run one by one). A step with prompt
 portions sorts its (row, choice) pairs by expert and gives each expert's block of rows to the ordinary products (the
 tensor-core kernels in bfloat16), for which the host reads the experts' row counts once a layer.
 
@@ -45,7 +46,7 @@ from .registry import Part, register_part, to_compute
 
 SORTED_MIN_PAIRS = 64     # fewer (row, choice) pairs than this never go to the ordinary products
 SHARED_MIN_ROWS = 9       # fewer rows run the shared expert row by row
-GROUPED_MIN_PAIRS = 20    # fewer than this run row by row; from here on an expert's rows share one pass over its weights
+GROUPED_MIN_PAIRS = 20    # fewer than this run row by row where the grouped kernels are the any-size ones
 
 
 class RoutedFF(Part):
@@ -81,7 +82,7 @@ class RoutedFF(Part):
         self.shared = int(params.get("shared_size") or 0)
         self.shared_gated = bool(params.get("shared_gate", False)) and self.shared > 0
         self.shared_prefix = prefix + params.get("shared_prefix", "mlp.shared")
-        self.shared_gate = self.s_gu = self.s_down = self.index = self.shared_ff = None
+        self.shared_gate = self.s_gu = self.s_down = self.index = self.bounds = self.shared_ff = None
         if self.shared and not self.shared_gated:
             self.shared_ff = GatedFF(dict(hidden_size=self.hidden, intermediate_size=self.shared, activation="silu",
                                           **{k + "_name": f"{params.get('shared_prefix', 'mlp.shared')}.{k}" for k in ("gate", "up", "down")}),
@@ -144,18 +145,22 @@ class RoutedFF(Part):
         if self.index is None or self.index[0].numel() < T:
             n = max(T, 2048)
             self.index = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, 1, dtype=torch.int32, device=dev))
+            self.bounds = torch.tensor([[0, t] for t in range(SHARED_MIN_ROWS)], dtype=torch.int32, device=dev)
         return tuple(t[:T] for t in self.index)
 
     def _add_shared(self, xn, x, weight):
         """x += weight * shared expert: the weight enters at the activation in 32-bit (the down product is linear)."""
         T, F = xn.shape[0], self.shared
         rows, zeros = self._row_index(T, xn.device)
+        act = torch.empty(T, F, dtype=self.ctx.dtype, device=xn.device)
         if T < SHARED_MIN_ROWS:
+            if ops.moe_grouped_act(xn, rows, 1, self.s_gu.t.unsqueeze(0), self.bounds[T], weight, act, True):
+                ops.linear_into_stream(act, self.s_down, x)
+                return
             ops.moe_rows(xn, self.s_gu.t.unsqueeze(0), self.s_down.t.unsqueeze(0), zeros, weight, x, True)
             return
         gu = torch.empty(T, 2 * F, dtype=torch.float32, device=xn.device)
         ops.linear(xn, self.s_gu, gu)
-        act = torch.empty(T, F, dtype=self.ctx.dtype, device=xn.device)
         ops.moe_act(gu, rows, weight, act, True)
         ops.linear_into_stream(act, self.s_down, x)
 
@@ -169,17 +174,18 @@ class RoutedFF(Part):
             self.shared_ff.forward(xn, x, None)
         elif self.shared:
             self._add_shared(xn, x, shared_weight)
-        if T * top < GROUPED_MIN_PAIRS:
+        if T * top < GROUPED_MIN_PAIRS and not ops.moe_grouped_fast(xn, self.wgu, self.wdown):
             ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output, idw)
             return None
         offsets, pos, src = ops.moe_sort(expert, self.choices)
         # identity experts come last in the order: their sorted rows hold nothing
         limit, rows_in = (offsets[self.experts:], xn) if self.identity else (None, None)
         if getattr(batch, "max_q_len", 1) <= 1 or T * top < SORTED_MIN_PAIRS:
-            gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
-            ops.moe_grouped(xn, src, top, self.wgu, offsets, gu)
             act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
-            ops.moe_act(gu, src, score, act, self.at_output, limit)
+            if not ops.moe_grouped_act(xn, src, top, self.wgu, offsets, score, act, self.at_output):
+                gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
+                ops.moe_grouped(xn, src, top, self.wgu, offsets, gu)
+                ops.moe_act(gu, src, score, act, self.at_output, limit)
             planes.record(batch, "activation", act)
             ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
             ops.moe_grouped(act, None, 1, self.wdown, offsets, ys)
