@@ -64,6 +64,7 @@ struct RowsArgs {
   const __nv_bfloat16* next_w; __nv_bfloat16* xb; long ldxb; float* ssq_part;
   // A_SCALED: A is such an xb; the row's 1 / RMS comes from ssq_part (n_parts tiles) and is applied in the epilogue
   int n_parts;
+  int store;                             // ADD: out = the product, not out += it
 };
 
 __device__ __forceinline__ void rw_bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
@@ -313,7 +314,7 @@ __global__ void __launch_bounds__(RW_THREADS, 2) rows_product_kernel(const RowsA
           const int m = i >> 4, r = i & 15;
           const long n = (long)t * RW_R + r;
           if (i < EPI_ITEMS && m < a.M && n < a.N) {
-            pre_x[e] = __ldcg((const float*)a.out + (long)m * a.ldo + n);
+            if (!a.store) pre_x[e] = __ldcg((const float*)a.out + (long)m * a.ldo + n);
             if (a.next_w) pre_w[e] = __bfloat162float(a.next_w[n]);
           }
         } else if constexpr (EPI == RW_ROPE_KV) {
@@ -552,8 +553,9 @@ HB_EXPORT int hb_rows_norm_qkv_rope(const float* x, long ldx, const void* norm_w
 // `out` next): also xb [M, N] bf16 (row stride ldxb) = out * next_w, and ssq_part [ceil(N / 16)][16] floats = each 16-column
 // tile's share of the rows' sums of squares; hb_rows_scaled_* take those in place of the residual rows.
 HB_EXPORT int hb_rows_add(const void* act, long lda, const void* W, long ldw, float* out, long ldo, int M, int N, int K,
-                          const void* next_w, void* xb, long ldxb, float* ssq_part, int* status, cudaStream_t s) {
+                          const void* next_w, void* xb, long ldxb, float* ssq_part, int store, int* status, cudaStream_t s) {
   RowsArgs a = {};
+  a.store = store;
   a.A = act; a.lda = lda; a.W = (const __nv_bfloat16*)W; a.ldw = ldw; a.M = M; a.N = N; a.K = K; a.out = out; a.ldo = ldo;
   a.status = status; a.next_w = (const __nv_bfloat16*)next_w; a.xb = (__nv_bfloat16*)xb; a.ldxb = ldxb; a.ssq_part = ssq_part;
   if (M <= 0 || N <= 0) return 0;

@@ -38,7 +38,7 @@ _SIGS = {
     "hb_attn_decode_supported": [_i, _i, _i],
     "hb_wait_selftest": [_p, _i, _p, _p],
     "hb_rows_norm_qkv_rope": [_p, _l, _p, _f, _p, _l, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
-    "hb_rows_add": [_p, _l, _p, _l, _p, _l, _i, _i, _i, _p, _p, _l, _p, _p, _p],
+    "hb_rows_add": [_p, _l, _p, _l, _p, _l, _i, _i, _i, _p, _p, _l, _p, _i, _p, _p],
     "hb_rows_scaled_qkv_rope": [_p, _l, _p, _i, _f, _p, _l, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
     "hb_rows_scaled_swiglu": [_p, _l, _p, _i, _f, _p, _l, _p, _l, _i, _i, _i, _p, _p],
     "hb_rows_norm_swiglu": [_p, _l, _p, _f, _p, _l, _p, _l, _i, _i, _i, _p, _p],
@@ -363,8 +363,8 @@ def norm_feed_applies(weight, rows) -> bool:
             and rows <= ROWS_MAX and weight.numel() % 32 == 0)
 
 
-def rows_add(act, w, out, feed: "NormFeed" = None) -> bool:
-    """out (fp32) += act @ w.T for a few bf16 rows, finished in one kernel (no slices). With feed (a NormFeed for the
+def rows_add(act, w, out, feed: "NormFeed" = None, store: bool = False) -> bool:
+    """out (fp32) += (store: =) act @ w.T for a few bf16 rows, finished in one kernel (no slices). With feed (a NormFeed for the
     norm of width N that reads `out` next) the kernel fills it as well. False: nothing done."""
     M, K = act.shape
     if (M > ROWS_LIMIT or not act.is_cuda or act.dtype != torch.bfloat16 or act.stride(1) != 1 or act.stride(0) % 8
@@ -374,7 +374,7 @@ def rows_add(act, w, out, feed: "NormFeed" = None) -> bool:
         feed = None
     _call("hb_rows_add", act.data_ptr(), act.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, w.shape[0],
           K, None if feed is None else feed.weight.data_ptr(), None if feed is None else feed.xb.data_ptr(),
-          0 if feed is None else feed.xb.stride(0), None if feed is None else feed.ssq.data_ptr(),
+          0 if feed is None else feed.xb.stride(0), None if feed is None else feed.ssq.data_ptr(), 1 if store else 0,
           status_word().data_ptr(), _stream())
     if feed is not None:
         feed.filled = True

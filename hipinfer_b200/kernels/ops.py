@@ -657,12 +657,13 @@ def linear_into_stream(a: torch.Tensor, w: Weight, x: torch.Tensor) -> torch.Ten
 
 
 def linear_rows32(a: torch.Tensor, w: Weight, out: torch.Tensor) -> torch.Tensor:
-    """out = a @ w.T as 32-bit rows for a 32-bit consumer. For a few bfloat16 rows the whole-K rows kernel adds into the
-    zeroed rows (one kernel behind a memset instead of a split-K product and the reduction of its slices); else `linear`."""
-    if a.is_cuda and a.dtype == torch.bfloat16 and out.dtype == torch.float32 and out.is_contiguous() and a.shape[0] <= 8:
-        out.zero_()
-        if linear_add_rows(a, w, out):
-            return out
+    """out = a @ w.T as 32-bit rows for a 32-bit consumer. For a few bfloat16 rows the whole-K rows kernel (one kernel
+    instead of a split-K product and the reduction of its slices); else `linear`."""
+    from . import fast
+
+    if (a.is_cuda and a.dtype == torch.bfloat16 and out.dtype == torch.float32 and out.is_contiguous() and a.shape[0] <= fast.ROWS_MAX
+            and fast.rows_add(a, w.t, out, store=True)):
+        return out
     return linear(a, w, out)
 
 
