@@ -10,6 +10,11 @@ scripts/bench.py:126-212, and reports GB/s or TFLOP/s from algorithmic bytes and
     python -m hipinfer_b200.kernels.microbench delta_rule --tokens 2048 --batch 1 --heads 32 --head-dim 64
     python -m hipinfer_b200.kernels.microbench attn_window --batch 8 --context 2048 --window 1024        (single rows)
     python -m hipinfer_b200.kernels.microbench attn_window --portion --tokens 2048 --window 1024         (a prompt portion)
+    python -m hipinfer_b200.kernels.microbench attn_window --keep 0 ...                                  (the same without kept first tokens)
+    python -m hipinfer_b200.kernels.microbench two_norms --m 2048 --n 2048
+    python -m hipinfer_b200.kernels.microbench rope_maps --m 2048 --heads 32 --kv-heads 8 --head-dim 64  (two maps a head, values --value-dim wide)
+    python -m hipinfer_b200.kernels.microbench router --m 2048 --k 2048 --experts 12
+    python -m hipinfer_b200.kernels.microbench experts --batch 64 --k 2048 --n 4096 --experts 8          (single rows, two experts each)
     python -m hipinfer_b200.kernels.microbench layernorm|polynorm|scale_add --m 2048 --n 2048
     python -m hipinfer_b200.kernels.microbench selective_scan --tokens 2048 --batch 1 --n 2048 --states 16   (a prompt portion)
     python -m hipinfer_b200.kernels.microbench selective_scan --tokens 1 --batch 64 --n 2048 --states 16     (single rows)
@@ -68,7 +73,7 @@ def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
     ap.add_argument("kernel", choices=["gemm_tc", "gemm_stream", "rows_add", "rows_swiglu", "rows_qkv", "attn_decode", "flash_prefill", "flash_prefill_tc", "rmsnorm",
                                        "delta_rule", "attn_window", "layernorm", "polynorm", "scale_add", "selective_scan", "residual_norm",
-                                       "matrix_memory", "gated_delta", "output_norm"])
+                                       "matrix_memory", "gated_delta", "output_norm", "two_norms", "rope_maps", "router", "experts"])
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=16384)
     ap.add_argument("--k", type=int, default=2048)
@@ -81,7 +86,9 @@ def main(argv=None) -> int:
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--head-dim", type=int, default=64)
     ap.add_argument("--page-size", type=int, default=16)
-    ap.add_argument("--window", type=int, default=1024, help="attn_window: the window (0: none); 4 first tokens are kept")
+    ap.add_argument("--window", type=int, default=1024, help="attn_window: the window (0: none)")
+    ap.add_argument("--keep", type=int, default=4, help="attn_window: first tokens that the window keeps (0: the TMA and tcgen05 kernels)")
+    ap.add_argument("--experts", type=int, default=8, help="experts, router: how many (--n is their width, --k the rows')")
     ap.add_argument("--value-dim", type=int, default=64, help="attn_window: width of a head's values (a score map is --head-dim / 2 wide)")
     ap.add_argument("--portion", action="store_true", help="attn_window: one request's portion of --tokens rows instead of --batch single rows")
     ap.add_argument("--states", type=int, default=16, help="selective_scan: states a channel (--n is the number of channels)")
@@ -244,12 +251,12 @@ def main(argv=None) -> int:
             batch = SimpleNamespace(block_tables=[bt], row_request=i32([0] * T), positions=i32(list(range(T))), max_q_len=T,
                                     n_requests=1, req_q_start=i32([0]), req_q_len=i32([T]), req_ctx_len=i32([0]), h_q_len=[T],
                                     max_pos=T - 1)
-            pairs = sum(min(p + 1, window + 4) if window else p + 1 for p in range(T))
+            pairs = sum(min(p + 1, window + a.keep) if window else p + 1 for p in range(T))
         else:
             batch = SimpleNamespace(block_tables=[bt], row_request=i32(list(range(R))), positions=i32([ctx] * R), max_q_len=1,
-                                    max_pos=ctx)
-            pairs = R * (min(ctx + 1, window + 4) if window else ctx + 1)
-        fn = lambda: ops.attention_window(q, kc, vc, batch, 0, y, H, G, D, E, 2, ps, window, 4, D ** -0.5, 0.5, 0.5, 1e-5, True,
+                                    max_pos=ctx, n_requests=R, req_ctx_len=i32([ctx] * R))
+            pairs = R * (min(ctx + 1, window + a.keep) if window else ctx + 1)
+        fn = lambda: ops.attention_window(q, kc, vc, batch, 0, y, H, G, D, E, 2, ps, window, a.keep, D ** -0.5, 0.5, 0.5, 1e-5, True,
                                           gate=gate)
         ms = timeit(fn, a.iters, a.flush)
         nbytes = pairs * G * (2 * D + E) * 2                   # single rows: every visible key and value once a kv head
@@ -257,6 +264,36 @@ def main(argv=None) -> int:
                    tflops=pairs * H * (4 * D + 4 * E) / ms / 1e9)
         if not rows:
             out.update(gbs=nbytes / ms / 1e6)
+    elif a.kernel == "two_norms":
+        x, w1, w2 = rnd(a.m, a.n), rnd(a.n), rnd(a.n)
+        ms = timeit(lambda: ops.two_norms(x, w1, w2, 1e-5, torch.bfloat16), a.iters, a.flush)
+        out.update(M=a.m, H=a.n, ms=ms, gbs=a.m * a.n * 8 / ms / 1e6)
+    elif a.kernel == "rope_maps":
+        H, G, D, E, ps, T = a.heads, a.kv_heads, a.head_dim // 2, a.value_dim, a.page_size, a.m
+        cols = H * 2 * D + G * 2 * D + G * E
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        proj, q, table = rnd(T, cols), torch.empty(T, H * 2 * D, device=dev, dtype=torch.bfloat16), ops.shared_rope_table(D, 10000.0, T, dev)
+        kc, vc = (torch.empty(-(-T // ps), G, ps, n, device=dev, dtype=torch.bfloat16) for n in (2 * D, E))
+        pos, slots = i32(list(range(T))), i32(list(range(T)))
+        ms = timeit(lambda: ops.rope_norm_store(proj, (0, H * 2 * D, H * 2 * D + G * 2 * D), pos, slots, table, D, "half", False, 0.0, q, kc,
+                                                vc, H * 2, G * 2, D, E, ps, maps=2), a.iters, a.flush)
+        out.update(rows=T, heads=H, kv_heads=G, map_dim=D, value_dim=E, ms=ms, gbs=T * cols * 6 / ms / 1e6)
+    elif a.kernel == "router":
+        x, w, c = rnd(a.m, a.k).bfloat16(), rnd(a.experts, a.k).bfloat16() * 0.02, rnd(a.experts).bfloat16() * 0.01
+        ms = timeit(lambda: ops.moe_route(x, w, 2, None, "softmax", c), a.iters, a.flush)
+        out.update(rows=a.m, experts=a.experts, K=a.k, ms=ms, gbs=(a.m + a.experts) * a.k * 2 / ms / 1e6)
+    elif a.kernel == "experts":
+        T, W, F, E = a.batch, a.k, a.n, a.experts
+        wgu, wd = rnd(E, 2 * F, W).bfloat16() * 0.02, rnd(E, W, F).bfloat16() * 0.02
+        ex = torch.stack([torch.randperm(E, generator=g, device=dev)[:2] for _ in range(T)]).to(torch.int32)
+        x, y, sc = rnd(T, W).bfloat16(), rnd(T, W), torch.rand(T, 2, generator=g, device=dev)
+        offsets, pos, src = ops.moe_sort(ex, E)
+        act, ys = torch.empty(2 * T, F, device=dev, dtype=torch.bfloat16), torch.empty(2 * T, W, device=dev)
+        used = int(ex.unique().numel())
+        up = timeit(lambda: ops.moe_grouped_act(x, src, 2, wgu, offsets, sc, act, True), a.iters, a.flush)
+        down = timeit(lambda: ops.moe_grouped(act, None, 1, wd, offsets, ys), a.iters, a.flush)
+        out.update(rows=T, experts=E, experts_used=used, gate_up_ms=up, gate_up_gbs=used * 4 * F * W / up / 1e6, down_ms=down,
+                   down_gbs=used * 2 * F * W / down / 1e6)
     elif a.kernel == "rmsnorm":
         x, w = rnd(a.m, a.n), torch.ones(a.n, device=dev, dtype=torch.bfloat16)
         y = torch.empty(a.m, a.n, device=dev, dtype=torch.bfloat16)

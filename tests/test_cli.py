@@ -162,3 +162,23 @@ def test_generate_serves_the_gakupel_architecture(tmp_path):
             assert float(top[0] - top[1]) < 1e-3 * float(steps[i].abs().max()), (i, got, want)
             break
     assert len(got) == len(want)
+
+
+@pytest.mark.gpu
+def test_generate_serves_the_selovik_architecture(tmp_path):
+    """The same command on a Selovik folder (a loop of three passes, a bigram embedding, identity experts): prompt portions of 8
+    tokens through the scheduler, then greedy decoding, in 32-bit: every token is the plain implementation's first choice after
+    those before it, or nearly ties with it."""
+    import selovik_models as tm
+
+    folder, cfg, w = tm.make_folder(tmp_path / "model", "a", seed=5, dtype=torch.float32)
+    prompt = tm.safe_tokens(cfg, w, 29, 8, 1e-3)
+    r = run([sys.executable, "-m", "hipinfer_b200", "generate", "--model", folder, "--tokens", *map(str, prompt), "--new", "6",
+             "--mode", "fp32", "--max-seq", "64", "--max-batch", "2", "--max-prefill", "8"])
+    assert r.returncode == 0, r.stderr[-2000:]
+    lines = r.stdout.strip().splitlines()
+    shape = ast.literal_eval(lines[-2])
+    assert shape["vocab"] == cfg["vocab"] and shape["hidden"] == cfg["width"]
+    got = ast.literal_eval(lines[-1])
+    logits = tm.plain.forward(cfg, w, prompt + got[:-1])[len(prompt) - 1:]
+    assert len(got) == 6 and all(float(row.max() - row[t]) < 1e-3 * float(row.abs().max()) for row, t in zip(logits, got))
