@@ -702,3 +702,217 @@ HB_EXPORT int hb_gemm_tc_rope_kv(const void* A, long lda, const void* W, long ld
   HB_CHECK_LAUNCH("hb_gemm_tc_rope_kv");
   return 0;
 }
+
+// ---------------------------------------------------------------------------------------------------------------------
+// The products of a routed layer's experts as ONE kernel: the rows are sorted by expert, expert e's are offsets[e] ..
+// offsets[e + 1] - 1 (on the device: nothing is read by the host), its weights rows e N .. of W [E N, K]. The kernel above, but a
+// tile is (expert, 128 of its rows, BN of its columns); experts one after the other, an expert's row tiles fastest, so that a
+// weight tile is read once from memory. A row tile may reach into the next expert's rows: those are computed and not stored.
+// epi 0: fp32 rows of N; epi 3: bf16 rows of N / 2 after act(gate) * up over 16-interleaved columns, with the pair's weight: it
+// multiplies the result (at_output) or the product's both halves.
+// ---------------------------------------------------------------------------------------------------------------------
+constexpr int GROUPED_MAX_E = 256;
+
+struct GroupedArgs {
+  const int* offsets;     // [E + 1]
+  const int* src;         // epi 3: sorted row -> pair
+  const float* weight;    // epi 3: [pairs]
+  int E, at_output;
+};
+
+template <int BN, int STAGES, int EPI, int MAX_E>
+__global__ void __launch_bounds__(192, 1) gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a,
+                                                                 const __grid_constant__ CUtensorMap map_w,
+                                                                 const __grid_constant__ CUtensorMap map_c, void* C, long ldc, int N,
+                                                                 int K, int* status, GroupedArgs g) {
+  using S = GemmSmem<BN, STAGES>;
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ int sh_row[MAX_E + 1], sh_tile[MAX_E + 1];      // first row and first tile of every expert
+  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint64_t* full = (uint64_t*)(smem + S::BAR_OFFSET);
+  uint64_t* empty = full + STAGES;
+  uint64_t* tmem_full = empty + STAGES;
+  uint64_t* tmem_empty = tmem_full + 2;
+  uint32_t* tmem_slot = (uint32_t*)(tmem_empty + 2);
+  volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
+
+  hb_pdl_launch();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n_tiles = (N + BN - 1) / BN, num_kb = (K + BK - 1) / BK;
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < STAGES; s++) { hb_mbar_init(&full[s], 1); hb_mbar_init(&empty[s], 1); }
+    for (int b = 0; b < 2; b++) { hb_mbar_init(&tmem_full[b], 1); hb_mbar_init(&tmem_empty[b], 4); }
+    *abort_flag = 0;
+    hb_fence_barrier_init();
+  }
+  if (warp == 4 && lane == 0) { hb_tma_prefetch_desc(&map_a); hb_tma_prefetch_desc(&map_w); hb_tma_prefetch_desc(&map_c); }
+  hb_pdl_wait();
+  if (warp == 5) {            // (only now: no kernel ahead can still be about to ask for tensor memory)
+    hb_tmem_alloc(tmem_slot, 2 * BN);
+    hb_tmem_relinquish();
+  }
+  for (int e = threadIdx.x; e <= g.E; e += 192) sh_row[e] = g.offsets[e];
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int run = 0;
+    for (int e = 0; e < g.E; e++) {
+      sh_tile[e] = run;
+      run += (sh_row[e + 1] - sh_row[e] + BM - 1) / BM * n_tiles;
+    }
+    sh_tile[g.E] = run;
+  }
+  hb_tc_fence_before();
+  __syncthreads();
+  hb_tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  const int num_tiles = sh_tile[g.E];
+  // tiles come in ascending order, so an expert is found by going on from the last one
+  auto place = [&](int tile, int& e, int& m0, int& n0) {
+    while (tile >= sh_tile[e + 1]) e++;
+    const int local = tile - sh_tile[e], mt = (sh_row[e + 1] - sh_row[e] + BM - 1) / BM;
+    m0 = sh_row[e] + (local % mt) * BM;
+    n0 = (local / mt) * BN;
+  };
+
+  if (warp == 4) {
+    if (lane == 0) {  // ---------------- TMA producer
+      uint32_t it = 0;
+      int e = 0, m0, n0;
+      bool ok = true;
+      for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
+        place(tile, e, m0, n0);
+        for (int kb = 0; kb < num_kb; kb++, it++) {
+          const uint32_t s = it % STAGES, ph = (it / STAGES) & 1;
+          if (!hb_mbar_wait(&empty[s], ph ^ 1, abort_flag)) { ok = false; break; }
+          hb_mbar_expect_tx(&full[s], S::STAGE_BYTES);
+          hb_tma_load_2d(smem + s * S::STAGE_BYTES, &map_a, &full[s], kb * BK, m0);
+          hb_tma_load_2d(smem + s * S::STAGE_BYTES + S::A_BYTES, &map_w, &full[s], kb * BK, e * N + n0);
+        }
+      }
+    }
+  } else if (warp == 5) {
+    if (lane == 0) {  // ---------------- MMA issuer
+      constexpr uint32_t idesc = hb_umma_idesc_bf16(BM, BN);
+      uint32_t it = 0, tile_i = 0;
+      bool ok = true;
+      for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x, tile_i++) {
+        const uint32_t buf = tile_i & 1, aph = (tile_i >> 1) & 1;
+        if (!hb_mbar_wait(&tmem_empty[buf], aph ^ 1, abort_flag)) break;
+        hb_tc_fence_after();
+        const uint32_t d = tmem_base + buf * BN;
+        for (int kb = 0; kb < num_kb; kb++, it++) {
+          const uint32_t s = it % STAGES, ph = (it / STAGES) & 1;
+          if (!hb_mbar_wait(&full[s], ph, abort_flag)) { ok = false; break; }
+          hb_tc_fence_after();
+          const uint64_t da = hb_umma_desc_k128(hb_smem_u32(smem + s * S::STAGE_BYTES));
+          const uint64_t db = hb_umma_desc_k128(hb_smem_u32(smem + s * S::STAGE_BYTES + S::A_BYTES));
+#pragma unroll
+          for (int k = 0; k < BK / 16; k++) hb_umma_bf16(d, da + 2 * k, db + 2 * k, idesc, (kb | k) != 0);
+          hb_umma_commit(&empty[s]);
+        }
+        if (ok) hb_umma_commit(&tmem_full[buf]);
+      }
+    }
+  } else {  // ---------------- epilogue warps 0..3
+    uint32_t tile_i = 0;
+    int e = 0, m0, n0;
+    for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x, tile_i++) {
+      place(tile, e, m0, n0);
+      const int hi = sh_row[e + 1], row0 = m0 + warp * 32, row = row0 + lane;
+      const uint32_t buf = tile_i & 1, aph = (tile_i >> 1) & 1;
+      float s_all = 1.f, s_up = 1.f;
+      if (EPI_IS_GLU(EPI) && row < hi) {
+        const float w = g.weight[g.src[row]];
+        if (g.at_output) s_up = w;
+        else s_all = w;
+      }
+      if (!hb_mbar_wait(&tmem_full[buf], aph, abort_flag)) break;
+      hb_tc_fence_after();
+      const uint32_t t0 = tmem_base + ((uint32_t)(warp * 32) << 16) + buf * BN;
+      const bool whole = row0 + 32 <= hi;          // all of the warp's rows are this expert's: out by TMA, else row by row
+#pragma unroll 1
+      for (int c = 0; c < BN / 32; c++) {
+        float v[32];
+        hb_tmem_ld32(t0 + c * 32, v);
+        if (n0 + c * 32 >= N) continue;
+        if (EPI_IS_GLU(EPI)) {
+#pragma unroll
+          for (int j = 0; j < 16; j++) { v[j] *= s_all; v[16 + j] *= s_all * s_up; }
+        }
+        if (whole) ts_chunk<EPI>(v, c, n0, N, row0, smem + S::STAGING_OFFSET + warp * 8192, lane, &map_c);
+        else epilogue_store<EPI>(v, C, ldc, row, n0 + c * 32, hi, N);
+      }
+      hb_tc_fence_before();
+      __syncwarp();
+      if (lane == 0) hb_mbar_arrive(&tmem_empty[buf]);
+    }
+    if (lane == 0) hb_tma_store_wait_all();   // before the shared memory is given up and the kernel ends
+  }
+
+  hb_tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) {
+    if (threadIdx.x == 0) atomicExch(status, 1);
+    __nanosleep(100000);  // let copies that may still be in flight land before the shared memory is given up
+  }
+  if (warp == 5) {
+    __syncwarp();
+    hb_tmem_dealloc(tmem_base, 2 * BN);
+  }
+}
+
+template <int BN, int STAGES, int EPI, int MAX_E>
+static int launch_grouped(const CUtensorMap& ma, const void* W, void* C, long ldc, long rows, int E, int N, int K, int* status,
+                          const GroupedArgs& g, cudaStream_t s) {
+  CUtensorMap mw, mc;
+  if (hb_make_tensor_map_bf16(&mw, W, (uint64_t)E * N, (uint64_t)K, (uint64_t)K, BN)) return -1;
+  if (EPI == EPI_F32) {
+    if (hb_make_tensor_map_f32_box32(&mc, C, (uint64_t)rows, (uint64_t)N, (uint64_t)ldc)) return -1;
+  } else if (hb_make_tensor_map_bf16(&mc, C, (uint64_t)rows, (uint64_t)N / 2, (uint64_t)ldc, 32)) {
+    return -1;
+  }
+  constexpr int smem = GemmSmem<BN, STAGES>::TOTAL_TS;
+  static_assert(smem + 8 * (MAX_E + 1) <= 227 * 1024, "shared memory of a block");
+  auto kern = gemm_tc_grouped_kernel<BN, STAGES, EPI, MAX_E>;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) HB_FAIL("hb_gemm_tc_grouped: %s", cudaGetErrorString(e));
+    configured = true;
+  }
+  cudaError_t e = hb_launch(kern, sm_count(), 192, smem, s, ma, mw, mc, C, ldc, N, K, status, g);
+  if (e != cudaSuccess) HB_FAIL("hb_gemm_tc_grouped: %s", cudaGetErrorString(e));
+  return 0;
+}
+
+// A [rows, K] bf16 sorted by expert, W [E, N, K] bf16, offsets int32 [E + 1] on the device (offsets[E] <= rows). epi 0: C fp32 [rows,
+// N]; epi 3: C bf16 [rows, N / 2], src and weight as above. tile_n 128 or 256 (0: chosen from the sizes).
+HB_EXPORT int hb_gemm_tc_grouped(const void* A, long lda, const void* W, int E, int N, int K, const int* offsets, void* C, long ldc,
+                                 long rows, int epi, const int* src, const float* weight, int at_output, int tile_n, int* status,
+                                 cudaStream_t s) {
+  if (rows <= 0 || E <= 0 || N <= 0) return 0;
+  if (E > GROUPED_MAX_E || (long)E * N >= (1L << 31) || rows >= (1L << 31)) HB_FAIL("hb_gemm_tc_grouped: %d experts of %d rows are beyond this kernel", E, N);
+  if (K <= 0 || (K & 7)) HB_FAIL("hb_gemm_tc_grouped: K = %d must be a positive multiple of 8 (16-byte rows for TMA)", K);
+  if (epi != EPI_F32 && epi != EPI_SWIGLU_BF16) HB_FAIL("hb_gemm_tc_grouped: unknown epilogue %d", epi);
+  if (epi == EPI_SWIGLU_BF16 && ((N & 31) || !src || !weight)) HB_FAIL("hb_gemm_tc_grouped: the gated epilogue needs N = %d to be a multiple of 32, and the pairs' weights", N);
+  if (((uintptr_t)C & 15) || (ldc & (epi == EPI_F32 ? 3 : 7))) HB_FAIL("hb_gemm_tc_grouped: C must be 16-byte aligned, rows too");
+  if (!status) HB_FAIL("hb_gemm_tc_grouped: no status word");
+  CUtensorMap ma;
+  if (hb_make_tensor_map_bf16(&ma, A, (uint64_t)rows, (uint64_t)K, (uint64_t)lda, BM)) return -1;
+  const GroupedArgs g{offsets, src, weight, E, at_output};
+  if (tile_n == 0) {   // the row tiles the experts will have, about: half a tile of every expert is padding
+    const double mt = (double)rows / BM + 0.5 * E;
+    auto cost = [&](int bn, double per_col) { const double t = mt * ((N + bn - 1) / bn) / sm_count(); return (double)(long)(t + 0.999) * bn * per_col; };
+    tile_n = cost(128, 1.35) < cost(256, 1.0) ? 128 : 256;
+  }
+  if (tile_n != 128 && tile_n != 256) HB_FAIL("hb_gemm_tc_grouped: tiles of %d columns", tile_n);
+  int r;
+#define HB_GR_ARGS ma, W, C, ldc, rows, E, N, K, status, g, s
+  if (E > 64) r = epi == EPI_F32 ? launch_grouped<128, 5, EPI_F32, GROUPED_MAX_E>(HB_GR_ARGS) : launch_grouped<128, 5, EPI_SWIGLU_BF16, GROUPED_MAX_E>(HB_GR_ARGS);
+  else if (epi == EPI_F32) r = tile_n == 256 ? launch_grouped<256, 4, EPI_F32, 64>(HB_GR_ARGS) : launch_grouped<128, 6, EPI_F32, 64>(HB_GR_ARGS);
+  else r = tile_n == 256 ? launch_grouped<256, 4, EPI_SWIGLU_BF16, 64>(HB_GR_ARGS) : launch_grouped<128, 6, EPI_SWIGLU_BF16, 64>(HB_GR_ARGS);
+#undef HB_GR_ARGS
+  if (r) return r;
+  HB_CHECK_LAUNCH("hb_gemm_tc_grouped");
+  return 0;
+}

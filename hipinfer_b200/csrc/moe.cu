@@ -205,11 +205,15 @@ __device__ __forceinline__ float moe_warp_dot(const TW* __restrict__ w, const fl
 
 constexpr int MG_THREADS = 256, MG_ROWS = 32;
 
+// An expert's gate and up rows take turns, grp of each (16: the layout of the gated epilogues; F: gate rows first): where hidden
+// unit j's gate row lies; its up row is grp further.
+__device__ __forceinline__ int moe_gate_row(int j, int grp) { return j / grp * 2 * grp + j % grp; }
+
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(MG_THREADS) moe_gate_up_rows_kernel(const TA* __restrict__ xn, long ldx,
                                                                       const TW* __restrict__ wgu, const int* __restrict__ expert,
                                                                       const float* __restrict__ weight, TO* __restrict__ act,
-                                                                      int W, int F, int top, int vec, int at_output, int E) {
+                                                                      int W, int F, int top, int vec, int at_output, int E, int grp) {
   extern __shared__ __align__(16) float mg_row[];      // [W]
   hb_pdl_launch();
   hb_pdl_wait();
@@ -220,18 +224,20 @@ __global__ void __launch_bounds__(MG_THREADS) moe_gate_up_rows_kernel(const TA* 
   const int e = expert[pair];
   const float sw = weight[pair];
   const float s = at_output ? 1.f : sw, so = at_output ? sw : 1.f;     // the weight multiplies the input, or the result
-  const TW* we = wgu + (size_t)e * 2 * F * W;          // [gate rows (F) | up rows (F)][W]
+  const TW* we = wgu + (size_t)e * 2 * F * W;          // gate and up rows in turn, grp of each
   const int j1 = min(F, (int)(blockIdx.x + 1) * MG_ROWS);
   for (int j = blockIdx.x * MG_ROWS + warp; j < j1; j += MG_THREADS / 32) {
-    const float g = s * moe_warp_dot(we + (size_t)j * W, mg_row, W, lane, vec);
-    const float u = s * moe_warp_dot(we + (size_t)(F + j) * W, mg_row, W, lane, vec);
+    const int jg = moe_gate_row(j, grp);
+    const float g = s * moe_warp_dot(we + (size_t)jg * W, mg_row, W, lane, vec);
+    const float u = s * moe_warp_dot(we + (size_t)(jg + grp) * W, mg_row, W, lane, vec);
     if (lane == 0) act[(size_t)pair * F + j] = hb_from_float<TO>(g / (1.f + expf(-g)) * u * so);
   }
 }
 
 HB_EXPORT int hb_moe_gate_up_rows(const void* xn, int x_dt, long ldx, const void* wgu, int w_dt, const int* expert,
-                                  const float* weight, void* act, int T, int W, int F, int top, int at_output, int E, cudaStream_t s) {
+                                  const float* weight, void* act, int T, int W, int F, int top, int at_output, int E, int grp, cudaStream_t s) {
   if (T <= 0) return 0;
+  if (grp < 1 || F % grp) HB_FAIL("hb_moe_gate_up_rows: %d hidden rows in groups of %d", F, grp);
   const size_t smem = (size_t)W * sizeof(float);
   if (smem > 200 * 1024) HB_FAIL("hb_moe_gate_up_rows: a row of %d does not fit shared memory", W);
   const int vec = (W % 4 == 0) ? 1 : 0;
@@ -241,7 +247,7 @@ HB_EXPORT int hb_moe_gate_up_rows(const void* xn, int x_dt, long ldx, const void
   HB_DISPATCH_2(x_dt, w_dt, "hb_moe_gate_up_rows", do {
     auto kern = moe_gate_up_rows_kernel<TA, TB, TA>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)wgu, expert, weight, (TA*)act, W, F, top, vec, at_output, E);
+    hb_launch(kern, grid, dim3(MG_THREADS), smem, s, (const TA*)xn, ldx, (const TB*)wgu, expert, weight, (TA*)act, W, F, top, vec, at_output, E, grp);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_gate_up_rows");
   return 0;
@@ -440,7 +446,7 @@ struct MmArgs {
   const float* weight;         // ACT: [pairs]
   __nv_bfloat16* act;          // ACT: [sorted rows][Nout]
   float* out;                  // else: [sorted rows][Nout]
-  int Nout, Nw, K, at_output;
+  int Nout, Nw, K, at_output, grp;
 };
 
 template <int NT, int KW, bool ACT>
@@ -450,7 +456,7 @@ __device__ __forceinline__ void mm_round(const MmArgs& A, const __nv_bfloat16* _
   const int tile = warp / KW, part = warp % KW, n0 = (blockIdx.x * TILES + tile) * FT;
   const int nb = A.K >> 5, b0 = nb * part / KW, b1 = nb * (part + 1) / KW;
   // features past the end read the last one's weights, rows past the round's end its first row: their sums are not stored
-  const int ra = min(n0 + g, A.Nout - 1), rb = ACT ? A.Nout + ra : min(n0 + g + 8, A.Nout - 1);
+  const int fa = min(n0 + g, A.Nout - 1), ra = ACT ? moe_gate_row(fa, A.grp) : fa, rb = ACT ? ra + A.grp : min(n0 + g + 8, A.Nout - 1);
   const uint4* wa = (const uint4*)(we + (size_t)ra * A.K) + t;
   const uint4* wb = (const uint4*)(we + (size_t)rb * A.K) + t;
   const uint4* row[NT];
@@ -568,12 +574,13 @@ static void mm_launch(const MmArgs& A, int E, int parts, cudaStream_t s) {
 // act[r] (bfloat16, sorted rows) = silu(s g) * (s u) times the rest of the pair's weight, [g | u] = w[e] row: the gate/up product
 // with its activation in one kernel. parts: of K, 1, 2 or 4 (0: what suits the sizes). Returns 1 (nothing done) where the sizes or element types are not its.
 HB_EXPORT int hb_moe_grouped_act(const void* a, int a_dt, long lda, const int* src, int top, const void* w, int w_dt, const int* offsets,
-                                 const float* weight, void* act, int E, int F, int K, int at_output, int parts, cudaStream_t s) {
+                                 const float* weight, void* act, int E, int F, int K, int at_output, int parts, int grp, cudaStream_t s) {
+  if (grp < 1 || F % grp) HB_FAIL("hb_moe_grouped_act: %d hidden rows in groups of %d", F, grp);
   if (parts != 0 && parts != 1 && parts != 2 && parts != 4) HB_FAIL("hb_moe_grouped_act: %d parts of K", parts);
   if (E <= 0 || F <= 0 || K <= 0) return 0;
   if (!mm_ok(a, a_dt, lda, w, w_dt, K) || !src || E > 65535) return 1;
   mm_launch<true>(MmArgs{(const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, weight, (__nv_bfloat16*)act, nullptr, F, 2 * F,
-                         K, at_output}, E, parts, s);
+                         K, at_output, grp}, E, parts, s);
   HB_CHECK_LAUNCH("hb_moe_grouped_act");
   return 0;
 }
@@ -584,7 +591,7 @@ HB_EXPORT int hb_moe_grouped(const void* a, int a_dt, long lda, const int* src, 
   if (E <= 0 || Nout <= 0 || K <= 0) return 0;
   if (E > 65535) HB_FAIL("hb_moe_grouped: %d experts are too many for this kernel", E);
   if (mm_ok(a, a_dt, lda, w, w_dt, K)) {
-    mm_launch<false>(MmArgs{(const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, nullptr, nullptr, out, Nout, Nout, K, 0}, E, parts, s);
+    mm_launch<false>(MmArgs{(const __nv_bfloat16*)a, lda, src, top, (const __nv_bfloat16*)w, offsets, nullptr, nullptr, out, Nout, Nout, K, 0, 0}, E, parts, s);
     HB_CHECK_LAUNCH("hb_moe_grouped");
     return 0;
   }
@@ -672,7 +679,7 @@ HB_EXPORT int hb_moe_gather(const void* xn, int x_dt, long ldx, const int* src, 
 template <typename TO>
 __global__ void __launch_bounds__(256) moe_act_kernel(const float* __restrict__ gu, const int* __restrict__ src,
                                                       const float* __restrict__ weight, TO* __restrict__ act, long n, int F,
-                                                      int at_output, const int* __restrict__ limit) {
+                                                      int at_output, const int* __restrict__ limit, int grp) {
   hb_pdl_launch();
   hb_pdl_wait();
   if (limit) n = (long)*limit * F;
@@ -681,7 +688,8 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const float* __restrict__ 
     const int j = (int)(idx - r * F);
     const float sw = weight[src[r]];
     const float s = at_output ? 1.f : sw, so = at_output ? sw : 1.f;
-    const float g = s * gu[r * 2 * F + j], u = s * gu[r * 2 * F + F + j];
+    const float* gr = gu + r * 2 * F + moe_gate_row(j, grp);
+    const float g = s * gr[0], u = s * gr[grp];
     act[idx] = hb_from_float<TO>(g / (1.f + expf(-g)) * u * so);
   }
 }
@@ -690,7 +698,7 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const float* __restrict__ 
 template <typename TO>
 __global__ void __launch_bounds__(256) moe_act_vec_kernel(const float* __restrict__ gu, const int* __restrict__ src,
                                                           const float* __restrict__ weight, TO* __restrict__ act, long n4, int F,
-                                                          int at_output, const int* __restrict__ limit) {
+                                                          int at_output, const int* __restrict__ limit, int grp) {
   hb_pdl_launch();
   hb_pdl_wait();
   const int F4 = F >> 2;
@@ -700,7 +708,8 @@ __global__ void __launch_bounds__(256) moe_act_vec_kernel(const float* __restric
     const int j = (int)(idx - r * F4) << 2;
     const float sw = weight[src[r]];
     const float s = at_output ? 1.f : sw, so = at_output ? sw : 1.f;
-    const float4 gv = *(const float4*)(gu + r * 2 * F + j), uv = *(const float4*)(gu + r * 2 * F + F + j);
+    const float* gr = gu + r * 2 * F + moe_gate_row(j, grp);
+    const float4 gv = *(const float4*)gr, uv = *(const float4*)(gr + grp);
     const float g0 = s * gv.x, g1 = s * gv.y, g2 = s * gv.z, g3 = s * gv.w;
     hb_store4(act + r * F + j, make_float4(g0 / (1.f + expf(-g0)) * (s * uv.x) * so, g1 / (1.f + expf(-g1)) * (s * uv.y) * so,
                                            g2 / (1.f + expf(-g2)) * (s * uv.z) * so, g3 / (1.f + expf(-g3)) * (s * uv.w) * so));
@@ -708,19 +717,20 @@ __global__ void __launch_bounds__(256) moe_act_vec_kernel(const float* __restric
 }
 
 HB_EXPORT int hb_moe_act(const float* gu, const int* src, const float* weight, void* act, int o_dt, int pairs, int F,
-                         int at_output, const int* limit, cudaStream_t s) {
+                         int at_output, const int* limit, int grp, cudaStream_t s) {
   if (pairs <= 0) return 0;
-  if (F % 4 == 0 && !(((uintptr_t)gu | (uintptr_t)act) & 15)) {
+  if (grp < 1 || F % grp) HB_FAIL("hb_moe_act: %d hidden rows in groups of %d", F, grp);
+  if (F % 4 == 0 && grp % 4 == 0 && !(((uintptr_t)gu | (uintptr_t)act) & 15)) {
     const long n4 = (long)pairs * (F / 4);
     const int blocks4 = (int)((n4 + 255) / 256 < 148 * 16 ? (n4 + 255) / 256 : 148 * 16);
     HB_DISPATCH_1(o_dt, "hb_moe_act",
-                  (hb_launch(moe_act_vec_kernel<TA>, dim3(blocks4), dim3(256), 0, s, gu, src, weight, (TA*)act, n4, F, at_output, limit)));
+                  (hb_launch(moe_act_vec_kernel<TA>, dim3(blocks4), dim3(256), 0, s, gu, src, weight, (TA*)act, n4, F, at_output, limit, grp)));
     HB_CHECK_LAUNCH("hb_moe_act");
     return 0;
   }
   const long n = (long)pairs * F;
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  HB_DISPATCH_1(o_dt, "hb_moe_act", (hb_launch(moe_act_kernel<TA>, dim3(blocks), dim3(256), 0, s, gu, src, weight, (TA*)act, n, F, at_output, limit)));
+  HB_DISPATCH_1(o_dt, "hb_moe_act", (hb_launch(moe_act_kernel<TA>, dim3(blocks), dim3(256), 0, s, gu, src, weight, (TA*)act, n, F, at_output, limit, grp)));
   HB_CHECK_LAUNCH("hb_moe_act");
   return 0;
 }

@@ -19,6 +19,7 @@ PLAIN_ONLY = os.environ.get("HIPINFER_B200_PLAIN", "0") == "1"
 _p, _i, _l, _f = C.c_void_p, C.c_int, C.c_long, C.c_float
 _SIGS = {
     "hb_gemm_tc": [_p, _l, _p, _l, _p, _l, _i, _i, _i, _i, _i, _p, _p],
+    "hb_gemm_tc_grouped": [_p, _l, _p, _i, _i, _i, _p, _p, _l, _l, _i, _p, _p, _i, _i, _p, _p],
     "hb_gemm_stream": [_p, _l, _p, _l, _p, _l, _i, _i, _i, _i, _p, _l, _p, _i, _p, _p],
     "hb_gemm_stream_plan": [_i, _i, _p, _p, _p, _p],
     "hb_gemm_stream_finish": [_p, _p, _l, _i, _i, _i, _i, _p],
@@ -45,7 +46,7 @@ _SIGS = {
     "hb_rows_norm_supported": [_i, _i],
 }
 _fns = {}
-_LAUNCHES = {"hb_rows_scaled_qkv_rope": 1, "hb_rows_scaled_swiglu": 1, "hb_rows_norm_qkv_rope": 1, "hb_rows_add": 1, "hb_rows_norm_swiglu": 1, "hb_gemm_tc_rope_kv": 1, "hb_gemm_stream_finish": 1, "hb_add_rmsnorm_slices": 1, "hb_rope_kv_slices": 1, "hb_gemm_tc": 1, "hb_gemm_stream": 1, "hb_attn_decode": 1, "hb_flash_prefill": 1, "hb_flash_prefill_tc": 1, "hb_flash_diff_tc": 1, "hb_attn_diff_decode": 1}
+_LAUNCHES = {"hb_rows_scaled_qkv_rope": 1, "hb_rows_scaled_swiglu": 1, "hb_rows_norm_qkv_rope": 1, "hb_rows_add": 1, "hb_rows_norm_swiglu": 1, "hb_gemm_tc_rope_kv": 1, "hb_gemm_stream_finish": 1, "hb_add_rmsnorm_slices": 1, "hb_rope_kv_slices": 1, "hb_gemm_tc": 1, "hb_gemm_stream": 1, "hb_attn_decode": 1, "hb_flash_prefill": 1, "hb_flash_prefill_tc": 1, "hb_flash_diff_tc": 1, "hb_attn_diff_decode": 1, "hb_gemm_tc_grouped": 1}
 _status = None
 
 EPI_F32, EPI_BF16, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_SLICES, EPI_GEGLU_BF16, EPI_GELU_BF16, EPI_RELU2_BF16 = 0, 1, 2, 3, 4, 5, 6, 7
@@ -289,6 +290,22 @@ def linear_gated(a, w, act_out, group, act) -> bool:
     if act != "gelu_tanh" or group != 16 or act_out.dtype != torch.bfloat16 or not _tc_ok(a, w.t) or w.shape[0] % 32:
         return False
     _gemm(a, w.t, act_out, EPI_GEGLU_BF16)
+    return True
+
+
+def grouped_linear(a, w, offsets, out, src, score, at_output, tile_n=0) -> bool:
+    """All experts' products with their sorted rows in one kernel: see ops.moe_sorted_linear."""
+    E, N, K = w.shape
+    gated = out.dtype == torch.bfloat16
+    if (PLAIN_ONLY or not (a.dtype == w.dtype == torch.bfloat16) or E > 256 or K % 8 or a.stride(0) % 8 or a.data_ptr() % 16
+            or w.data_ptr() % 16 or not w.is_contiguous() or out.data_ptr() % 16 or out.stride(0) % (8 if gated else 4)
+            or E * N >= 1 << 31 or (gated and N % 32)):
+        return False
+    assert offsets.dtype == torch.int32 and offsets.numel() >= E + 1 and out.shape == (a.shape[0], N // 2 if gated else N)
+    p = lambda t: None if t is None else t.data_ptr()
+    _call("hb_gemm_tc_grouped", a.data_ptr(), a.stride(0), w.data_ptr(), E, N, K, offsets.data_ptr(), out.data_ptr(), out.stride(0),
+          a.shape[0], EPI_SWIGLU_BF16 if gated else EPI_F32, p(src), p(score), 1 if at_output else 0, int(tile_n),
+          status_word().data_ptr(), _stream())
     return True
 
 

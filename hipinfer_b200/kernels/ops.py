@@ -74,13 +74,13 @@ _SIGS = {
         "hb_split_rounded": [_p, _l, _p, _p, _i, _i, _p],
         "hb_residual_norm": [_p, _p, _p, _p, _p, _p, _i, _f, _f, _f, _p, _f, _p, _i, _i, _i, _p],
         "hb_moe_route": [_p, _i, _l, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _f, _p, _p, _i, _p, _p],
-        "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p],
+        "hb_moe_gate_up_rows": [_p, _i, _l, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p],
         "hb_moe_down_rows": [_p, _i, _p, _i, _p, _p, _l, _i, _i, _i, _i, _i, _p, _l, _p, _p],
         "hb_moe_sort": [_p, _p, _p, _p, _i, _i, _p],
         "hb_moe_grouped": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p],
-        "hb_moe_grouped_act": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p],
+        "hb_moe_grouped_act": [_p, _i, _l, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p],
         "hb_moe_gather": [_p, _i, _l, _p, _p, _i, _i, _i, _p, _p],
-        "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p],
+        "hb_moe_act": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _i, _p],
         "hb_moe_combine": [_p, _p, _p, _l, _i, _i, _i, _p, _p, _i, _l, _p, _p],
     },
     "memory": {
@@ -1430,9 +1430,9 @@ def moe_route(xn: torch.Tensor, router: torch.Tensor, top: int, bias: Optional[t
 
 
 def moe_rows(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor, expert: torch.Tensor, score: torch.Tensor,
-             y: torch.Tensor, at_output: bool = False, identity_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
+             y: torch.Tensor, at_output: bool = False, identity_weight: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
     """y += sum over a row's chosen experts of Wd_e (silu(s Wg_e h) * (s Wu_e h)), row by row with nothing sorted and
-    nothing on the host. wgu [E, 2F, W] (gate rows, then up rows), wdown [E, W, F], y float32 [T, W]. at_output: the
+    nothing on the host. wgu [E, 2F, W] (gate and up rows in turn, `group` of each; 0: gate rows, then up rows), wdown [E, W, F], y float32 [T, W]. at_output: the
     weight multiplies the expert's result instead of its input, Wd_e (s silu(Wg_e h) * (Wu_e h)). Choices from E on are
     identity experts: y also gets identity_weight[t] * xn[t]."""
     _need_cuda(xn, wgu, wdown, expert, score, y, identity_weight)
@@ -1444,7 +1444,7 @@ def moe_rows(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor, expert: t
     assert wgu.is_contiguous() and wdown.is_contiguous() and wdown.shape == (E, W, F) and y.dtype == torch.float32
     act = torch.empty(T * top, F, dtype=xn.dtype, device=xn.device)
     _call("hybrid", "hb_moe_gate_up_rows", xn.data_ptr(), _dt(xn), xn.stride(0), wgu.data_ptr(), _dt(wgu), expert.data_ptr(),
-          score.data_ptr(), act.data_ptr(), T, W, F, top, 1 if at_output else 0, E, _stream())
+          score.data_ptr(), act.data_ptr(), T, W, F, top, 1 if at_output else 0, E, int(group) or F, _stream())
     _call("hybrid", "hb_moe_down_rows", act.data_ptr(), _dt(act), wdown.data_ptr(), _dt(wdown), expert.data_ptr(), y.data_ptr(),
           y.stride(0), T, W, F, top, E, xn.data_ptr(), xn.stride(0), _ptr(identity_weight), _stream())
     return y
@@ -1486,7 +1486,7 @@ def moe_grouped_fast(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor) -
 
 
 def moe_grouped_act(xn: torch.Tensor, src: torch.Tensor, top: int, wgu: torch.Tensor, offsets: torch.Tensor, score: torch.Tensor,
-                    act: torch.Tensor, at_output: bool = False, parts: int = 0) -> bool:
+                    act: torch.Tensor, at_output: bool = False, parts: int = 0, group: int = 0) -> bool:
     """moe_grouped of the gate/up weights [E, 2F, W] and moe_act as one kernel: act [sorted rows, F] (bfloat16). False where it does
     not take the sizes or element types (nothing was done). parts (here and in moe_grouped): K is summed in 1, 2 or 4 parts by
     warps of their own (0: what suits the sizes)."""
@@ -1498,11 +1498,33 @@ def moe_grouped_act(xn: torch.Tensor, src: torch.Tensor, top: int, wgu: torch.Te
         return False
     r = _fn("hybrid", "hb_moe_grouped_act")(xn.data_ptr(), _dt(xn), xn.stride(0), src.data_ptr(), int(top), wgu.data_ptr(), _dt(wgu),
                                             offsets.data_ptr(), score.data_ptr(), act.data_ptr(), E, F2 // 2, W, 1 if at_output else 0,
-                                            int(parts), _stream())
+                                            int(parts), int(group) or F2 // 2, _stream())
     if r < 0:
         raise KernelError(library.load("hybrid").hb_last_error().decode())
     library.launches[0] += r == 0
     return r == 0
+
+
+def moe_sorted_linear(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, out: torch.Tensor, src: Optional[torch.Tensor] = None,
+                      score: Optional[torch.Tensor] = None, at_output: bool = False) -> torch.Tensor:
+    """The products of every expert with its block of sorted rows as one tcgen05 kernel (csrc/gemm_tc.cu): a [sorted rows, K], w [E, N,
+    K], offsets int32 [>= E + 1] on the device; out float32 [rows, N], or bfloat16 [rows, N / 2] = silu(gate) * up over
+    16-interleaved weight rows with the pairs' scores (src, score, at_output as in moe_act). Rows beyond the last expert's are left
+    alone, nothing is read by the host. For sizes that `moe_sorted_fast` takes."""
+    from . import fast
+
+    if not fast.grouped_linear(a, w, offsets, out, src, score, at_output):
+        raise KernelError(f"moe_sorted_linear: {tuple(w.shape)} weights are not this kernel's")
+    return out
+
+
+def moe_sorted_fast(xn: torch.Tensor, wgu: torch.Tensor, wdown: torch.Tensor) -> bool:
+    """Whether moe_sorted_linear takes a routed layer's sizes (16-interleaved gate and up rows): bfloat16, at most 256 experts."""
+    from . import fast
+
+    E, F2, W = wgu.shape
+    return (xn.is_cuda and not fast.PLAIN_ONLY and xn.dtype == wgu.dtype == wdown.dtype == torch.bfloat16 and E <= 256 and W % 8 == 0
+            and F2 % 32 == 0 and E * max(F2, W) < 1 << 31 and (wgu.data_ptr() | wdown.data_ptr()) % 16 == 0)
 
 
 def moe_gather(xn: torch.Tensor, src: torch.Tensor, top: int, limit: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -1515,14 +1537,14 @@ def moe_gather(xn: torch.Tensor, src: torch.Tensor, top: int, limit: Optional[to
 
 
 def moe_act(gu: torch.Tensor, src: torch.Tensor, score: torch.Tensor, out: torch.Tensor, at_output: bool = False,
-            limit: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[r] = silu(s g) * (s u) of the sorted rows' float32 [g | u], s the score of the row's pair; with at_output
+            limit: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
+    """out[r] = silu(s g) * (s u) of the sorted rows' float32 gate and up columns (`group` of each in turn; 0: g, then u), s the score of the row's pair; with at_output
     s silu(g) * u (the weight of the expert's result, brought in before the linear down product). limit (int32 [1] on the
     device): only rows below it."""
     pairs, F = out.shape
     assert gu.dtype == torch.float32 and gu.is_contiguous() and gu.shape == (pairs, 2 * F) and out.is_contiguous()
     _call("hybrid", "hb_moe_act", gu.data_ptr(), src.data_ptr(), score.data_ptr(), out.data_ptr(), _dt(out), pairs, F,
-          1 if at_output else 0, _ptr(limit), _stream())
+          1 if at_output else 0, _ptr(limit), int(group) or F, _stream())
     return out
 
 

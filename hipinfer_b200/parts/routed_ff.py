@@ -22,11 +22,12 @@ With `identity` the last that many of the experts + identity router rows are exp
 With `shared_size` a shared expert of the same form and that size runs for every token and is added; with `shared_gate` its
 result is multiplied by sigmoid(w . h), one number per token (made beside the router's logits). One without a gate is a gated
 feed-forward like any other and runs on its kernels (parts/feed_forward.py).
-Steps of single rows (decoding) run on the device alone (csrc/moe.cu), so they replay from a CUDA graph: sorted by expert so
-that an expert's weights are read once for all of its rows (in 32-bit, and at sizes the warp-MMA kernels do not take, a few
-rows run one by one). A step with prompt
-portions sorts its (row, choice) pairs by expert and gives each expert's block of rows to the ordinary products (the
-tensor-core kernels in bfloat16), for which the host reads the experts' row counts once a layer.
+A step's (row, choice) pairs are sorted by expert, so that an expert's weights are read once for all of its rows, and in
+bfloat16 all of it runs on the device alone (csrc/moe.cu, gemm_tc.cu), so that it replays from a CUDA graph: where the experts
+have few rows each, warp-MMA kernels stream their weights (gate/up product with its activation, then the down product); where they
+have more, two tcgen05 kernels do the same over tiles of 128 rows. In 32-bit (and at sizes those kernels do not take) a few rows
+run one by one, single rows of a larger step on any-size kernels, and in a step with prompt portions each expert's block of rows
+goes to the ordinary products, for which the host reads the experts' row counts once a layer.
 
 params: hidden_size, experts, top, expert_size, score (default "sigmoid"), weight_at (default "input"), router_bias
 (default False), groups (count, keep) (default none), identity (default 0), weight_scale (default 1), shared_size (default none), shared_gate (default
@@ -45,6 +46,8 @@ from .feed_forward import GatedFF
 from .registry import Part, register_part, to_compute
 
 SORTED_MIN_PAIRS = 64     # fewer (row, choice) pairs than this never go to the ordinary products
+TILES_MIN_ROWS = 16       # from this many pairs a choice on, on average, the experts' rows go to the tcgen05 kernels
+GROUP = 16                # gate and up rows in turn, as the gated epilogues want them
 SHARED_MIN_ROWS = 9       # fewer rows run the shared expert row by row
 GROUPED_MIN_PAIRS = 20    # fewer than this run row by row where the grouped kernels are the any-size ones
 
@@ -128,7 +131,9 @@ class RoutedFF(Part):
         mats = [t(self._expert(i, k)) for i in range(self.experts) for k in ("gate", "up", "down")]
         dt = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
         E, F, W = self.experts, self.inter, self.hidden
-        self.wgu = torch.stack([torch.cat([mats[3 * i].to(dt), mats[3 * i + 1].to(dt)], 0) for i in range(E)], 0).contiguous()
+        G = self.group = GROUP if F % GROUP == 0 else F
+        turn = lambda gate, up: torch.stack([gate.to(dt).reshape(F // G, G, W), up.to(dt).reshape(F // G, G, W)], 1).reshape(2 * F, W)
+        self.wgu = torch.stack([turn(mats[3 * i], mats[3 * i + 1]) for i in range(E)], 0).contiguous()
         self.wdown = torch.stack([mats[3 * i + 2].to(dt) for i in range(E)], 0).contiguous()      # [E, W, F]
         assert self.wgu.shape == (E, 2 * F, W) and self.wdown.shape == (E, W, F)
         self.w_gu_e = [ops.Weight(self.wgu[i]) for i in range(E)]
@@ -175,33 +180,40 @@ class RoutedFF(Part):
         elif self.shared:
             self._add_shared(xn, x, shared_weight)
         if T * top < GROUPED_MIN_PAIRS and not ops.moe_grouped_fast(xn, self.wgu, self.wdown):
-            ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output, idw)
+            ops.moe_rows(xn, self.wgu, self.wdown, expert, score, x, self.at_output, idw, self.group)
             return None
         offsets, pos, src = ops.moe_sort(expert, self.choices)
         # identity experts come last in the order: their sorted rows hold nothing
         limit, rows_in = (offsets[self.experts:], xn) if self.identity else (None, None)
-        if getattr(batch, "max_q_len", 1) <= 1 or T * top < SORTED_MIN_PAIRS:
+        tiles = self.group == GROUP and ops.moe_sorted_fast(xn, self.wgu, self.wdown)
+        if T * top < TILES_MIN_ROWS * self.choices if tiles else getattr(batch, "max_q_len", 1) <= 1 or T * top < SORTED_MIN_PAIRS:
             act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
-            if not ops.moe_grouped_act(xn, src, top, self.wgu, offsets, score, act, self.at_output):
+            if not ops.moe_grouped_act(xn, src, top, self.wgu, offsets, score, act, self.at_output, group=self.group):
                 gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
                 ops.moe_grouped(xn, src, top, self.wgu, offsets, gu)
-                ops.moe_act(gu, src, score, act, self.at_output, limit)
+                ops.moe_act(gu, src, score, act, self.at_output, limit, self.group)
             planes.record(batch, "activation", act)
             ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
             ops.moe_grouped(act, None, 1, self.wdown, offsets, ys)
             ops.moe_combine(ys, pos, x, top, limit, rows_in, idw)
             return None
         xs = ops.moe_gather(xn, src, top, limit)
+        act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
+        ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
+        if tiles:
+            ops.moe_sorted_linear(xs, self.wgu, offsets, act, src, score, self.at_output)
+            planes.record(batch, "activation", act)
+            ops.moe_sorted_linear(act, self.wdown, offsets, ys)
+            ops.moe_combine(ys, pos, x, top, limit, rows_in, idw)
+            return None
         bounds = offsets.tolist()                      # the one read by the host: how many rows each expert has
         gu = torch.empty(T * top, 2 * F, dtype=torch.float32, device=xn.device)
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
                 ops.linear(xs[lo:hi], self.w_gu_e[e], gu[lo:hi])
-        act = torch.empty(T * top, F, dtype=self.ctx.dtype, device=xn.device)
-        ops.moe_act(gu, src, score, act, self.at_output, limit)
+        ops.moe_act(gu, src, score, act, self.at_output, limit, self.group)
         planes.record(batch, "activation", act)
-        ys = torch.empty(T * top, self.hidden, dtype=torch.float32, device=xn.device)
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
