@@ -302,6 +302,20 @@ def test_attention_part_in_portions(dtype, m, cuts):
     close(_attention(dtype, m, h, w, cuts), want, dtype, tol=4e-5 if dtype == torch.float32 else 2e-2)
 
 
+@pytest.mark.parametrize("page", [8, 32, 64])
+@pytest.mark.parametrize("H,G,D,window", [(1, 1, 32, 50), (4, 2, 32, 700), (6, 2, 32, 513), (4, 1, 32, None), (3, 1, 64, 300), (8, 2, 64, None), (2, 2, 64, 257)])
+def test_attention_over_pages_of_other_sizes_and_several_chunks(page, H, G, D, window):
+    """One to four heads a kv head, windows of several key chunks of the decode kernel, pages of 8 to 64 tokens: a long portion, then
+    single tokens far into the sequence (whose window starts inside a page, on its edge and on a chunk's edge)."""
+    m = dict(heads=H, kv_heads=G, dim=D, vdim=2 * D, scale=D ** -0.5, diff=0.4, rot=dict(dims=D, base=3000.0))
+    if window:
+        m["mask"] = dict(size=window)
+    dtype, T = torch.bfloat16, 1160
+    w, h = _weights(m, dtype), rnd(T, 48, seed=20).to(dtype).float()
+    want = plain.attention(h.double(), {n: t.double() for n, t in w.items()}, m, 1e-5)
+    close(_attention(dtype, m, h, w, (1020, 3, 1, 70) + (1,) * 66, page=page), want, dtype, tol=2e-2)
+
+
 @BOTH
 @pytest.mark.parametrize("window", [1, 2, 16, 63, 64, 65, 128, 150])
 @pytest.mark.parametrize("dim,vdim", [(32, 64), (64, 128), (24, 16)])
@@ -478,6 +492,46 @@ def test_experts_with_identity_and_shared_ones(dtype, W, Fe, Fs, r, T, prompt):
     if n_id and T > 8:
         chosen = plain.route(h.double(), t["mlp.router"].double(), t["mlp.correction"].double(), r)[0]
         assert bool((chosen >= r["experts"]).any()) and bool((chosen < r["experts"]).any())
+
+
+@pytest.mark.parametrize("E,W,F,T,top,n_id", [(3, 64, 32, 40, 2, 1), (8, 128, 96, 300, 2, 4), (5, 96, 160, 515, 3, 0), (70, 64, 64, 900, 4, 10),
+                                              (200, 64, 32, 600, 3, 0), (1, 64, 128, 129, 1, 0), (4, 256, 48, 1, 1, 3)])
+@pytest.mark.parametrize("at_output", [True, False])
+def test_all_experts_products_in_one_kernel(E, W, F, T, top, n_id, at_output):
+    """Blocks of sorted rows that end inside a tile of 128, experts without rows, more than 64 experts, both tile widths; rows of
+    identity experts are left alone. The weight multiplies the result, or both halves of the gate/up product."""
+    from hipinfer_b200.kernels import fast, ops
+
+    g = torch.Generator().manual_seed(E)
+    wgu, wd = (torch.randn(*s, generator=g) * s[2] ** -0.5 for s in ((E, 2 * F, W), (E, W, F)))
+    wgu, wd, x = wgu.bfloat16(), wd.bfloat16(), torch.randn(T, W, generator=g).bfloat16()
+    expert = torch.stack([torch.randperm(E + n_id, generator=g)[:top] for _ in range(T)]).to(torch.int32)
+    if E > 2:
+        expert[expert == 1] = 0                                  # an expert without rows, another with many
+    score = torch.rand(T, top, generator=g)
+    offsets, pos, src = ops.moe_sort(expert.to(DEV), E + n_id)
+    xs, sc = ops.moe_gather(x.to(DEV), src, top, offsets[E:]), score.to(DEV)
+    b, order = offsets.tolist(), src.cpu().long()
+    for tile in (128, 256, 0):
+        act = torch.full((T * top, F), 7.0, dtype=torch.bfloat16, device=DEV)
+        ys = torch.full((T * top, W), 7.0, device=DEV)
+        assert fast.grouped_linear(xs, wgu.to(DEV), offsets, act, src, sc, at_output, tile)
+        assert fast.grouped_linear(act, wd.to(DEV), offsets, ys, None, None, False, tile)
+        for e in range(E):
+            rows = order[b[e]:b[e + 1]]
+            if not rows.numel():
+                continue
+            gu = (x[rows // top].double() @ wgu[e].double().T).view(-1, F // 16, 2, 16)
+            gate, up, s = gu[:, :, 0].reshape(-1, F), gu[:, :, 1].reshape(-1, F), score.flatten()[rows][:, None].double()
+            close(act[b[e]:b[e + 1]], plain.silu(gate) * up * s if at_output else plain.silu(gate * s) * (up * s), torch.bfloat16)
+            close(ys[b[e]:b[e + 1]], act[b[e]:b[e + 1]].cpu().double() @ wd[e].double().T, torch.float32, tol=1e-4)
+        assert bool((act[b[E]:] == 7).all()) and bool((ys[b[E]:] == 7).all())
+    # the same by the kernels for few rows
+    few = torch.full((T * top, F), 7.0, dtype=torch.bfloat16, device=DEV)
+    for parts in (1, 2, 4):
+        assert ops.moe_grouped_act(x.to(DEV), src, top, wgu.to(DEV), offsets, sc, few, at_output, parts, 16)
+        close(few[:b[E]], act[:b[E]].cpu(), torch.bfloat16)
+        assert bool((few[b[E]:] == 7).all())
 
 
 def test_a_step_all_of_whose_choices_are_identity_experts():
