@@ -415,7 +415,7 @@ ROUTERS = [dict(experts=9, identity=6, top=4, groups=dict(count=5, keep=3)), dic
 @BOTH
 @pytest.mark.parametrize("r", ROUTERS, ids=lambda r: f"{r['experts']}-{r.get('identity', 0)}-{r['top']}-{(r.get('groups') or {}).get('count', 1)}")
 @pytest.mark.parametrize("W", [64, 50, 2048])
-@pytest.mark.parametrize("T", [3, 400])
+@pytest.mark.parametrize("T", [3, 400, 701])
 def test_router(dtype, r, W, T):
     """Corrections of both signs move the choice but not the weights; a group is as good as its best; choice scores below zero are
     still chosen; the identity experts' weights are summed. Rows whose call is close are left out."""
