@@ -34,66 +34,77 @@
 
 constexpr int MR_THREADS = 512;
 
-// A warp a router row (and the shared expert's gate), TOK tokens' rows read beside it (a router row is fetched once for all of
-// them); then a warp a token ranks the groups, marks the experts of those that do not stay as taken (NaN), and picks the largest
-// `top` times, ties to the lower index. A token's sums do not depend on TOK.
-template <typename TA, typename TW, int TOK>
+// Eight elements of two rows multiplied and added up: one 16-byte access a row where both are bfloat16.
+__device__ __forceinline__ float mr_dot8(const __nv_bfloat16* a, const __nv_bfloat16* w, float acc) {
+  const uint4 x = *(const uint4*)a, y = *(const uint4*)w;
+  const __nv_bfloat162 *xp = (const __nv_bfloat162*)&x, *yp = (const __nv_bfloat162*)&y;
+#pragma unroll
+  for (int i = 0; i < 4; i++) {
+    const float2 u = __bfloat1622float2(xp[i]), v = __bfloat1622float2(yp[i]);
+    acc = fmaf(v.x, u.x, acc);
+    acc = fmaf(v.y, u.y, acc);
+  }
+  return acc;
+}
+template <typename TA, typename TW>
+__device__ __forceinline__ float mr_dot8(const TA* a, const TW* w, float acc) {
+#pragma unroll
+  for (int i = 0; i < 8; i += 4) {
+    const float4 u = hb_load4(a + i), v = hb_load4(w + i);
+    acc = fmaf(v.x, u.x, acc);
+    acc = fmaf(v.y, u.y, acc);
+    acc = fmaf(v.z, u.z, acc);
+    acc = fmaf(v.w, u.w, acc);
+  }
+  return acc;
+}
+
+// A warp a router row (and the shared expert's gate), the token's row read beside it; then warp 0 ranks the groups, marks the
+// experts of those that do not stay as taken (NaN), and picks the largest `top` times, ties to the lower index.
+template <typename TA, typename TW>
 __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restrict__ xn, long ldx, const TW* __restrict__ router,
                                                                const TW* __restrict__ bias, int* __restrict__ expert,
-                                                               float* __restrict__ weight, int T, int W, int E, int top, int mode,
+                                                               float* __restrict__ weight, int W, int E, int top, int mode,
                                                                const TW* __restrict__ correction, int groups, int keep, float scale,
                                                                const TW* __restrict__ shared_gate, float* __restrict__ shared_weight,
                                                                int vec, int n_real, float* __restrict__ identity_weight) {
-  extern __shared__ float mr_sm[];     // per token: [E] the scores, [E] those without the correction, [groups] the groups' ranks
+  extern __shared__ float mr_sm[];     // [E] the scores, [E] those without the correction, [E] corrections, [groups] the groups' ranks, [top] weights
+  float* sc = mr_sm;
+  float* plain = sc + E;
+  float* corr = plain + E;
+  float* gs = corr + E;
+  float* picked = gs + groups;
   hb_pdl_launch();
   hb_pdl_wait();
-  const int t0 = blockIdx.x * TOK, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, per = 2 * E + groups;
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const TA* row = xn + (size_t)t * ldx;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) corr[e] = correction ? hb_to_float(correction[e]) : 0.f;     // (asked for beside the rows)
   for (int e = warp; e < E + (shared_gate ? 1 : 0); e += nw) {
     const TW* wr = e < E ? router + (size_t)e * W : shared_gate;
-    float sums[TOK];
-#pragma unroll
-    for (int k = 0; k < TOK; k++) sums[k] = 0.f;
+    float acc = 0.f;
     if (vec) {
-#pragma unroll(TOK > 1 ? 4 : 8)
-      for (int i = lane * 4; i < W; i += 128) {
-        const float4 wv = hb_load4(wr + i);
-#pragma unroll
-        for (int k = 0; k < TOK; k++) {
-          const float4 av = hb_load4(xn + (size_t)min(t0 + k, T - 1) * ldx + i);
-          sums[k] = fmaf(wv.x, av.x, sums[k]);
-          sums[k] = fmaf(wv.y, av.y, sums[k]);
-          sums[k] = fmaf(wv.z, av.z, sums[k]);
-          sums[k] = fmaf(wv.w, av.w, sums[k]);
-        }
-      }
+#pragma unroll 8
+      for (int i = lane * 8; i < W; i += 256) acc = mr_dot8(row + i, wr + i, acc);
     } else {
-      for (int i = lane; i < W; i += 32)
-#pragma unroll
-        for (int k = 0; k < TOK; k++) sums[k] = fmaf(hb_to_float(xn[(size_t)min(t0 + k, T - 1) * ldx + i]), hb_to_float(wr[i]), sums[k]);
+      for (int i = lane; i < W; i += 32) acc = fmaf(hb_to_float(row[i]), hb_to_float(wr[i]), acc);
     }
-#pragma unroll
-    for (int k = 0; k < TOK; k++) {
-      float acc = hb_warp_sum(sums[k]);
-      const int t = t0 + k;
-      if (lane != 0 || t >= T) continue;
-      float* sc = mr_sm + k * per;
-      float* plain = sc + E;
-      if (e == E) {
-        shared_weight[t] = 1.f / (1.f + expf(-acc));
-        continue;
-      }
-      if (bias) acc += hb_to_float(bias[e]);
-      const float v = mode == 1 || mode == 3 ? acc : 1.f / (1.f + expf(-acc));
-      sc[e] = mode == 2 ? v + hb_to_float(correction[e]) : v;
-      plain[e] = v;
+    acc = hb_warp_sum(acc);
+    if (lane != 0) continue;
+    if (e == E) {
+      shared_weight[t] = 1.f / (1.f + expf(-acc));
+      continue;
     }
+    if (bias) acc += hb_to_float(bias[e]);
+    const float v = mode == 1 || mode == 3 ? acc : 1.f / (1.f + expf(-acc));
+    sc[e] = v;
+    plain[e] = v;
   }
   __syncthreads();
-  const int t = t0 + warp;
-  if (warp >= TOK || t >= T) return;
-  float* sc = mr_sm + warp * per;
-  float* plain = sc + E;
-  float* gs = plain + E;
+  if (warp != 0) return;
+  if (mode == 2) {
+    for (int e = lane; e < E; e += 32) sc[e] += corr[e];
+    __syncwarp();
+  }
   if (mode == 3) {                       // the softmax over all E, then the corrections
     float mx = -INFINITY, sum = 0.f;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, plain[e]);
@@ -103,7 +114,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
     for (int e = lane; e < E; e += 32) {
       const float v = expf(plain[e] - mx) / sum;
       plain[e] = v;
-      sc[e] = v + (correction ? hb_to_float(correction[e]) : 0.f);
+      sc[e] = v + corr[e];
     }
     __syncwarp();
   }
@@ -127,7 +138,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
     }
     __syncwarp();
   }
-  float first = 0.f, den = 0.f;
+  float first = 0.f, den = 0.f, idw = 0.f;
   for (int k = 0; k < top; k++) {
     float bs = -INFINITY;
     int best = E;
@@ -146,24 +157,19 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const TA* __restr
     if (k == 0) first = bs;
     const float w = mode == 1 ? expf(bs - first) : plain[best];
     den += w;
+    if (best >= n_real) idw += w;
     if (lane == 0) {
       expert[(size_t)t * top + k] = best;
-      weight[(size_t)t * top + k] = w;
+      picked[k] = w;
       sc[best] = __int_as_float(0x7fc00000);
     }
     __syncwarp();
   }
-  if (identity_weight && lane == 0) {
-    float w = 0.f;
-    for (int k = 0; k < top; k++)
-      if (expert[(size_t)t * top + k] >= n_real) w += weight[(size_t)t * top + k];
-    identity_weight[t] = w;
+  if (identity_weight && lane == 0) identity_weight[t] = idw;
+  for (int k = lane; k < top; k += 32) {
+    const float w = picked[k];
+    weight[(size_t)t * top + k] = mode == 1 ? w / den : mode == 2 ? w / (den + 1e-20f) * scale : w;
   }
-  if ((mode == 1 || mode == 2) && lane == 0)
-    for (int k = 0; k < top; k++) {
-      const float w = weight[(size_t)t * top + k];
-      weight[(size_t)t * top + k] = mode == 1 ? w / den : w / (den + 1e-20f) * scale;
-    }
 }
 
 // mode 0: the scores are sigmoid(z) and the chosen scores are the weights; mode 1: the largest logits z choose and the
@@ -184,18 +190,15 @@ HB_EXPORT int hb_moe_route(const void* xn, int x_dt, long ldx, const void* route
     HB_FAIL("hb_moe_route: %d experts in %d groups of which %d stay, %d chosen", E, groups, keep, top);
   if (shared_gate && !shared_weight) HB_FAIL("hb_moe_route: a shared expert's gate needs a place for its result");
   if (top < 1 || top > E) HB_FAIL("hb_moe_route: top %d of %d experts", top, E);
-  const int vec = W % 4 == 0 && ldx % 4 == 0 && !(((uintptr_t)router | (uintptr_t)shared_gate | (uintptr_t)xn) & 15);
-  // many tokens: four a block, whose warps then read a router row once for all of them
-  const int tok = T >= 592 ? 4 : 1, rows = E + (shared_gate ? 1 : 0), want = rows < tok ? tok : rows;
-  const int threads = 32 * (want < MR_THREADS / 32 ? want : MR_THREADS / 32);
-  const size_t smem = (size_t)tok * (2 * E + groups) * sizeof(float);
+  const size_t smem = (size_t)(3 * E + groups + top) * sizeof(float);
+  const int vec = W % 8 == 0 && ldx % 8 == 0 && !(((uintptr_t)router | (uintptr_t)shared_gate | (uintptr_t)xn) & 15);
+  const int rows = E + (shared_gate ? 1 : 0), threads = 32 * (rows < MR_THREADS / 32 ? rows : MR_THREADS / 32);
   if (smem > 200 * 1024) HB_FAIL("hb_moe_route: %d experts in %d groups do not fit shared memory", E, groups);
   HB_DISPATCH_2(x_dt, w_dt, "hb_moe_route", do {
-    auto kern = tok == 4 ? moe_route_kernel<TA, TB, 4> : moe_route_kernel<TA, TB, 1>;
+    auto kern = moe_route_kernel<TA, TB>;
     if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    hb_launch(kern, dim3((T + tok - 1) / tok), dim3(threads), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert,
-              weight, T, W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight, vec, n_real,
-              identity_weight);
+    hb_launch(kern, dim3(T), dim3(threads), smem, s, (const TA*)xn, ldx, (const TB*)router, (const TB*)bias, expert, weight,
+              W, E, top, mode, (const TB*)correction, groups, keep, scale, (const TB*)shared_gate, shared_weight, vec, n_real, identity_weight);
   } while (0));
   HB_CHECK_LAUNCH("hb_moe_route");
   return 0;
