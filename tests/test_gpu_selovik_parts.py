@@ -282,7 +282,7 @@ def _weights(m, dtype, W=48, gain=0.2):
     return {n: t.to(dtype) for n, t in w.items()}
 
 
-ATTN = [dict(heads=4, kv_heads=2, dim=32, vdim=64, scale=0.2, diff=0.5, mask=dict(size=40), rot=dict(dims=16, base=1000.0, scaling=dict(factor=4.0, original=64, fast=32.0, slow=1.0))),
+ATTN = [dict(heads=9, kv_heads=3, dim=32, vdim=64, scale=0.2, diff=0.45, mask=dict(size=37), rot=dict(dims=16, base=1000.0, scaling=dict(factor=6.0, original=64, fast=32.0, slow=1.0))),
         dict(heads=6, kv_heads=2, dim=64, vdim=128, scale=0.125, diff=0.2, mask=dict(size=64), rot=dict(dims=64, base=500.0)),
         dict(heads=3, kv_heads=3, dim=10, vdim=6, scale=0.3, diff=0.8, mask=dict(size=17), rot=dict(dims=6, base=100.0)),
         dict(heads=4, kv_heads=1, dim=128, vdim=64, scale=0.1, diff=0.4, mask=dict(size=65)),
@@ -303,7 +303,7 @@ def test_attention_part_in_portions(dtype, m, cuts):
 
 
 @pytest.mark.parametrize("page", [8, 32, 64])
-@pytest.mark.parametrize("H,G,D,window", [(1, 1, 32, 50), (4, 2, 32, 700), (6, 2, 32, 513), (4, 1, 32, None), (3, 1, 64, 300), (8, 2, 64, None), (2, 2, 64, 257)])
+@pytest.mark.parametrize("H,G,D,window", [(1, 1, 32, 50), (8, 4, 32, 700), (6, 2, 32, 513), (4, 1, 32, None), (3, 1, 64, 300), (8, 2, 64, None), (2, 2, 64, 257)])
 def test_attention_over_pages_of_other_sizes_and_several_chunks(page, H, G, D, window):
     """One to four heads a kv head, windows of several key chunks of the decode kernel, pages of 8 to 64 tokens: a long portion, then
     single tokens far into the sequence (whose window starts inside a page, on its edge and on a chunk's edge)."""
@@ -494,7 +494,7 @@ def test_experts_with_identity_and_shared_ones(dtype, W, Fe, Fs, r, T, prompt):
         assert bool((chosen >= r["experts"]).any()) and bool((chosen < r["experts"]).any())
 
 
-@pytest.mark.parametrize("E,W,F,T,top,n_id", [(3, 64, 32, 40, 2, 1), (8, 128, 96, 300, 2, 4), (5, 96, 160, 515, 3, 0), (70, 64, 64, 900, 4, 10),
+@pytest.mark.parametrize("E,W,F,T,top,n_id", [(3, 64, 32, 40, 2, 1), (9, 128, 80, 300, 2, 5), (5, 96, 160, 515, 3, 0), (70, 64, 64, 900, 4, 10),
                                               (200, 64, 32, 600, 3, 0), (1, 64, 128, 129, 1, 0), (4, 256, 48, 1, 1, 3)])
 @pytest.mark.parametrize("at_output", [True, False])
 def test_all_experts_products_in_one_kernel(E, W, F, T, top, n_id, at_output):
