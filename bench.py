@@ -432,9 +432,9 @@ def breakdown(layers: int, batch: int, prefill: bool = False) -> int:
 # --design torirax: the Torirax design beside the Llama decoder at equal layer sizes (random weights)
 # ------------------------------------------------------------------------------------------
 DESIGN_SIZES = {
-    # width, layers, heads, kv heads, feed-forward, vocabulary: the 1B and (with 8 of its 32 layers) the 8B Llama layer sizes
+    # width, layers, heads, kv heads, feed-forward, vocabulary: the 1B and (with 16 of its 32 layers) the 8B Llama layer sizes
     "1b": dict(width=2048, layers=16, heads=32, kv=8, head_dim=64, ff=8192, vocab=128256),
-    "8b": dict(width=4096, layers=8, heads=32, kv=8, head_dim=128, ff=14336, vocab=128256),
+    "8b": dict(width=4096, layers=16, heads=32, kv=8, head_dim=128, ff=14336, vocab=128256),
 }
 
 
